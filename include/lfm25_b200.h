@@ -630,6 +630,107 @@ const uint32_t* lfm25_decode_executor_sampled(const lfm25_decode_executor* execu
 const void* lfm25_decode_executor_logits(const lfm25_decode_executor* executor);      /* bf16 [maximum_tokens, 65536] */
 
 /* ------------------------------------------------------------------------------------------
+ * Layer-stack models: a decoder described layer by layer, for designs other than the one above
+ * ------------------------------------------------------------------------------------------
+ * A layer is x <- x + (mixer(h + conv(h)) + ff(n)) with h = norm(x) * mixer_norm, n = norm(x) * ff_norm and conv a causal
+ * per-channel convolution over time; the mixer is attention over the paged cache or a recurrence over a state that
+ * every request slot carries.  Every size and constant is a field; bf16 weights, activations in bf16 or f32, and the
+ * residual stream, norms, rotation, softmax and recurrent state in f32 in both.  Unlike lfm25_model, which fixes the
+ * LFM2 shapes, nothing here is a compile-time constant except the page size (16 tokens). */
+
+#define LFM25_ACTIVATION_BF16 0u
+#define LFM25_ACTIVATION_F32 1u
+#define LFM25_MIXER_ATTENTION 0u
+#define LFM25_MIXER_GENERAL_DELTA 1u
+
+/* Matrix [n, k] in bf16; rows beyond the layer's own columns (up to n) are zero. */
+typedef struct lfm25_stack_linear {
+    const void* weight;
+    size_t n;
+    size_t k;
+} lfm25_stack_linear;
+
+typedef struct lfm25_stack_layer {
+    uint32_t mixer;                    /* LFM25_MIXER_* */
+    const void* mixer_norm;            /* bf16 [width] */
+    const void* ff_norm;               /* bf16 [width]; NULL with ff == 0 */
+    const void* conv;                  /* bf16 [conv_taps, width], tap-major, last row = current token */
+    size_t conv_offset;                /* of [conv_taps - 1, width] activations in a request slot's record (bytes) */
+    /* projections of the mixer input, one matrix: attention q | k | v; delta rule r | k | v | g | a | z */
+    lfm25_stack_linear projection;
+    /* output projection of the mixer beside that of the feed-forward: [width, mixer columns + ff] */
+    lfm25_stack_linear output;
+    /* feed-forward: up -> PolyNorm a N(z) + b N(z^2) + c N(z^3) + e -> (part of output); ff == 0: none */
+    uint32_t ff;
+    lfm25_stack_linear up;
+    float poly[4];
+    uint32_t heads;
+    uint32_t dim;                      /* query / key size per head; delta rule: also the value size, <= 256 */
+    /* attention */
+    uint32_t kv_heads;
+    uint32_t vdim;
+    uint32_t rot_dims;                 /* leading rotated dimensions (even), 0 = none */
+    uint32_t chunk;                    /* tokens of a position-0-based chunk that see each other, 0 = all before */
+    float scale;
+    const float* inv_freq;             /* f32 [rot_dims / 2] */
+    const void* bias;                  /* bf16 q | k | v, or NULL */
+    const void* query_norm;            /* bf16 [heads * dim] */
+    const void* key_norm;              /* bf16 [kv_heads * dim] */
+    void* key_cache;                   /* activations [num_pages, kv_heads, 16, dim] */
+    void* value_cache;                 /* activations [num_pages, kv_heads, 16, vdim] */
+    /* generalised delta rule */
+    uint32_t rank;
+    const void* decay_up;              /* bf16 [heads * dim, rank] */
+    const void* decay_base;            /* bf16 [heads * dim] */
+    const void* removal_bias;          /* bf16 [heads * dim] */
+    const void* head_norm;             /* bf16 [heads * dim] */
+    size_t state_offset;               /* of f32 [heads, dim (value), dim (key)] in a request slot's record (bytes) */
+} lfm25_stack_layer;
+
+typedef struct lfm25_stack_model {
+    uint32_t num_layers;
+    const lfm25_stack_layer* layers;   /* host array */
+    uint32_t activation;               /* LFM25_ACTIVATION_* */
+    uint32_t conv_taps;
+    size_t vocab;
+    size_t width;
+    float norm_eps;
+    const void* embedding;             /* bf16 [vocab, width] */
+    const void* final_norm;            /* bf16 [width] */
+    lfm25_stack_linear head;           /* [>= vocab, width] */
+    void* records;                     /* [num_request_slots, record_bytes]: the recurrent state of every layer */
+    size_t record_bytes;               /* a multiple of 256 */
+    size_t num_request_slots;
+    size_t num_pages;
+} lfm25_stack_model;
+
+/* Steps of a layer-stack model on fixed scratch: up to maximum_tokens tokens in up to maximum_rows sequences (or rows
+ * that get logits).  The model struct, its layer array and the device memory behind them must outlive the executor. */
+typedef struct lfm25_stack_executor lfm25_stack_executor;
+int32_t lfm25_stack_executor_create(lfm25_blaslt* blaslt, const lfm25_stack_model* model, size_t maximum_tokens,
+                                    size_t maximum_rows, lfm25_stack_executor** out);
+void lfm25_stack_executor_destroy(lfm25_stack_executor* executor);
+/* One decode step (one token per sequence); advance as in lfm25_decode_executor_forward. */
+int32_t lfm25_stack_executor_forward(lfm25_stack_executor* executor, const lfm25_decode_batch* batch, uint32_t advance);
+/* The same step replayed from a CUDA graph, see lfm25_decode_executor_step_graph. */
+int32_t lfm25_stack_executor_step_graph(lfm25_stack_executor* executor, const lfm25_decode_batch* batch,
+                                        uint32_t advance);
+/* One mixed step.  batch->output_rows holds num_output_rows token indices in any order; row i of logits / sampled
+ * belongs to output_rows[i].  0: the step only fills cache and state. */
+int32_t lfm25_stack_executor_forward_ragged(lfm25_stack_executor* executor, const lfm25_ragged_batch* batch,
+                                            size_t num_output_rows);
+int32_t lfm25_stack_executor_download_sampled(lfm25_stack_executor* executor, uint32_t* host, size_t count);
+/* Logits of the last step as f32 [rows, vocab] on the host; synchronises the stream. */
+int32_t lfm25_stack_executor_read_logits(lfm25_stack_executor* executor, float* host, size_t rows);
+/* The f32 residual stream entering the final norm, [tokens, width]: what `layers` layers of the last step's tokens left
+ * (layers counts from 1).  A debugging and test aid: runs the next steps' layers only up to `layers` when set with
+ * lfm25_stack_executor_set_depth (0 = all). */
+int32_t lfm25_stack_executor_set_depth(lfm25_stack_executor* executor, uint32_t layers);
+int32_t lfm25_stack_executor_read_residual(lfm25_stack_executor* executor, float* host, size_t tokens);
+size_t lfm25_stack_executor_graph_kernels(const lfm25_stack_executor* executor);
+size_t lfm25_stack_executor_graph_captures(const lfm25_stack_executor* executor);
+
+/* ------------------------------------------------------------------------------------------
  * Host-side state: page allocator, block tables, decode scheduling, replica dispatch (no device work)
  * ------------------------------------------------------------------------------------------ */
 
@@ -878,6 +979,25 @@ typedef struct lfm25_engine_stats {
 } lfm25_engine_stats;
 int32_t lfm25_engine_create(lfm25_blaslt* blaslt, const lfm25_model* model, const lfm25_engine_config* config,
                             lfm25_engine** out);
+/* The same loop around a layer-stack model: request slots, pages, prefix checkpoints (the whole record of a slot is one
+ * checkpoint), planning and sampling are the engine's own; use_fp8 is ignored. */
+int32_t lfm25_engine_create_stack(lfm25_blaslt* blaslt, const lfm25_stack_model* model, const lfm25_engine_config* config,
+                                  lfm25_engine** out);
+/* Given tokens instead of sampled ones: feeds every entry's next tokens through the engine's step (its slots, pages,
+ * state and kernels) and returns the logits at `wanted` places (ascending indices into the entry's tokens) as f32
+ * [sum of num_wanted, vocab] in the order of the entries.  A request id seen for the first time takes a slot;
+ * lfm25_engine_end_forced gives back what it holds.  Long portions are cut into steps of the engine's size.  The
+ * engine must have no submitted requests. */
+typedef struct lfm25_forced_entry {
+    uint64_t request_id;
+    const uint32_t* tokens;
+    size_t num_tokens;
+    const uint32_t* wanted;
+    size_t num_wanted;
+} lfm25_forced_entry;
+int32_t lfm25_engine_forced_step(lfm25_engine* engine, const lfm25_forced_entry* entries, size_t num_entries,
+                                 float* logits, size_t logits_capacity);
+int32_t lfm25_engine_end_forced(lfm25_engine* engine, uint64_t request_id);
 void lfm25_engine_destroy(lfm25_engine* engine);
 int32_t lfm25_engine_calibrate(lfm25_engine* engine);
 const lfm25_cost_model* lfm25_engine_cost_model(const lfm25_engine* engine);

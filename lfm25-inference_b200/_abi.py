@@ -199,6 +199,40 @@ HybridAttentionLaunch = _launch_struct("HybridAttentionLaunch", [
     "position_ids", "segment_offsets", "output", "#num_tokens", "#num_pages", "#block_table_stride", "#num_segments",
     "#query_token_stride", "#kv_token_stride"])
 
+ACTIVATION_BF16, ACTIVATION_F32 = 0, 1
+MIXER_ATTENTION, MIXER_GENERAL_DELTA = 0, 1
+
+
+class StackLinear(ctypes.Structure):
+    _fields_ = [("weight", ctypes.c_void_p), ("n", ctypes.c_size_t), ("k", ctypes.c_size_t)]
+
+
+class StackLayer(ctypes.Structure):
+    _fields_ = ([("mixer", ctypes.c_uint32), ("mixer_norm", ctypes.c_void_p), ("ff_norm", ctypes.c_void_p),
+                 ("conv", ctypes.c_void_p), ("conv_offset", ctypes.c_size_t), ("projection", StackLinear),
+                 ("output", StackLinear), ("ff", ctypes.c_uint32), ("up", StackLinear), ("poly", ctypes.c_float * 4)]
+                + [(name, ctypes.c_uint32) for name in ("heads", "dim", "kv_heads", "vdim", "rot_dims", "chunk")]
+                + [("scale", ctypes.c_float)]
+                + [(name, ctypes.c_void_p) for name in ("inv_freq", "bias", "query_norm", "key_norm", "key_cache",
+                                                        "value_cache")]
+                + [("rank", ctypes.c_uint32)]
+                + [(name, ctypes.c_void_p) for name in ("decay_up", "decay_base", "removal_bias", "head_norm")]
+                + [("state_offset", ctypes.c_size_t)])
+
+
+class StackModel(ctypes.Structure):
+    _fields_ = [("num_layers", ctypes.c_uint32), ("layers", _P(StackLayer)), ("activation", ctypes.c_uint32),
+                ("conv_taps", ctypes.c_uint32), ("vocab", ctypes.c_size_t), ("width", ctypes.c_size_t),
+                ("norm_eps", ctypes.c_float), ("embedding", ctypes.c_void_p), ("final_norm", ctypes.c_void_p),
+                ("head", StackLinear), ("records", ctypes.c_void_p), ("record_bytes", ctypes.c_size_t),
+                ("num_request_slots", ctypes.c_size_t), ("num_pages", ctypes.c_size_t)]
+
+
+class ForcedEntry(ctypes.Structure):
+    _fields_ = [("request_id", ctypes.c_uint64), ("tokens", _P(ctypes.c_uint32)), ("num_tokens", ctypes.c_size_t),
+                ("wanted", _P(ctypes.c_uint32)), ("num_wanted", ctypes.c_size_t)]
+
+
 # name -> (restype, argtypes); every symbol that include/lfm25_b200.h declares
 PROTOTYPES = {
     "lfm25_last_error": (ctypes.c_char_p, []),
@@ -290,6 +324,23 @@ PROTOTYPES = {
     "lfm25_schedule_decode": (_size, [_P(ctypes.c_uint32), _P(ctypes.c_uint64), _P(ctypes.c_uint32), _size,
                                       ctypes.c_uint64, _P(ctypes.c_uint32), _P(_size)]),
     "lfm25_engine_create": (ctypes.c_int32, [ctypes.c_void_p, _P(Model), _P(EngineConfig), _P(ctypes.c_void_p)]),
+    "lfm25_stack_executor_create": (
+        ctypes.c_int32, [ctypes.c_void_p, _P(StackModel), _size, _size, _P(ctypes.c_void_p)]),
+    "lfm25_stack_executor_destroy": (None, [ctypes.c_void_p]),
+    "lfm25_stack_executor_forward": (ctypes.c_int32, [ctypes.c_void_p, _P(DecodeBatch), ctypes.c_uint32]),
+    "lfm25_stack_executor_step_graph": (ctypes.c_int32, [ctypes.c_void_p, _P(DecodeBatch), ctypes.c_uint32]),
+    "lfm25_stack_executor_forward_ragged": (ctypes.c_int32, [ctypes.c_void_p, _P(RaggedBatch), _size]),
+    "lfm25_stack_executor_download_sampled": (ctypes.c_int32, [ctypes.c_void_p, ctypes.c_void_p, _size]),
+    "lfm25_stack_executor_read_logits": (ctypes.c_int32, [ctypes.c_void_p, ctypes.c_void_p, _size]),
+    "lfm25_stack_executor_set_depth": (ctypes.c_int32, [ctypes.c_void_p, ctypes.c_uint32]),
+    "lfm25_stack_executor_read_residual": (ctypes.c_int32, [ctypes.c_void_p, ctypes.c_void_p, _size]),
+    "lfm25_stack_executor_graph_kernels": (_size, [ctypes.c_void_p]),
+    "lfm25_stack_executor_graph_captures": (_size, [ctypes.c_void_p]),
+    "lfm25_engine_create_stack": (
+        ctypes.c_int32, [ctypes.c_void_p, _P(StackModel), _P(EngineConfig), _P(ctypes.c_void_p)]),
+    "lfm25_engine_forced_step": (
+        ctypes.c_int32, [ctypes.c_void_p, _P(ForcedEntry), _size, ctypes.c_void_p, _size]),
+    "lfm25_engine_end_forced": (ctypes.c_int32, [ctypes.c_void_p, ctypes.c_uint64]),
     "lfm25_engine_destroy": (None, [ctypes.c_void_p]),
     "lfm25_engine_calibrate": (ctypes.c_int32, [ctypes.c_void_p]),
     "lfm25_engine_cost_model": (ctypes.c_void_p, [ctypes.c_void_p]),

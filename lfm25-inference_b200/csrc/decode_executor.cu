@@ -20,6 +20,7 @@
 #include "blaslt_handle.h"
 #include "kernels.h"
 #include "options.h"
+#include "step_graphs.h"
 
 namespace {
 
@@ -56,22 +57,7 @@ struct lfm25_decode_executor {
     // around every op of an eager step, summed per region
     bool profiling = false;
     std::vector<std::pair<int, std::pair<cudaEvent_t, cudaEvent_t>>> marks;
-    // captured steps: one per (batch size, attention split count, flags, buffers); a serving loop walks through many
-    // batch sizes, so the table is large and the least recently used entry is recycled
-    struct Captured {
-        size_t num_tokens = 0;
-        size_t splits = 0;
-        uint32_t use_fp8 = 0;
-        uint32_t advance = 0;
-        uint64_t signature = 0;   // of everything else the graph bakes in, see step_signature()
-        bool warmed = false;
-        cudaGraphExec_t exec = nullptr;
-        size_t kernel_nodes = 0;
-        uint64_t last_used = 0;
-    } captured[96];
-    uint64_t graph_clock = 0;
-    size_t last_graph_kernel_nodes = 0;   // of the graph launched most recently
-    size_t graph_captures = 0;            // captures made so far
+    lfm25::StepGraphs graphs;   // captured steps: one per (batch size, attention split count, flags, signature)
 };
 
 namespace {
@@ -101,32 +87,18 @@ struct RegionTimer {
 // signature hashes all of them (and the switches that change which kernels a step launches), so a caller who
 // regrows a block table, resizes the pool or swaps weights under the same array gets a fresh capture instead of a
 // replay of stale arguments.
-struct Fnv1a {
-    uint64_t state = 1469598103934665603ull;
-    void word(uint64_t value) { state = (state ^ value) * 1099511628211ull; }
-    template <typename Value>
-    void add(const Value& value) {   // values of up to 8 bytes are mixed in one step, longer ones word by word
-        static_assert(sizeof(Value) % 4 == 0, "hashed fields are 4-byte multiples");
-        const unsigned char* cursor = reinterpret_cast<const unsigned char*>(&value);
-        for (size_t offset = 0; offset < sizeof(Value); offset += 4) {
-            uint32_t part;
-            memcpy(&part, cursor + offset, 4);
-            word(part);
-        }
-    }
-    void linear(const lfm25_linear_weights& weights) {
-        add(weights.bf16);
-        add(weights.fp8.data);
-        add(weights.fp8.activation_quantize);
-        add(weights.fp8.activation_dequantize);
-        add(weights.fp8.weight_dequantize);
-        add(weights.n);
-        add(weights.k);
-    }
-};
+void hash_linear(lfm25::Fnv1a& hash, const lfm25_linear_weights& weights) {
+    hash.add(weights.bf16);
+    hash.add(weights.fp8.data);
+    hash.add(weights.fp8.activation_quantize);
+    hash.add(weights.fp8.activation_dequantize);
+    hash.add(weights.fp8.weight_dequantize);
+    hash.add(weights.n);
+    hash.add(weights.k);
+}
 
 uint64_t step_signature(const lfm25_decode_executor* self, const lfm25_model* model, const lfm25_decode_batch* batch) {
-    Fnv1a hash;
+    lfm25::Fnv1a hash;
     hash.add(batch->token_ids);
     hash.add(batch->positions);
     hash.add(batch->request_slots);
@@ -151,20 +123,20 @@ uint64_t step_signature(const lfm25_decode_executor* self, const lfm25_model* mo
         hash.add(layer.is_attention);
         hash.add(layer.operator_norm);
         hash.add(layer.ffn_norm);
-        hash.linear(layer.conv_input);
+        hash_linear(hash, layer.conv_input);
         hash.add(layer.conv_kernel);
-        hash.linear(layer.conv_output);
+        hash_linear(hash, layer.conv_output);
         hash.add(layer.conv_state);
-        hash.linear(layer.query);
-        hash.linear(layer.key);
-        hash.linear(layer.value);
-        hash.linear(layer.output);
+        hash_linear(hash, layer.query);
+        hash_linear(hash, layer.key);
+        hash_linear(hash, layer.value);
+        hash_linear(hash, layer.output);
         hash.add(layer.query_norm);
         hash.add(layer.key_norm);
         hash.add(layer.key_cache);
         hash.add(layer.value_cache);
-        hash.linear(layer.gate_up);
-        hash.linear(layer.down);
+        hash_linear(hash, layer.gate_up);
+        hash_linear(hash, layer.down);
     }
     for (int which = 0; which < lfm25::kOptCount; ++which) {
         if (which != lfm25::kOptEngineGraph) {
@@ -862,11 +834,6 @@ void lfm25_decode_executor_destroy(lfm25_decode_executor* self) {
     if (self == nullptr) {
         return;
     }
-    for (auto& entry : self->captured) {
-        if (entry.exec != nullptr) {
-            cudaGraphExecDestroy(entry.exec);
-        }
-    }
     cudaFree(self->allocation);
     delete self;
 }
@@ -971,83 +938,21 @@ int32_t lfm25_decode_executor_step_graph(lfm25_decode_executor* self, const lfm2
     // the split count of the attention launches is decided on the host from the longest context, so it is part of
     // what a captured step is valid for
     const size_t splits = lfm25_splitk_decode_splits(batch->num_tokens, batch->max_context_tokens, 16);
-    const uint64_t signature = step_signature(self, model, batch);
-    lfm25_decode_executor::Captured* entry = nullptr;
-    for (auto& candidate : self->captured) {
-        if (candidate.num_tokens == batch->num_tokens && candidate.splits == splits && candidate.use_fp8 == use_fp8 &&
-            candidate.advance == advance && candidate.signature == signature) {
-            entry = &candidate;
-            break;
-        }
-    }
-    if (entry == nullptr) {
-        // take a free entry, or recycle the least recently used one
-        for (auto& candidate : self->captured) {
-            if (candidate.num_tokens == 0) {
-                entry = &candidate;
-                break;
-            }
-            if (entry == nullptr || candidate.last_used < entry->last_used) {
-                entry = &candidate;
-            }
-        }
-        if (entry->exec != nullptr) {
-            cudaGraphExecDestroy(entry->exec);
-        }
-        *entry = lfm25_decode_executor::Captured();
-        entry->num_tokens = batch->num_tokens;
-        entry->splits = splits;
-        entry->use_fp8 = use_fp8;
-        entry->advance = advance;
-        entry->signature = signature;
-    }
-    entry->last_used = ++self->graph_clock;
-    cudaStream_t stream = self->blaslt->stream;
-    if (stream == nullptr || stream == cudaStreamLegacy) {
-        return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT,
-                                   "graph replay needs the BlasLt handle bound to a non-default stream");
-    }
-    if (!entry->warmed) {
-        // The first step of a bucket runs eagerly: cuBLASLt plans, function attributes and symbol lookups happen
-        // here, outside any capture.
-        entry->warmed = true;
-        return forward(self, model, batch, use_fp8 != 0, advance != 0);
-    }
-    if (entry->exec == nullptr) {
-        cudaError_t status = cudaStreamBeginCapture(stream, cudaStreamCaptureModeThreadLocal);
-        if (status != cudaSuccess) return cuda_failure(status, "stream capture could not begin");
+    lfm25::StepKey key;
+    key.num_tokens = batch->num_tokens;
+    key.splits = splits;
+    key.flags = (use_fp8 != 0 ? 1u : 0u) | (advance != 0 ? 2u : 0u);
+    key.signature = step_signature(self, model, batch);
+    return self->graphs.run(key, self->blaslt->stream, [&]() -> int32_t {
+        // region timing brackets eager steps only
+        cudaStreamCaptureStatus capturing = cudaStreamCaptureStatusNone;
+        cudaStreamIsCapturing(self->blaslt->stream, &capturing);
         const bool was_profiling = self->profiling;
-        self->profiling = false;
+        if (capturing != cudaStreamCaptureStatusNone) self->profiling = false;
         const int32_t rc = forward(self, model, batch, use_fp8 != 0, advance != 0);
         self->profiling = was_profiling;
-        cudaGraph_t graph = nullptr;
-        status = cudaStreamEndCapture(stream, &graph);
-        if (rc != LFM25_OK) {
-            if (graph != nullptr) cudaGraphDestroy(graph);
-            return rc;
-        }
-        if (status != cudaSuccess) return cuda_failure(status, "stream capture failed");
-        size_t node_count = 0;
-        if (cudaGraphGetNodes(graph, nullptr, &node_count) == cudaSuccess && node_count > 0) {
-            std::vector<cudaGraphNode_t> nodes(node_count);
-            if (cudaGraphGetNodes(graph, nodes.data(), &node_count) == cudaSuccess) {
-                for (size_t node = 0; node < node_count; ++node) {
-                    cudaGraphNodeType type;
-                    if (cudaGraphNodeGetType(nodes[node], &type) == cudaSuccess && type == cudaGraphNodeTypeKernel) {
-                        ++entry->kernel_nodes;
-                    }
-                }
-            }
-        }
-        status = cudaGraphInstantiate(&entry->exec, graph, 0);
-        cudaGraphDestroy(graph);
-        if (status != cudaSuccess) return cuda_failure(status, "graph instantiation failed");
-        ++self->graph_captures;
-    }
-    const cudaError_t status = cudaGraphLaunch(entry->exec, stream);
-    if (status != cudaSuccess) return cuda_failure(status, "graph launch failed");
-    self->last_graph_kernel_nodes = entry->kernel_nodes;
-    return LFM25_OK;
+        return rc;
+    });
 }
 
 int32_t lfm25_decode_executor_serve_step(lfm25_decode_executor* self, const lfm25_model* model,
@@ -1083,11 +988,11 @@ int32_t lfm25_decode_executor_serve_step(lfm25_decode_executor* self, const lfm2
 }
 
 size_t lfm25_decode_executor_graph_kernels(const lfm25_decode_executor* self) {
-    return self != nullptr ? self->last_graph_kernel_nodes : 0;
+    return self != nullptr ? self->graphs.last_kernel_nodes() : 0;
 }
 
 size_t lfm25_decode_executor_graph_captures(const lfm25_decode_executor* self) {
-    return self != nullptr ? self->graph_captures : 0;
+    return self != nullptr ? self->graphs.captures() : 0;
 }
 
 }  // extern "C"

@@ -17,17 +17,19 @@
 #include <cstdint>
 #include <cstring>
 #include <deque>
+#include <memory>
 #include <new>
 #include <vector>
 
 #include "../../include/lfm25_b200.h"
 #include "kernels.h"
 #include "options.h"
+#include "step_backend.h"
 
 namespace {
 
 constexpr size_t kPage = 16;
-constexpr size_t kHidden = 2048;
+constexpr uint32_t kPhaseForced = 3;   // a slot whose tokens come from lfm25_engine_forced_step
 
 struct Slot {
     uint32_t phase = LFM25_PHASE_FREE;
@@ -65,7 +67,7 @@ int32_t cuda_failure(cudaError_t status, const char* what) {
 
 struct lfm25_engine {
     lfm25_blaslt* blaslt = nullptr;
-    const lfm25_model* model = nullptr;
+    std::unique_ptr<lfm25::StepBackend> backend;
     lfm25_engine_config config{};
     size_t pages_per_slot = 0;
     size_t max_tokens = 0;
@@ -76,13 +78,12 @@ struct lfm25_engine {
     std::vector<size_t> grow_from;       // per work item of the step being built: tokens cached before ...
     std::vector<size_t> grow_to;         // ... and after it
     lfm25_cost_model* cost = nullptr;
-    lfm25_decode_executor* executor = nullptr;
-    std::vector<uint32_t> conv_layers;   // indices of the gated-convolution layers in the model
     std::vector<Slot> slots;
     std::vector<uint32_t> free_slots;
     std::deque<Pending> queue;
     // device metadata, one allocation: [token_ids | positions | request_slots | segment_offsets | segment_slots |
-    // output_rows] as u32, then physical slots (i64), then the block tables
+    // output_rows] as u32, then physical slots (i64), then the block tables.  Output rows come last, with room for one
+    // per token; only the used part is uploaded.
     uint32_t* d_meta = nullptr;
     int64_t* d_physical_slots = nullptr;
     uint32_t* d_tables = nullptr;
@@ -119,6 +120,8 @@ struct StepShape {
     std::vector<size_t> chunks;
     std::vector<uint32_t> segment_slots;
     std::vector<uint32_t> token_ids;
+    bool chosen_rows = false;             // output_rows are given instead of every segment's last token
+    std::vector<uint32_t> output_rows;
 };
 
 int32_t upload_tables(lfm25_engine* self, const uint32_t* table) {
@@ -149,7 +152,7 @@ int32_t enqueue_step(lfm25_engine* self, const StepShape& shape) {
             h_request_slots[tokens] = shape.segment_slots[segment];
             ++tokens;
         }
-        h_output_rows[segment] = static_cast<uint32_t>(tokens - 1);
+        if (!shape.chosen_rows) h_output_rows[segment] = static_cast<uint32_t>(tokens - 1);
         if (leading && shape.chunks[segment] == 1) {
             ++decode_segments;
             decode_context = std::max(decode_context, shape.prefixes[segment] + 1);
@@ -158,8 +161,11 @@ int32_t enqueue_step(lfm25_engine* self, const StepShape& shape) {
         }
     }
     h_offsets[segments] = static_cast<uint32_t>(tokens);
+    const size_t num_rows = shape.chosen_rows ? shape.output_rows.size() : segments;
+    if (shape.chosen_rows) std::copy(shape.output_rows.begin(), shape.output_rows.end(), h_output_rows);
     std::memcpy(meta, shape.token_ids.data(), tokens * sizeof(uint32_t));
-    cudaError_t status = cudaMemcpyAsync(self->d_meta, self->h_meta, self->meta_words * sizeof(uint32_t),
+    const size_t words = static_cast<size_t>(h_output_rows - meta) + num_rows;
+    cudaError_t status = cudaMemcpyAsync(self->d_meta, self->h_meta, words * sizeof(uint32_t),
                                          cudaMemcpyHostToDevice, self->stream());
     if (status != cudaSuccess) return cuda_failure(status, "step metadata upload failed");
     if (segments == tokens) {
@@ -174,11 +180,8 @@ int32_t enqueue_step(lfm25_engine* self, const StepShape& shape) {
         batch.num_tokens = tokens;
         batch.max_context_tokens = decode_context;
         // a pure decode step replays the captured step of its batch size (the first two steps of a size run eagerly
-        // and capture); the metadata was uploaded above, so the step does not advance it on the device
-        if (self->graph_decode) {
-            return lfm25_decode_executor_step_graph(self->executor, self->model, &batch, self->config.use_fp8, 0);
-        }
-        return lfm25_decode_executor_forward(self->executor, self->model, &batch, self->config.use_fp8, 0);
+        // and capture)
+        return self->backend->decode(batch, self->graph_decode);
     }
     lfm25_ragged_batch batch;
     batch.token_ids = self->token_ids();
@@ -195,16 +198,7 @@ int32_t enqueue_step(lfm25_engine* self, const StepShape& shape) {
     batch.num_segments = segments;
     batch.num_decode_segments = decode_segments;
     batch.max_decode_context_tokens = decode_context;
-    return lfm25_decode_executor_forward_ragged(self->executor, self->model, &batch, self->config.use_fp8);
-}
-
-int32_t clear_conv_state(lfm25_engine* self, size_t slot) {
-    for (uint32_t layer : self->conv_layers) {
-        char* state = static_cast<char*>(self->model->layers[layer].conv_state) + slot * kHidden * 2 * 2;
-        const cudaError_t status = cudaMemsetAsync(state, 0, kHidden * 2 * 2, self->stream());
-        if (status != cudaSuccess) return cuda_failure(status, "convolution state reset failed");
-    }
-    return LFM25_OK;
+    return self->backend->mixed(batch, num_rows);
 }
 
 // admit_request_radix (src/engine/serving/radix_owner.rs:549-708): a free slot, the longest reusable checkpointed
@@ -307,13 +301,9 @@ int32_t admit(lfm25_engine* self, uint64_t now_us, lfm25_engine_event* rejection
         if (matched > 0) {
             ENGINE_TRY(lfm25_kv_allocator_retain_pages(self->allocator, self->lookup_pages.data(), pages_found));
             std::copy(self->lookup_pages.begin(), self->lookup_pages.begin() + pages_found, row);
-            for (size_t index = 0; index < self->conv_layers.size(); ++index) {
-                ENGINE_TRY(lfm25_conv_checkpoints_restore_layer(
-                    self->checkpoints, self->stream(), checkpoint, index,
-                    self->model->layers[self->conv_layers[index]].conv_state, slot_index, self->config.max_slots));
-            }
+            ENGINE_TRY(self->backend->restore_state(self->checkpoints, checkpoint, slot_index));
         } else {
-            ENGINE_TRY(clear_conv_state(self, slot_index));
+            ENGINE_TRY(self->backend->clear_state(slot_index));
         }
         slot.phase = LFM25_PHASE_QUEUED_PREFILL;
         slot.request_id = request.request_id;
@@ -343,11 +333,7 @@ int32_t publish(lfm25_engine* self, uint32_t slot_index, const Slot& slot) {
     if (checkpoint < 0) {
         return LFM25_OK;
     }
-    for (size_t index = 0; index < self->conv_layers.size(); ++index) {
-        ENGINE_TRY(lfm25_conv_checkpoints_capture_layer(self->checkpoints, self->stream(), static_cast<uint32_t>(checkpoint),
-                                                        index, self->model->layers[self->conv_layers[index]].conv_state,
-                                                        slot_index, self->config.max_slots));
-    }
+    ENGINE_TRY(self->backend->capture_state(self->checkpoints, static_cast<uint32_t>(checkpoint), slot_index));
     const uint32_t* row = lfm25_block_tables_slot(self->tables, slot_index);
     const size_t pages = slot.prefilled / kPage;
     const int64_t created = lfm25_radix_cache_insert_checkpoint(self->radix, slot.tokens.data(), slot.prompt_len,
@@ -370,16 +356,9 @@ void release(lfm25_engine* self, uint32_t slot_index) {
     self->tables_dirty = true;
 }
 
-}  // namespace
-
-extern "C" {
-
-int32_t lfm25_engine_create(lfm25_blaslt* blaslt, const lfm25_model* model, const lfm25_engine_config* config,
-                            lfm25_engine** out) {
-    if (blaslt == nullptr || model == nullptr || config == nullptr || out == nullptr) {
-        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "engine received a null argument");
-    }
-    if (config->max_slots == 0 || config->max_slots > 256 || config->max_slots > model->num_request_slots) {
+int32_t create_engine(lfm25_blaslt* blaslt, std::unique_ptr<lfm25::StepBackend> backend,
+                      const lfm25_engine_config* config, lfm25_engine** out) {
+    if (config->max_slots == 0 || config->max_slots > 256 || config->max_slots > backend->num_request_slots()) {
         return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT,
                                    "engine needs 1..=256 request slots, at most the model's state rows");
     }
@@ -390,7 +369,7 @@ int32_t lfm25_engine_create(lfm25_blaslt* blaslt, const lfm25_model* model, cons
     lfm25_engine* self = new (std::nothrow) lfm25_engine();
     if (self == nullptr) return lfm25::report_error(LFM25_ERR_CUDA, "out of host memory");
     self->blaslt = blaslt;
-    self->model = model;
+    self->backend = std::move(backend);
     self->config = *config;
     self->pages_per_slot = (config->max_sequence_tokens + kPage - 1) / kPage;
     self->max_tokens = config->max_slots + config->max_prefill_tokens;
@@ -400,21 +379,15 @@ int32_t lfm25_engine_create(lfm25_blaslt* blaslt, const lfm25_model* model, cons
         self->graph_decode = lfm25::option(lfm25::kOptEngineGraph) != 0 && bound != nullptr &&
                              bound != cudaStreamLegacy;
     }
-    for (uint32_t layer = 0; layer < model->num_layers; ++layer) {
-        if (!model->layers[layer].is_attention) self->conv_layers.push_back(layer);
-    }
-    int32_t rc = lfm25_kv_allocator_create(model->num_pages, kPage, &self->allocator);
+    int32_t rc = lfm25_kv_allocator_create(self->backend->num_pages(), kPage, &self->allocator);
     if (rc == LFM25_OK) rc = lfm25_block_tables_create(config->max_slots, self->pages_per_slot, &self->tables);
     if (rc == LFM25_OK) rc = lfm25_radix_cache_create(kPage, std::max<size_t>(config->radix_pages, 1), &self->radix);
-    if (rc == LFM25_OK && !self->conv_layers.empty()) {
-        rc = lfm25_conv_checkpoints_create(self->conv_layers.size(), std::max<size_t>(config->checkpoint_capacity, 1),
-                                           kHidden, 2, &self->checkpoints);
-    }
     if (rc == LFM25_OK) {
-        rc = lfm25_decode_executor_create_ragged(blaslt, self->max_tokens, config->max_slots, &self->executor);
+        rc = self->backend->create_checkpoints(std::max<size_t>(config->checkpoint_capacity, 1), &self->checkpoints);
     }
+    if (rc == LFM25_OK) rc = self->backend->create_executor(self->max_tokens, config->max_slots);
     if (rc == LFM25_OK) {
-        self->meta_words = 3 * self->max_tokens + 3 * config->max_slots + 1;
+        self->meta_words = 4 * self->max_tokens + 2 * config->max_slots + 1;
         const size_t table_words = config->max_slots * self->pages_per_slot;
         cudaError_t status = cudaMalloc(reinterpret_cast<void**>(&self->d_meta), self->meta_words * sizeof(uint32_t));
         if (status == cudaSuccess) {
@@ -448,9 +421,29 @@ int32_t lfm25_engine_create(lfm25_blaslt* blaslt, const lfm25_model* model, cons
     return LFM25_OK;
 }
 
+}  // namespace
+
+extern "C" {
+
+int32_t lfm25_engine_create(lfm25_blaslt* blaslt, const lfm25_model* model, const lfm25_engine_config* config,
+                            lfm25_engine** out) {
+    if (blaslt == nullptr || model == nullptr || config == nullptr || out == nullptr) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "engine received a null argument");
+    }
+    return create_engine(blaslt, lfm25::lfm2_backend(blaslt, model, config->use_fp8, config->max_slots), config, out);
+}
+
+int32_t lfm25_engine_create_stack(lfm25_blaslt* blaslt, const lfm25_stack_model* model, const lfm25_engine_config* config,
+                                  lfm25_engine** out) {
+    if (blaslt == nullptr || model == nullptr || config == nullptr || out == nullptr) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "engine received a null argument");
+    }
+    return create_engine(blaslt, lfm25::stack_backend(blaslt, model), config, out);
+}
+
 void lfm25_engine_destroy(lfm25_engine* self) {
     if (self == nullptr) return;
-    lfm25_decode_executor_destroy(self->executor);
+    self->backend.reset();
     lfm25_conv_checkpoints_destroy(self->checkpoints);
     lfm25_radix_cache_destroy(self->radix);
     if (self->tables != nullptr) lfm25_block_tables_destroy(self->tables);
@@ -507,7 +500,7 @@ int32_t lfm25_engine_calibrate(lfm25_engine* self) {
         const size_t pages = (context + 1 + kPage - 1) / kPage;
         size_t previous = 0;
         for (size_t sequences : batches) {
-            if (sequences == previous || sequences * pages > self->model->num_pages) continue;
+            if (sequences == previous || sequences * pages > self->backend->num_pages()) continue;
             previous = sequences;
             std::fill(table.begin(), table.end(), 0xffffffffu);
             StepShape shape;
@@ -544,7 +537,7 @@ int32_t lfm25_engine_calibrate(lfm25_engine* self) {
         return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "engine limits leave no point to calibrate on");
     }
     for (size_t slot = 0; slot < self->config.max_slots; ++slot) {
-        ENGINE_TRY(clear_conv_state(self, slot));
+        ENGINE_TRY(self->backend->clear_state(slot));
     }
     self->tables_dirty = true;
     lfm25_cost_model_destroy(self->cost);
@@ -595,7 +588,7 @@ int32_t lfm25_engine_step(lfm25_engine* self, uint64_t now_us, lfm25_engine_even
     for (size_t index = 0; index < self->slots.size(); ++index) {
         const Slot& slot = self->slots[index];
         lfm25_request_view& view = self->views[index];
-        view.phase = slot.phase;
+        view.phase = slot.phase == kPhaseForced ? LFM25_PHASE_FREE : slot.phase;
         view.prompt_len = slot.prompt_len;
         view.prefilled = slot.prefilled;
         view.context_tokens = slot.tokens.size();
@@ -668,7 +661,7 @@ int32_t lfm25_engine_step(lfm25_engine* self, uint64_t now_us, lfm25_engine_even
     cudaEventRecord(self->start, self->stream());
     ENGINE_TRY(enqueue_step(self, shape));
     cudaEventRecord(self->stop, self->stream());
-    ENGINE_TRY(lfm25_decode_executor_download_sampled(self->executor, self->h_sampled, plan.work_count));
+    ENGINE_TRY(self->backend->download_sampled(self->h_sampled, plan.work_count));
     cudaError_t status = cudaStreamSynchronize(self->stream());
     if (status != cudaSuccess) return cuda_failure(status, "serving step failed");
     float elapsed = 0.0f;
@@ -717,6 +710,193 @@ int32_t lfm25_engine_step(lfm25_engine* self, uint64_t now_us, lfm25_engine_even
     }
     *num_events = produced;
     return LFM25_OK;
+}
+
+// Feeds given tokens.  Each pass takes the next portion of every entry (as much as one step holds, single tokens
+// first, as the planner orders a step) and runs it like any other step; a family that only yields a segment's last row
+// gets its portions cut behind every wanted token.
+int32_t lfm25_engine_forced_step(lfm25_engine* self, const lfm25_forced_entry* entries, size_t num_entries, float* logits,
+                                 size_t logits_capacity) {
+    if (self == nullptr || (entries == nullptr && num_entries > 0)) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "forced step received a null argument");
+    }
+    if (!self->queue.empty()) {
+        return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "forced steps need an engine without requests");
+    }
+    for (const Slot& slot : self->slots) {
+        if (slot.phase != LFM25_PHASE_FREE && slot.phase != kPhaseForced) {
+            return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "forced steps need an engine without requests");
+        }
+    }
+    const size_t vocab = self->backend->vocab();
+    struct Cursor {
+        const lfm25_forced_entry* entry;
+        uint32_t slot;
+        size_t done = 0;          // tokens fed
+        size_t answered = 0;      // wanted places answered
+        size_t first_row = 0;     // of its logits
+        size_t take = 0;          // of the current pass
+    };
+    std::vector<Cursor> cursors;
+    size_t total_rows = 0;
+    for (size_t index = 0; index < num_entries; ++index) {
+        const lfm25_forced_entry& entry = entries[index];
+        if (entry.num_tokens == 0 || entry.tokens == nullptr || (entry.num_wanted > 0 && entry.wanted == nullptr)) {
+            return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "forced entry brings no tokens");
+        }
+        for (size_t place = 0; place < entry.num_wanted; ++place) {
+            if (entry.wanted[place] >= entry.num_tokens || (place > 0 && entry.wanted[place] <= entry.wanted[place - 1])) {
+                return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "wanted places must ascend inside the entry");
+            }
+        }
+        for (size_t token = 0; token < entry.num_tokens; ++token) {
+            if (entry.tokens[token] >= vocab) {
+                return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "token id beyond the vocabulary");
+            }
+        }
+        for (size_t other = 0; other < index; ++other) {
+            if (entries[other].request_id == entry.request_id) {
+                return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "a request appears twice in a forced step");
+            }
+        }
+        total_rows += entry.num_wanted;
+    }
+    if (total_rows > 0 && (logits == nullptr || logits_capacity < total_rows * vocab)) {
+        return lfm25::report_error(LFM25_ERR_BUFFER_TOO_SMALL, "logits buffer too small for the wanted places");
+    }
+    size_t row = 0;
+    for (size_t index = 0; index < num_entries; ++index) {
+        Cursor cursor;
+        cursor.entry = &entries[index];
+        cursor.first_row = row;
+        row += entries[index].num_wanted;
+        bool found = false;
+        for (size_t slot = 0; slot < self->slots.size(); ++slot) {
+            if (self->slots[slot].phase == kPhaseForced && self->slots[slot].request_id == entries[index].request_id) {
+                cursor.slot = static_cast<uint32_t>(slot);
+                found = true;
+            }
+        }
+        if (!found) {
+            if (self->free_slots.empty()) {
+                return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "no free request slot for a forced request");
+            }
+            cursor.slot = self->free_slots.back();
+            uint32_t* table = lfm25_block_tables_slot(self->tables, cursor.slot);
+            std::fill(table, table + self->pages_per_slot, 0xffffffffu);
+            self->tables_dirty = true;
+            ENGINE_TRY(self->backend->clear_state(cursor.slot));
+            self->free_slots.pop_back();
+            self->slots[cursor.slot].phase = kPhaseForced;
+            self->slots[cursor.slot].request_id = entries[index].request_id;
+        }
+        if (self->slots[cursor.slot].cached_tokens + entries[index].num_tokens > self->pages_per_slot * kPage) {
+            return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "request exceeds fixed token capacity");
+        }
+        cursors.push_back(cursor);
+    }
+    const bool any_rows = self->backend->any_output_rows();
+    std::vector<float> step_logits;
+    for (;;) {
+        // portions of this pass
+        size_t budget = self->max_tokens;
+        size_t rows = self->backend->maximum_rows();
+        std::vector<Cursor*> order;
+        for (Cursor& cursor : cursors) {
+            const lfm25_forced_entry& entry = *cursor.entry;
+            size_t take = std::min(entry.num_tokens - cursor.done, budget);
+            if (take == 0 || rows == 0) continue;
+            size_t inside = 0;     // wanted places inside the portion
+            while (cursor.answered + inside < entry.num_wanted &&
+                   entry.wanted[cursor.answered + inside] < cursor.done + take) {
+                ++inside;
+            }
+            const size_t most = any_rows ? rows : 1;
+            if (inside > most || (!any_rows && inside == 1)) {
+                inside = std::min(inside, most);
+                take = entry.wanted[cursor.answered + inside - 1] + 1 - cursor.done;
+            }
+            cursor.take = take;
+            budget -= take;
+            rows -= any_rows ? inside : 1;
+            order.push_back(&cursor);
+        }
+        if (order.empty()) break;
+        std::stable_sort(order.begin(), order.end(),
+                         [](const Cursor* a, const Cursor* b) { return (a->take == 1) > (b->take == 1); });
+        StepShape shape;
+        self->grow_from.clear();
+        self->grow_to.clear();
+        shape.chosen_rows = any_rows;
+        size_t wanted_rows = 0;
+        std::vector<std::pair<size_t, size_t>> answers;      // (row of the step, row of the caller)
+        const bool single = std::all_of(order.begin(), order.end(), [](const Cursor* c) { return c->take == 1; });
+        for (Cursor* cursor : order) {
+            const lfm25_forced_entry& entry = *cursor->entry;
+            const Slot& slot = self->slots[cursor->slot];
+            const size_t base = shape.token_ids.size();
+            self->grow_from.push_back(slot.cached_tokens);
+            self->grow_to.push_back(slot.cached_tokens + cursor->take);
+            shape.prefixes.push_back(slot.cached_tokens);
+            shape.chunks.push_back(cursor->take);
+            shape.segment_slots.push_back(cursor->slot);
+            shape.token_ids.insert(shape.token_ids.end(), entry.tokens + cursor->done,
+                                   entry.tokens + cursor->done + cursor->take);
+            while (cursor->answered < entry.num_wanted &&
+                   entry.wanted[cursor->answered] < cursor->done + cursor->take) {
+                const size_t step_row = single || !any_rows ? shape.chunks.size() - 1 : wanted_rows;
+                answers.push_back({step_row, cursor->first_row + cursor->answered});
+                if (any_rows && !single) {
+                    shape.output_rows.push_back(
+                        static_cast<uint32_t>(base + entry.wanted[cursor->answered] - cursor->done));
+                }
+                ++wanted_rows;
+                ++cursor->answered;
+            }
+        }
+        if (single) shape.chosen_rows = false;
+        if (lfm25_kv_allocator_pages_short(self->allocator, self->grow_from.data(), self->grow_to.data(),
+                                           order.size()) != 0) {
+            return lfm25::report_error(LFM25_KV_PHYSICAL_PAGES_EXHAUSTED, "KV pages exhausted by forced requests");
+        }
+        for (size_t index = 0; index < order.size(); ++index) {
+            const int64_t grown = lfm25_kv_allocator_grow_sequence(
+                self->allocator, self->grow_from[index], self->grow_to[index],
+                lfm25_block_tables_slot(self->tables, order[index]->slot), self->pages_per_slot);
+            if (grown != 0) self->tables_dirty = true;
+            if (grown < 0) return lfm25::report_error(static_cast<int32_t>(grown), "KV pages exhausted by forced requests");
+            self->slots[order[index]->slot].cached_tokens = self->grow_to[index];
+        }
+        if (self->tables_dirty) {
+            ENGINE_TRY(upload_tables(self, lfm25_block_tables_data(self->tables)));
+            self->tables_dirty = false;
+        }
+        ENGINE_TRY(enqueue_step(self, shape));
+        const size_t step_rows = shape.chosen_rows ? shape.output_rows.size() : shape.chunks.size();
+        if (!answers.empty()) {
+            step_logits.resize(step_rows * vocab);
+            ENGINE_TRY(self->backend->read_logits(step_logits.data(), step_rows));
+            for (const auto& answer : answers) {
+                std::memcpy(logits + answer.second * vocab, step_logits.data() + answer.first * vocab,
+                            vocab * sizeof(float));
+            }
+        }
+        const cudaError_t status = cudaStreamSynchronize(self->stream());
+        if (status != cudaSuccess) return cuda_failure(status, "forced step failed");
+        for (Cursor* cursor : order) cursor->done += cursor->take;
+    }
+    return LFM25_OK;
+}
+
+int32_t lfm25_engine_end_forced(lfm25_engine* self, uint64_t request_id) {
+    if (self == nullptr) return lfm25::report_error(LFM25_ERR_NULL_POINTER, "engine is null");
+    for (size_t slot = 0; slot < self->slots.size(); ++slot) {
+        if (self->slots[slot].phase == kPhaseForced && self->slots[slot].request_id == request_id) {
+            release(self, static_cast<uint32_t>(slot));
+            return LFM25_OK;
+        }
+    }
+    return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "no such forced request");
 }
 
 size_t lfm25_engine_active(const lfm25_engine* self) {

@@ -1,0 +1,554 @@
+// Steps of a layer-stack model: the launches of one decode or mixed step on fixed-address scratch, and decode steps
+// replayed from CUDA graphs.
+//
+// Per layer:  residual sum + both norms + input convolution  ->  mixer projections (one GEMM)  ->  mixer
+//             feed-forward up projection  ->  PolyNorm                                          \ side by side in one
+//             [mixer output | activation] x [W_o | W_down]^T (one GEMM, f32 accumulation)       / buffer
+// The residual stream stays in f32 and ping-pongs between two buffers, because a tile of the first kernel also reads
+// rows of its neighbours.
+#include <stdio.h>
+
+#include <algorithm>
+#include <new>
+#include <vector>
+
+#include "../../include/lfm25_b200.h"
+#include "blaslt_handle.h"
+#include "kernels.h"
+#include "options.h"
+#include "stack_kernels.h"
+#include "step_graphs.h"
+
+using lfm25::Activation;
+
+struct lfm25_stack_executor {
+    lfm25_blaslt* blaslt;
+    const lfm25_stack_model* model;
+    Activation type;
+    size_t maximum_tokens;
+    size_t maximum_rows;
+    uint32_t depth;            // layers that run, num_layers unless a test asked for fewer
+    void* allocation;
+    float* residual[2];        // [T, width]
+    void* mixed;               // [T, width]: mixer input
+    void* normalized;          // [T, width]: feed-forward input
+    void* projected;           // [T, widest projection]
+    void* query;               // [T, widest heads * dim]
+    void* up;                  // [T, widest ff]
+    void* joined;              // [T, widest output.k]: mixer output | activation
+    void* update;              // [T, width]
+    void* head_input;          // [R, width]
+    void* logits;              // [R, head.n]
+    float* raw;                // [T, widest heads * dim] when a delta rule needs it
+    uint32_t* sampled;         // [R]
+    size_t last_tokens = 0;
+    const float* last_residual = nullptr;
+    std::vector<unsigned char> staging;
+    lfm25::StepGraphs graphs;
+};
+
+namespace {
+
+int32_t cuda_failure(cudaError_t status, const char* what) {
+    char message[200];
+    snprintf(message, sizeof message, "%s: %s", what, cudaGetErrorString(status));
+    return lfm25::report_error(LFM25_ERR_CUDA, message);
+}
+
+#define STACK_TRY(expression)              \
+    do {                                   \
+        const int32_t rc_ = (expression);  \
+        if (rc_ != LFM25_OK) return rc_;   \
+    } while (0)
+#define STACK_CUDA(expression, what)                                \
+    do {                                                            \
+        const cudaError_t status_ = (expression);                   \
+        if (status_ != cudaSuccess) return cuda_failure(status_, what); \
+    } while (0)
+
+size_t mixer_columns(const lfm25_stack_layer& layer) {
+    return static_cast<size_t>(layer.heads) * (layer.mixer == LFM25_MIXER_ATTENTION ? layer.vdim : layer.dim);
+}
+
+// Columns of the projection that the mixer reads (the matrix may have more rows, all zero).
+size_t projection_columns(const lfm25_stack_layer& layer) {
+    if (layer.mixer == LFM25_MIXER_ATTENTION) {
+        return (static_cast<size_t>(layer.heads) + layer.kv_heads) * layer.dim +
+               static_cast<size_t>(layer.kv_heads) * layer.vdim;
+    }
+    return 5 * static_cast<size_t>(layer.heads) * layer.dim + layer.rank;
+}
+
+const char* layer_fault(const lfm25_stack_model& model, const lfm25_stack_layer& layer) {
+    if (layer.mixer > LFM25_MIXER_GENERAL_DELTA) return "unknown mixer";
+    if (!layer.mixer_norm || !layer.conv || !layer.projection.weight || !layer.output.weight) return "missing weights";
+    if (layer.heads == 0 || layer.dim == 0) return "mixer without heads";
+    if (layer.projection.k != model.width || layer.projection.n < projection_columns(layer)) return "projection shape";
+    if (layer.output.n != model.width || layer.output.k < mixer_columns(layer) + layer.ff) return "output shape";
+    if (layer.ff > 0) {
+        if (!layer.ff_norm || !layer.up.weight) return "missing feed-forward weights";
+        if (layer.up.k != model.width || layer.up.n < layer.ff) return "up projection shape";
+    } else if (layer.output.k != mixer_columns(layer)) {
+        return "output shape";
+    }
+    const size_t bytes = lfm25::activation_bytes(static_cast<Activation>(model.activation));
+    if (layer.conv_offset % 16 != 0 || layer.conv_offset + (model.conv_taps - 1) * model.width * bytes > model.record_bytes)
+        return "convolution state outside the record";
+    if (layer.mixer == LFM25_MIXER_ATTENTION) {
+        if (layer.kv_heads == 0 || layer.heads % layer.kv_heads != 0 || layer.vdim == 0) return "attention heads";
+        if (layer.rot_dims % 2 != 0 || layer.rot_dims > layer.dim || (layer.rot_dims > 0 && !layer.inv_freq))
+            return "rotary dimensions";
+        if (!layer.query_norm || !layer.key_norm || !layer.key_cache || !layer.value_cache) return "attention tensors";
+    } else {
+        if (layer.dim > lfm25::kDeltaMaxDim) return "delta-rule head size beyond 256";
+        if (layer.rank == 0 || !layer.decay_up || !layer.decay_base || !layer.removal_bias || !layer.head_norm)
+            return "delta-rule tensors";
+        const size_t state = static_cast<size_t>(layer.heads) * layer.dim * layer.dim * sizeof(float);
+        if (layer.state_offset % 16 != 0 || layer.state_offset + state > model.record_bytes)
+            return "recurrent state outside the record";
+    }
+    return nullptr;
+}
+
+// y[m, n] = x[m, k] w[n, k]^T: tensor cores for bf16 shapes with 16-byte rows, plain f32 arithmetic otherwise.
+int32_t linear(lfm25_stack_executor* self, const lfm25_stack_linear& site, const void* x, void* y, size_t rows) {
+    if (self->type == Activation::kBf16 && site.k % 8 == 0 && site.n % 8 == 0) {
+        lfm25_slice x_slice = {const_cast<void*>(x), rows * site.k};
+        lfm25_slice w_slice = {const_cast<void*>(site.weight), site.n * site.k};
+        lfm25_slice y_slice = {y, rows * site.n};
+        return lfm25_blaslt_linear_bf16(self->blaslt, x_slice, w_slice, y_slice, rows, site.n, site.k);
+    }
+    STACK_CUDA(lfm25::launch_linear_simt(self->blaslt->stream, self->type, x, site.weight, y, rows, site.n, site.k),
+               "linear launch failed");
+    return LFM25_OK;
+}
+
+// One step as both batch kinds describe it.
+struct Step {
+    uint32_t* token_ids;
+    uint32_t* positions;
+    const uint32_t* request_slots;
+    int64_t* physical_slots;
+    const uint32_t* block_tables;
+    size_t block_table_stride, block_table_rows;
+    lfm25::StackSegments segments;
+    const uint32_t* output_rows;   // nullptr: every token, in order
+    size_t num_outputs;
+    size_t max_context;
+    bool advance;
+};
+
+int32_t enqueue(lfm25_stack_executor* self, const Step& step) {
+    const lfm25_stack_model& model = *self->model;
+    cudaStream_t stream = self->blaslt->stream;
+    const size_t tokens = step.segments.num_tokens;
+    STACK_CUDA(lfm25::launch_decode_metadata(stream, step.token_ids, step.positions, step.request_slots,
+                                             step.block_tables, self->sampled, step.physical_slots, tokens,
+                                             step.block_table_stride, step.block_table_rows, model.num_pages,
+                                             step.advance),
+               "step metadata launch failed");
+    int current = 0;
+    for (uint32_t index = 0; index < self->depth; ++index) {
+        const lfm25_stack_layer& layer = model.layers[index];
+        lfm25::ResidualNormConvLaunch head;
+        head.type = self->type;
+        head.segments = step.segments;
+        head.residual = self->residual[current];
+        head.update = index == 0 ? nullptr : self->update;
+        head.token_ids = step.token_ids;
+        head.embedding = index == 0 ? model.embedding : nullptr;
+        head.vocab = model.vocab;
+        head.mixer_norm = layer.mixer_norm;
+        head.ff_norm = layer.ff > 0 ? layer.ff_norm : nullptr;
+        head.conv = layer.conv;
+        head.taps = model.conv_taps;
+        head.record = {model.records, model.record_bytes, layer.conv_offset};
+        head.residual_out = self->residual[1 - current];
+        head.mixed_out = self->mixed;
+        head.ff_out = self->normalized;
+        head.width = model.width;
+        head.eps = model.norm_eps;
+        STACK_CUDA(lfm25::launch_residual_norm_conv(stream, head), "residual norm convolution launch failed");
+        current = 1 - current;
+
+        STACK_TRY(linear(self, layer.projection, self->mixed, self->projected, tokens));
+        if (layer.mixer == LFM25_MIXER_ATTENTION) {
+            const lfm25::StackAttentionShape shape = {layer.heads, layer.kv_heads, layer.dim,  layer.vdim,
+                                                      layer.rot_dims, layer.chunk, layer.scale};
+            lfm25::ProjectionNormRopeLaunch post;
+            post.type = self->type;
+            post.shape = shape;
+            post.projected = self->projected;
+            post.pitch = layer.projection.n;
+            post.bias = layer.bias;
+            post.query_norm = layer.query_norm;
+            post.key_norm = layer.key_norm;
+            post.inv_freq = layer.inv_freq;
+            post.positions = step.positions;
+            post.physical_slots = step.physical_slots;
+            post.query_out = self->query;
+            post.key_cache = layer.key_cache;
+            post.value_cache = layer.value_cache;
+            post.num_tokens = tokens;
+            post.num_pages = model.num_pages;
+            post.eps = model.norm_eps;
+            STACK_CUDA(lfm25::launch_projection_norm_rope(stream, post), "projection norm rope launch failed");
+            lfm25::StackAttentionLaunch attention;
+            attention.type = self->type;
+            attention.shape = shape;
+            attention.query = self->query;
+            attention.key_cache = layer.key_cache;
+            attention.value_cache = layer.value_cache;
+            attention.block_tables = step.block_tables;
+            attention.block_table_stride = step.block_table_stride;
+            attention.block_table_rows = step.block_table_rows;
+            attention.num_pages = model.num_pages;
+            attention.request_slots = step.request_slots;
+            attention.positions = step.positions;
+            attention.segments = step.segments;
+            attention.max_context = step.max_context;
+            attention.out = self->joined;
+            attention.out_pitch = layer.output.k;
+            STACK_CUDA(lfm25::launch_stack_attention(stream, attention), "attention launch failed");
+        } else {
+            lfm25::DeltaRuleLaunch delta;
+            delta.type = self->type;
+            delta.segments = step.segments;
+            delta.heads = layer.heads;
+            delta.dim = layer.dim;
+            delta.rank = layer.rank;
+            delta.projected = self->projected;
+            delta.pitch = layer.projection.n;
+            delta.decay_up = layer.decay_up;
+            delta.decay_base = layer.decay_base;
+            delta.removal_bias = layer.removal_bias;
+            delta.norm = layer.head_norm;
+            delta.record = {model.records, model.record_bytes, layer.state_offset};
+            delta.raw = self->raw;
+            delta.out = self->joined;
+            delta.out_pitch = layer.output.k;
+            delta.eps = model.norm_eps;
+            STACK_CUDA(lfm25::launch_delta_rule(stream, delta), "delta rule launch failed");
+        }
+        if (layer.ff > 0) {
+            STACK_TRY(linear(self, layer.up, self->normalized, self->up, tokens));
+            const size_t column = mixer_columns(layer);
+            unsigned char* activation =
+                static_cast<unsigned char*>(self->joined) + column * lfm25::activation_bytes(self->type);
+            STACK_CUDA(lfm25::launch_poly_norm(stream, self->type, self->up, layer.up.n, activation, layer.output.k,
+                                               tokens, layer.ff, layer.output.k - column - layer.ff, layer.poly,
+                                               model.norm_eps),
+                       "polynomial activation launch failed");
+        }
+        STACK_TRY(linear(self, layer.output, self->joined, self->update, tokens));
+    }
+    self->last_residual = self->residual[current];
+    self->last_tokens = tokens;
+    if (step.num_outputs == 0) {
+        return LFM25_OK;
+    }
+    STACK_CUDA(lfm25::launch_residual_norm_rows(stream, self->type, self->residual[current], self->update,
+                                                model.final_norm, step.output_rows, self->head_input, step.num_outputs,
+                                                tokens, model.width, model.norm_eps),
+               "final norm launch failed");
+    STACK_TRY(linear(self, model.head, self->head_input, self->logits, step.num_outputs));
+    STACK_CUDA(lfm25::launch_argmax_rows(stream, self->type, self->logits, model.head.n, self->sampled, step.num_outputs,
+                                         model.vocab),
+               "argmax launch failed");
+    return LFM25_OK;
+}
+
+uint64_t signature(const lfm25_stack_executor* self, const lfm25_decode_batch* batch) {
+    lfm25::Fnv1a hash;
+    hash.add(batch->token_ids);
+    hash.add(batch->positions);
+    hash.add(batch->request_slots);
+    hash.add(batch->physical_slots);
+    hash.add(batch->block_tables);
+    hash.add(batch->block_table_stride);
+    hash.add(batch->block_table_rows);
+    hash.add(self->depth);
+    const lfm25_stack_model& model = *self->model;
+    hash.add(model.layers);
+    hash.add(model.embedding);
+    hash.add(model.final_norm);
+    hash.add(model.head.weight);
+    hash.add(model.head.n);
+    hash.add(model.vocab);
+    hash.add(model.width);
+    hash.add(model.norm_eps);
+    hash.add(model.records);
+    hash.add(model.record_bytes);
+    hash.add(model.num_request_slots);
+    hash.add(model.num_pages);
+    for (uint32_t index = 0; index < model.num_layers; ++index) {
+        const lfm25_stack_layer& layer = model.layers[index];
+        const void* pointers[] = {layer.mixer_norm, layer.ff_norm, layer.conv, layer.projection.weight, layer.output.weight,
+                                  layer.up.weight, layer.inv_freq, layer.bias, layer.query_norm, layer.key_norm,
+                                  layer.key_cache, layer.value_cache, layer.decay_up, layer.decay_base,
+                                  layer.removal_bias, layer.head_norm};
+        for (const void* pointer : pointers) hash.add(pointer);
+        const size_t sizes[] = {layer.conv_offset, layer.projection.n, layer.output.k, layer.up.n, layer.state_offset};
+        for (size_t size : sizes) hash.add(size);
+        const uint32_t words[] = {layer.mixer, layer.ff, layer.heads, layer.dim, layer.kv_heads, layer.vdim,
+                                  layer.rot_dims, layer.chunk, layer.rank};
+        for (uint32_t word : words) hash.add(word);
+        for (float value : layer.poly) hash.add(value);
+        hash.add(layer.scale);
+    }
+    for (int which = 0; which < lfm25::kOptCount; ++which) {
+        if (which != lfm25::kOptEngineGraph) hash.add(lfm25::option(static_cast<lfm25::Option>(which)));
+    }
+    hash.add(self->blaslt->tuning_kernel);
+    hash.add(self->blaslt->tuning);
+    hash.add(self->blaslt->stream);
+    return hash.state;
+}
+
+int32_t decode_step(const lfm25_stack_executor* self, const lfm25_decode_batch* batch, bool advance, Step* step) {
+    if (self == nullptr || batch == nullptr) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "stack executor received a null argument");
+    }
+    if (batch->num_tokens == 0 || batch->num_tokens > self->maximum_tokens || batch->num_tokens > self->maximum_rows) {
+        return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "stack executor token count exceeds workspace");
+    }
+    if (!batch->token_ids || !batch->positions || !batch->request_slots || !batch->physical_slots ||
+        !batch->block_tables || batch->block_table_stride == 0 || batch->block_table_rows == 0) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "decode batch metadata is incomplete");
+    }
+    step->token_ids = batch->token_ids;
+    step->positions = batch->positions;
+    step->request_slots = batch->request_slots;
+    step->physical_slots = batch->physical_slots;
+    step->block_tables = batch->block_tables;
+    step->block_table_stride = batch->block_table_stride;
+    step->block_table_rows = batch->block_table_rows;
+    step->segments = {nullptr, batch->request_slots, batch->num_tokens, batch->num_tokens, self->model->num_request_slots};
+    step->output_rows = nullptr;
+    step->num_outputs = batch->num_tokens;
+    step->max_context = batch->max_context_tokens;
+    step->advance = advance;
+    return LFM25_OK;
+}
+
+}  // namespace
+
+extern "C" {
+
+int32_t lfm25_stack_executor_create(lfm25_blaslt* blaslt, const lfm25_stack_model* model, size_t maximum_tokens,
+                                    size_t maximum_rows, lfm25_stack_executor** out) {
+    if (blaslt == nullptr || model == nullptr || out == nullptr) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "stack executor received a null argument");
+    }
+    if (maximum_rows == 0 || maximum_tokens < maximum_rows || maximum_tokens > 65536) {
+        return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT,
+                                   "stack executor needs 1..=65536 tokens per step and at most as many output rows");
+    }
+    if (model->num_layers == 0 || model->layers == nullptr || model->embedding == nullptr ||
+        model->final_norm == nullptr || model->head.weight == nullptr || model->records == nullptr) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "stack model is incomplete");
+    }
+    if (model->activation > LFM25_ACTIVATION_F32 || model->conv_taps == 0 || model->width == 0 || model->vocab == 0 ||
+        model->head.n < model->vocab || model->head.k != model->width || model->record_bytes % 256 != 0 ||
+        model->num_request_slots == 0 || model->num_pages == 0) {
+        return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "stack model sizes are inconsistent");
+    }
+    size_t projection = 0, query = 0, up = 0, joined = 0, raw = 0;
+    for (uint32_t index = 0; index < model->num_layers; ++index) {
+        const lfm25_stack_layer& layer = model->layers[index];
+        const char* fault = layer_fault(*model, layer);
+        if (fault != nullptr) {
+            char message[120];
+            snprintf(message, sizeof message, "layer %u: %s", index, fault);
+            return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, message);
+        }
+        projection = std::max(projection, layer.projection.n);
+        joined = std::max(joined, layer.output.k);
+        up = std::max(up, layer.ff > 0 ? layer.up.n : 0);
+        const size_t width = static_cast<size_t>(layer.heads) * layer.dim;
+        if (layer.mixer == LFM25_MIXER_ATTENTION) query = std::max(query, width);
+        if (layer.mixer == LFM25_MIXER_GENERAL_DELTA && lfm25::delta_rule_needs_scratch(layer.dim))
+            raw = std::max(raw, width);
+    }
+    lfm25_stack_executor* self = new (std::nothrow) lfm25_stack_executor();
+    if (self == nullptr) return lfm25::report_error(LFM25_ERR_CUDA, "out of host memory");
+    self->blaslt = blaslt;
+    self->model = model;
+    self->type = static_cast<Activation>(model->activation);
+    self->maximum_tokens = maximum_tokens;
+    self->maximum_rows = maximum_rows;
+    self->depth = model->num_layers;
+    const size_t t = maximum_tokens, r = maximum_rows, bytes = lfm25::activation_bytes(self->type);
+    void** fields[] = {reinterpret_cast<void**>(&self->residual[0]), reinterpret_cast<void**>(&self->residual[1]),
+                       &self->mixed, &self->normalized, &self->projected, &self->query, &self->up, &self->joined,
+                       &self->update, &self->head_input, &self->logits, reinterpret_cast<void**>(&self->raw),
+                       reinterpret_cast<void**>(&self->sampled)};
+    const size_t sizes[] = {t * model->width * 4, t * model->width * 4, t * model->width * bytes,
+                            t * model->width * bytes, t * projection * bytes, t * query * bytes, t * up * bytes,
+                            t * joined * bytes, t * model->width * bytes, r * model->width * bytes,
+                            r * model->head.n * bytes, t * raw * 4, r * 4};
+    size_t total = 0;
+    for (size_t size : sizes) total += (size + 255) & ~static_cast<size_t>(255);
+    cudaError_t status = cudaMalloc(&self->allocation, total);
+    if (status == cudaSuccess) status = cudaMemsetAsync(self->allocation, 0, total, blaslt->stream);
+    if (status != cudaSuccess) {
+        cudaFree(self->allocation);
+        delete self;
+        return cuda_failure(status, "failed to allocate stack scratch");
+    }
+    unsigned char* cursor = static_cast<unsigned char*>(self->allocation);
+    for (size_t index = 0; index < sizeof sizes / sizeof sizes[0]; ++index) {
+        *fields[index] = sizes[index] > 0 ? cursor : nullptr;
+        cursor += (sizes[index] + 255) & ~static_cast<size_t>(255);
+    }
+    *out = self;
+    return LFM25_OK;
+}
+
+void lfm25_stack_executor_destroy(lfm25_stack_executor* self) {
+    if (self == nullptr) return;
+    cudaFree(self->allocation);
+    delete self;
+}
+
+int32_t lfm25_stack_executor_forward(lfm25_stack_executor* self, const lfm25_decode_batch* batch, uint32_t advance) {
+    Step step;
+    STACK_TRY(decode_step(self, batch, advance != 0, &step));
+    return enqueue(self, step);
+}
+
+int32_t lfm25_stack_executor_step_graph(lfm25_stack_executor* self, const lfm25_decode_batch* batch, uint32_t advance) {
+    Step step;
+    STACK_TRY(decode_step(self, batch, advance != 0, &step));
+    lfm25::StepKey key;
+    key.num_tokens = batch->num_tokens;
+    key.splits = 0;
+    key.flags = advance != 0 ? 1u : 0u;
+    key.signature = signature(self, batch);
+    return self->graphs.run(key, self->blaslt->stream, [&]() -> int32_t { return enqueue(self, step); });
+}
+
+int32_t lfm25_stack_executor_forward_ragged(lfm25_stack_executor* self, const lfm25_ragged_batch* batch,
+                                            size_t num_output_rows) {
+    if (self == nullptr || batch == nullptr) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "stack executor received a null argument");
+    }
+    if (batch->num_tokens == 0 || batch->num_tokens > self->maximum_tokens || num_output_rows > self->maximum_rows ||
+        batch->num_segments == 0 || batch->num_segments > batch->num_tokens) {
+        return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "ragged step exceeds the stack executor's workspace");
+    }
+    if (!batch->token_ids || !batch->positions || !batch->request_slots || !batch->physical_slots ||
+        !batch->segment_offsets || !batch->segment_slots || (num_output_rows > 0 && !batch->output_rows) ||
+        !batch->block_tables || batch->block_table_stride == 0 || batch->block_table_rows == 0) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "ragged batch metadata is incomplete");
+    }
+    Step step;
+    step.token_ids = const_cast<uint32_t*>(batch->token_ids);
+    step.positions = const_cast<uint32_t*>(batch->positions);
+    step.request_slots = batch->request_slots;
+    step.physical_slots = batch->physical_slots;
+    step.block_tables = batch->block_tables;
+    step.block_table_stride = batch->block_table_stride;
+    step.block_table_rows = batch->block_table_rows;
+    step.segments = {batch->segment_offsets, batch->segment_slots, batch->num_segments, batch->num_tokens,
+                     self->model->num_request_slots};
+    step.output_rows = batch->output_rows;
+    step.num_outputs = num_output_rows;
+    step.max_context = batch->max_decode_context_tokens;
+    step.advance = false;
+    return enqueue(self, step);
+}
+
+int32_t lfm25_stack_executor_download_sampled(lfm25_stack_executor* self, uint32_t* host, size_t count) {
+    if (self == nullptr || host == nullptr) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "sampled download received a null argument");
+    }
+    if (count > self->maximum_rows) {
+        return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "sampled download exceeds the executor's capacity");
+    }
+    STACK_CUDA(cudaMemcpyAsync(host, self->sampled, count * sizeof(uint32_t), cudaMemcpyDeviceToHost,
+                               self->blaslt->stream),
+               "sampled download failed");
+    return LFM25_OK;
+}
+
+int32_t lfm25_stack_executor_read_logits(lfm25_stack_executor* self, float* host, size_t rows) {
+    if (self == nullptr || host == nullptr) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "logits read received a null argument");
+    }
+    if (rows > self->maximum_rows) {
+        return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "logits read exceeds the executor's capacity");
+    }
+    const lfm25_stack_model& model = *self->model;
+    const size_t bytes = lfm25::activation_bytes(self->type);
+    cudaStream_t stream = self->blaslt->stream;
+    if (self->type == Activation::kF32) {
+        STACK_CUDA(cudaMemcpy2DAsync(host, model.vocab * 4, self->logits, model.head.n * 4, model.vocab * 4, rows,
+                                     cudaMemcpyDeviceToHost, stream),
+                   "logits download failed");
+        STACK_CUDA(cudaStreamSynchronize(stream), "logits download failed");
+        return LFM25_OK;
+    }
+    self->staging.resize(rows * model.vocab * bytes);
+    STACK_CUDA(cudaMemcpy2DAsync(self->staging.data(), model.vocab * bytes, self->logits, model.head.n * bytes,
+                                 model.vocab * bytes, rows, cudaMemcpyDeviceToHost, stream),
+               "logits download failed");
+    STACK_CUDA(cudaStreamSynchronize(stream), "logits download failed");
+    for (size_t index = 0; index < rows * model.vocab; ++index) {
+        uint16_t half;
+        memcpy(&half, self->staging.data() + index * 2, 2);
+        const uint32_t word = static_cast<uint32_t>(half) << 16;
+        memcpy(host + index, &word, 4);
+    }
+    return LFM25_OK;
+}
+
+int32_t lfm25_stack_executor_set_depth(lfm25_stack_executor* self, uint32_t layers) {
+    if (self == nullptr) return lfm25::report_error(LFM25_ERR_NULL_POINTER, "stack executor is null");
+    if (layers > self->model->num_layers) {
+        return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "depth exceeds the model's layers");
+    }
+    self->depth = layers == 0 ? self->model->num_layers : layers;
+    return LFM25_OK;
+}
+
+int32_t lfm25_stack_executor_read_residual(lfm25_stack_executor* self, float* host, size_t tokens) {
+    if (self == nullptr || host == nullptr) {
+        return lfm25::report_error(LFM25_ERR_NULL_POINTER, "residual read received a null argument");
+    }
+    if (tokens == 0 || tokens > self->last_tokens) {
+        return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "residual read exceeds the last step");
+    }
+    const size_t count = tokens * self->model->width;
+    const size_t bytes = lfm25::activation_bytes(self->type);
+    cudaStream_t stream = self->blaslt->stream;
+    self->staging.resize(count * bytes);
+    STACK_CUDA(cudaMemcpyAsync(host, self->last_residual, count * 4, cudaMemcpyDeviceToHost, stream),
+               "residual download failed");
+    STACK_CUDA(cudaMemcpyAsync(self->staging.data(), self->update, count * bytes, cudaMemcpyDeviceToHost, stream),
+               "residual download failed");
+    STACK_CUDA(cudaStreamSynchronize(stream), "residual download failed");
+    for (size_t index = 0; index < count; ++index) {
+        float add;
+        if (self->type == Activation::kF32) {
+            memcpy(&add, self->staging.data() + index * 4, 4);
+        } else {
+            uint16_t half;
+            memcpy(&half, self->staging.data() + index * 2, 2);
+            const uint32_t word = static_cast<uint32_t>(half) << 16;
+            memcpy(&add, &word, 4);
+        }
+        host[index] += add;
+    }
+    return LFM25_OK;
+}
+
+size_t lfm25_stack_executor_graph_kernels(const lfm25_stack_executor* self) {
+    return self != nullptr ? self->graphs.last_kernel_nodes() : 0;
+}
+
+size_t lfm25_stack_executor_graph_captures(const lfm25_stack_executor* self) {
+    return self != nullptr ? self->graphs.captures() : 0;
+}
+
+}  // extern "C"

@@ -88,6 +88,7 @@ class RandomModel:
         that concatenates them would leave them), which lets the executor run the three projections as one GEMM;
         False keeps three separate allocations (three GEMMs, the reference's layout)."""
         self.device = device
+        self.vocab = VOCAB
         self.num_pages = num_pages
         self.num_request_slots = num_request_slots
         generator = torch.Generator(device=device).manual_seed(seed)
@@ -171,6 +172,9 @@ class RandomModel:
         head = self.lm_head.struct().fp8
         self.struct = _abi.Model(NUM_LAYERS, array, self.embedding.data_ptr(), head, self.final_norm.data_ptr(),
                                  self.inv_freq.data_ptr(), NORM_EPS, self.num_pages, self.num_request_slots)
+
+    def create_engine(self, blaslt_handle, config: _abi.EngineConfig, out) -> int:
+        return library().lfm25_engine_create(blaslt_handle, self.struct, ctypes.byref(config), out)
 
     def fill_caches(self, seed: int) -> None:
         """KV pools and convolution states ~ N(0,1): stricter than the reference's own benchmark, which leaves the

@@ -4,8 +4,8 @@ The GPU-owner loop itself -- request slots, admission with prefix reuse, step pl
 mixed prefill / decode steps, token bookkeeping -- is native (`csrc/serving_engine.cu`, `lfm25_engine_*`, the
 counterpart of the reference's src/engine/serving/radix_owner.rs).  This module is the thin front of it that the tests
 and the benchmark use: it feeds requests in arrival order, calls `lfm25_engine_step` until the trace is drained, and
-turns the token events into per-request latency records.  Sampling is greedy; the model is whatever `RandomModel`
-the caller built.
+turns the token events into per-request latency records.  Sampling is greedy; the model is whatever family the caller
+built (`registry.load_model`): it only has to offer `create_engine`.
 """
 from __future__ import annotations
 
@@ -17,7 +17,6 @@ from dataclasses import dataclass
 import numpy as np
 
 from . import _abi, ops
-from . import model as lfm_model
 from ._abi import check, library
 
 
@@ -36,7 +35,7 @@ class Request:
 class ServingEngine:
     """One engine per GPU, driven from one host thread (the reference's GPU-owner thread)."""
 
-    def __init__(self, model: lfm_model.RandomModel, device, max_slots: int = 64, max_sequence_tokens: int = 8704,
+    def __init__(self, model, device, max_slots: int = 64, max_sequence_tokens: int = 8704,
                  max_prefill_tokens: int = 512, radix_pages: int = 4096, checkpoint_capacity: int = 64,
                  use_fp8: bool = True, ttft_slo_us: int = 400_000, tpot_slo_us: int = 50_000,
                  step_budget_ms: float = 40.0, admission_control: bool = False, interactive_prompt_limit: int = 0):
@@ -50,8 +49,7 @@ class ServingEngine:
                                    checkpoint_capacity, int(use_fp8), ttft_slo_us, tpot_slo_us, step_budget_ms,
                                    int(admission_control), interactive_prompt_limit)
         self._handle = ctypes.c_void_p()
-        check(library().lfm25_engine_create(self.blaslt._handle, model.struct, ctypes.byref(config),
-                                            ctypes.byref(self._handle)))
+        check(model.create_engine(self.blaslt._handle, config, ctypes.byref(self._handle)))
         self._capacity = 2 * max_slots
         self._events = (_abi.EngineEvent * self._capacity)()
         self._count = ctypes.c_size_t(0)
@@ -86,6 +84,23 @@ class ServingEngine:
                    int(e.rejected)) for e in self._events[:self._count.value]]
         return events, float(self._gpu_ms.value)
 
+    def forced_step(self, entries, vocab: int) -> np.ndarray:
+        """Feeds given tokens: `entries` is a list of (request_id, tokens, wanted places in ascending order).  Returns the
+        wanted logits as f32 [total wanted, vocab] in the order of the entries."""
+        total = sum(len(wanted) for _, _, wanted in entries)
+        logits = np.empty((total, vocab), dtype=np.float32)
+        held = [(request_id, np.ascontiguousarray(tokens, dtype=np.uint32),
+                 np.ascontiguousarray(wanted, dtype=np.uint32)) for request_id, tokens, wanted in entries]
+        pointer = ctypes.POINTER(ctypes.c_uint32)
+        array = (_abi.ForcedEntry * len(held))(*[
+            _abi.ForcedEntry(request_id, tokens.ctypes.data_as(pointer), tokens.size, wanted.ctypes.data_as(pointer),
+                             wanted.size) for request_id, tokens, wanted in held])
+        check(library().lfm25_engine_forced_step(self._handle, array, len(held), logits.ctypes.data, logits.size))
+        return logits
+
+    def end_forced(self, request_id: int) -> None:
+        check(library().lfm25_engine_end_forced(self._handle, request_id))
+
     def active(self) -> int:
         return int(library().lfm25_engine_active(self._handle))
 
@@ -106,6 +121,14 @@ class ServingEngine:
             library().lfm25_engine_destroy(self._handle)
             self._handle = None
         self.blaslt.close()
+
+
+def generate(engine: ServingEngine, prompts, max_new_tokens: int) -> list[list[int]]:
+    """Greedy continuations of `prompts` (token ids), batched by the engine's scheduler."""
+    requests = [Request(index, np.asarray(prompt, dtype=np.uint32), max_new_tokens, 0)
+                for index, prompt in enumerate(prompts)]
+    records = run_trace(engine, requests)["requests"]
+    return [record["tokens"] for record in sorted(records, key=lambda record: record["request_id"])]
 
 
 def run_trace(engine: ServingEngine, requests: list[Request]) -> dict:
