@@ -1,7 +1,7 @@
 """Benchmark of the decode hot path.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
-                    [--workload step|attention|gemm|prefill|serving]
+                    [--workload step|attention|gemm|prefill|serving|stack]
 
 Default workload `step` (one "step" = one decode step of the whole model): the LFM2.5-1.2B architecture with
 random-init weights under continuous batching -- 16 layers (6 GQA attention, 10 gated short-conv), hidden 2048,
@@ -22,6 +22,9 @@ LM head 2048 -> 65536) and the BF16 sites of the step at M in {1, 8, 32, 128, 25
 copies of at least 512 MB, cuBLASLt on the same buffers beside every point, each against
 max(bytes / HBM peak, flops / tensor peak).  A compact table of its E4M3 half is part of the default line
 (`gemm_roofline`).
+
+Workload `stack` times a layer-stack model (Fegidra) at LFM2.5-1.2B's sizes beside the LFM2 model, both in BF16:
+decode steps replayed from graphs at several batch sizes, mixed prefill steps, and every kernel's device time.
 
 `cpu_baseline` / `--impl reference`: the reference project is GPU-only, so the CPU arm is the multithreaded C
 restatement of its kernels (oracle/), timed on the same step (all 128 sequences, one step) on the host's cores.
@@ -62,7 +65,7 @@ STEP_POOL_PAGES = 32768
 def parse_arguments():
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
-    parser.add_argument("--workload", default="step", choices=["step", "attention", "gemm", "prefill", "serving"])
+    parser.add_argument("--workload", default="step", choices=["step", "attention", "gemm", "prefill", "serving", "stack"])
     parser.add_argument("--steps", type=int, default=0, help="timed steps (default 256 for step, 1024 for attention)")
     parser.add_argument("--warmup", type=int, default=0, help="warm-up steps (default 8 / 32)")
     parser.add_argument("--no-fp8", action="store_true", help="step workload: run every site in BF16")
@@ -98,9 +101,9 @@ def parse_arguments():
                              "reference's admission) instead of queueing them")
     arguments = parser.parse_args()
     if arguments.steps <= 0:
-        arguments.steps = {"step": 256, "attention": 1024, "prefill": 16, "serving": 1, "gemm": 64}[arguments.workload]
+        arguments.steps = {"step": 256, "attention": 1024, "prefill": 16, "serving": 1, "gemm": 64, "stack": 64}[arguments.workload]
     if arguments.warmup <= 0:
-        arguments.warmup = {"step": 8, "attention": 32, "prefill": 3, "serving": 3, "gemm": 3}[arguments.workload]
+        arguments.warmup = {"step": 8, "attention": 32, "prefill": 3, "serving": 3, "gemm": 3, "stack": 3}[arguments.workload]
     globals().update(SEQUENCES=arguments.sequences, NUM_PAGES=arguments.pool_pages,
                      STEP_SEQUENCES=arguments.step_sequences)
     return arguments
@@ -1452,6 +1455,38 @@ def run_serving_arm(arguments, rank, world):
         dist.destroy_process_group()
 
 
+def run_stack_arm(arguments, rank, world):
+    """Layer-stack model beside the LFM2 model (stack_bench): one JSON line; every replica measures the same cases."""
+    import torch
+    import torch.distributed as dist
+
+    local_rank = int(os.environ.get("LOCAL_RANK", rank))
+    torch.cuda.set_device(local_rank)
+    device = torch.device("cuda", local_rank)
+    if world > 1:
+        dist.init_process_group("nccl", device_id=device)
+    entry.load_package()
+    from lfm25_inference_b200 import ops, stack_bench
+    hbm, hbm_source = peaks()
+    tensor, tensor_source = tensor_peaks()
+    with ClockSampler(local_rank) as sampler:
+        result = stack_bench.run(device, arguments.steps, hbm, tensor)
+    slowest = max_over_ranks([result["decode"][-1]["stack"]["ms_per_step"]], device, world)[0]
+    if rank == 0:
+        sequences = result["decode"][-1]["sequences"]
+        print(json.dumps({
+            "metric": "decode tok/s (Fegidra at LFM2.5-1.2B sizes, random weights)",
+            "value": aggregate_throughput(sequences, world, slowest), "unit": "tok/s", "n_gpus": world,
+            "steps": arguments.steps, "warmup": arguments.warmup, "ms_per_step": slowest, "higher_is_better": True,
+            "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+            "config": {"model": "Fegidra, width 2048, 16 layers", "sequences": sequences, "replicas": world,
+                       "l2": "more than 2 GB of weights streamed per step exceed L2"},
+            "peaks": {"hbm_gbs": [hbm, hbm_source], "bf16_tflops": [tensor, tensor_source]},
+            "cases": result, "device_status": list(ops.device_status()), "clocks": sampler.summary()}), flush=True)
+    if world > 1:
+        dist.destroy_process_group()
+
+
 def main():
     arguments = parse_arguments()
     rank = int(os.environ.get("RANK", 0))
@@ -1474,6 +1509,11 @@ def main():
             run_dispatched_serving_arm(arguments, rank, world)
         else:
             run_serving_arm(arguments, rank, world)
+        return
+    if arguments.workload == "stack":
+        if arguments.impl == "reference":
+            raise SystemExit("--impl reference times the decode workloads")
+        run_stack_arm(arguments, rank, world)
         return
     if arguments.workload == "prefill":
         if arguments.impl == "reference":

@@ -215,6 +215,7 @@ int32_t linear_fp8_dispatch(cudaStream_t stream, lfm25_slice x, lfm25_slice weig
 
 namespace lfm25 {
 int32_t report_error(int32_t code, const char* message) { return fail(code, "%s", message); }
+unsigned int* device_status_words() { return device_status_pointer(); }
 }  // namespace lfm25
 
 extern "C" {

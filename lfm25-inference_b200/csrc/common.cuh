@@ -32,7 +32,9 @@ enum StatusTag : uint32_t {
     kTagGemmStream = 2,
     kTagGemmUmma = 3,
     kTagHybridAttention = 4,
-    kTagGemmRows = 5
+    kTagGemmRows = 5,
+    kTagStackAttention = 6,
+    kTagStackDecode = 7
 };
 __device__ __forceinline__ void record_wait_timeout(unsigned int* status, uint32_t tag, uint32_t detail) {
     atomicAdd(&status[0], 1u);

@@ -4,13 +4,19 @@
 // per head, with w_t = exp(-exp(-1/2) sigmoid(W2 tanh(z_t) + w0)) and a_t = sigmoid(a_t' + bias), followed by the
 // head's RMS norm, the norm weight and the output gate.
 //
-// A column of S (one value channel) never meets another one, so a CTA takes the columns of one head of one sequence,
-// LANES threads a column, and keeps them in registers over the whole segment: the state is read from and written to
-// memory once per step however long the segment is.  Everything a token contributes is prepared for a tile of tokens
-// in shared memory (all in f32) and then consumed token by token: per token a thread forms its share of u^T S, LANES
-// threads add theirs up, and the same pass over its rows updates S and accumulates r^T S.  Arithmetic on the state
-// uses the packed two-wide f32 instructions of sm_100 (each half rounds like the scalar one).
+// A column of S (one value channel) never meets another one, so a CTA takes the columns of one head of one sequence and
+// keeps them in registers over the whole segment: the state is read from and written to memory once per step however
+// long the segment is.  Three kernels:
+//   decode    one token per sequence: every load is issued up front, then three barriers
+//   prompt    bf16 segments: half of the warps prepare a tile of 16 tokens (decays with one small tensor-core product,
+//             removal rates, unit scales) and finish the previous one (norm, gate), the others run the recurrence over
+//             the tile between them; projections arrive through cp.async two tiles ahead
+//   general   any activation type and head size
+// All arithmetic on the state is f32 multiply-adds, two-wide where the sm_100 packed instructions take it (each half
+// rounds like the scalar one).
 #include <math.h>
+
+#include <type_traits>
 
 #include "launch.h"
 #include "stack_common.cuh"
@@ -31,6 +37,8 @@ __device__ __forceinline__ float pair_sum(Pair value) {
     asm("mov.b64 {%0, %1}, %2;" : "=f"(low), "=f"(high) : "l"(value));
     return low + high;
 }
+__device__ __forceinline__ float low_of(Pair value) { return __uint_as_float(static_cast<uint32_t>(value)); }
+__device__ __forceinline__ float high_of(Pair value) { return __uint_as_float(static_cast<uint32_t>(value >> 32)); }
 __device__ __forceinline__ Pair fma_pair(Pair a, Pair b, Pair c) {
     Pair out;
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(out) : "l"(a), "l"(b), "l"(c));
@@ -95,6 +103,11 @@ __device__ __forceinline__ Prepared prepare(const DeltaArgs<T>& args, const T* r
     return p;
 }
 
+// ------------------------------------------------------------------------------------------------ general kernel
+
+// LANES threads a column.  Everything a token contributes is prepared for a tile of tokens in shared memory (all in f32)
+// and then consumed token by token: per token a thread forms its share of u^T S, LANES threads add theirs up, and the
+// same pass over its rows updates S and accumulates r^T S.
 // TOKENS: tokens per tile (1 = decode steps).  STAGED: the head's rows of W2 sit in shared memory.
 template <typename T, uint32_t DP, uint32_t LANES, uint32_t COLUMNS, uint32_t TOKENS, bool STAGED>
 __global__ void __launch_bounds__(LANES * COLUMNS)
@@ -351,6 +364,587 @@ delta_output_kernel(const DeltaArgs<T> args) {
     }
 }
 
+
+// ------------------------------------------------------------------------------------------------ decode kernel
+
+// One token per sequence, one CTA per sequence and head; four threads per value column (for the state) and per key
+// channel (for what the token contributes).
+template <typename T, uint32_t DP>
+__global__ void __launch_bounds__(DP * 4)
+delta_decode_kernel(const DeltaArgs<T> args) {
+    constexpr uint32_t kThreads = DP * 4;
+    constexpr uint32_t kGroups = DP / 16;              // groups of four key channels per thread
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) float shared[];
+    float* r_values = shared;                          // [DP] each
+    float* w_values = r_values + DP;
+    float* removal_values = w_values + DP;
+    float* u_values = removal_values + DP;
+    float* k_values = u_values + DP;
+    float* partial = k_values + DP;                    // [warps] twice: |k|^2, |o|^2
+    float* z_values = partial + 2 * (kThreads / 32);   // [rank]
+    const uint32_t dim = args.dim;
+    const uint32_t head = blockIdx.x % args.heads;
+    const size_t token = blockIdx.x / args.heads;
+    const size_t slot = args.segments.slots[token];
+    if (slot >= args.segments.num_request_slots) {
+        return;
+    }
+    const uint32_t channel = threadIdx.x / 4;          // value column and key channel
+    const uint32_t lane = threadIdx.x % 4;
+    const bool live = channel < dim;
+    const size_t width = static_cast<size_t>(args.heads) * dim;
+    const size_t head_base = static_cast<size_t>(head) * dim;
+    float* state_column = reinterpret_cast<float*>(static_cast<unsigned char*>(args.record.base) +
+                                                   slot * args.record.stride + args.record.offset) +
+                          (head_base + channel) * dim;
+    const bool vector_state = dim % 4 == 0;
+    Pair state[kGroups * 2];
+#pragma unroll
+    for (uint32_t g = 0; g < kGroups; ++g) {
+        const uint32_t row = (g * 4 + lane) * 4;
+        float4 value = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (live && row < dim) {
+            if (vector_state) {
+                value = __ldcs(reinterpret_cast<const float4*>(state_column + row));
+            } else {
+                value.x = state_column[row];
+                if (row + 1 < dim) value.y = state_column[row + 1];
+                if (row + 2 < dim) value.z = state_column[row + 2];
+                if (row + 3 < dim) value.w = state_column[row + 3];
+            }
+        }
+        state[2 * g] = pair_of(value.x, value.y);
+        state[2 * g + 1] = pair_of(value.z, value.w);
+    }
+    const T* row = args.projected + token * args.pitch;
+    float r = 0.0f, k = 0.0f, v = 0.0f, gate = 0.0f, removal = 0.0f, base = 0.0f, weight = 0.0f;
+    if (live) {
+        const size_t index = head_base + channel;
+        r = to_float<T>(row[index]);
+        k = to_float<T>(row[width + index]);
+        v = to_float<T>(row[2 * width + index]);
+        gate = to_float<T>(row[3 * width + index]);
+        removal = to_float<T>(row[4 * width + index]) + __bfloat162float(args.removal_bias[index]);
+        base = __bfloat162float(args.decay_base[index]);
+        weight = __bfloat162float(args.norm[index]);
+    }
+    for (uint32_t z = threadIdx.x; z < args.rank; z += kThreads) z_values[z] = tanhf(to_float<T>(row[5 * width + z]));
+    // this thread's quarter of the channel's row of W2, its first 16 values in registers before the barrier
+    const uint32_t part = (args.rank / 4 + 7) / 8 * 8;
+    const uint32_t from = min(lane * part, args.rank);
+    const uint32_t to = lane == 3 ? args.rank : min(from + part, args.rank);
+    const __nv_bfloat16* decay_row = args.decay_up + (head_base + (live ? channel : 0)) * args.rank;
+    const bool vector_rank = args.rank % 8 == 0;
+    uint4 early[2] = {};
+    if (live && vector_rank) {
+#pragma unroll
+        for (uint32_t i = 0; i < 2; ++i) {
+            if (from + 8 * i < to) early[i] = *reinterpret_cast<const uint4*>(decay_row + from + 8 * i);
+        }
+    }
+    // every channel is held by four threads
+    const float k_squares = warp_sum(lane == 0 ? k * k : 0.0f);
+    const uint32_t warp = threadIdx.x / 32;
+    if (threadIdx.x % 32 == 0) partial[warp] = k_squares;
+    __syncthreads();
+    float logit = 0.0f;
+    if (live) {
+        if (vector_rank) {
+            for (uint32_t z = from; z < to; z += 8) {
+                const uint4 raw = z < from + 16 ? (z == from ? early[0] : early[1])
+                                                : *reinterpret_cast<const uint4*>(decay_row + z);
+                const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+                for (uint32_t i = 0; i < 4; ++i) {
+                    const float2 both = __bfloat1622float2(pairs[i]);
+                    logit = fmaf(both.x, z_values[z + 2 * i], logit);
+                    logit = fmaf(both.y, z_values[z + 2 * i + 1], logit);
+                }
+            }
+        } else {
+            for (uint32_t z = from; z < to; ++z) logit = fmaf(__bfloat162float(decay_row[z]), z_values[z], logit);
+        }
+    }
+    logit += __shfl_xor_sync(0xffffffffu, logit, 1);
+    logit += __shfl_xor_sync(0xffffffffu, logit, 2);
+    float squares = 0.0f;
+#pragma unroll
+    for (uint32_t w = 0; w < kThreads / 32; ++w) squares += partial[w];
+    const float u = k / sqrtf(squares + kUnitEps);
+    if (lane == 0) {
+        w_values[channel] = expf(-kDecayScale * sigmoidf(logit + base));
+    } else if (lane == 1) {
+        removal_values[channel] = -sigmoidf(removal) * u;
+    } else if (lane == 2) {
+        u_values[channel] = u;
+        r_values[channel] = r;
+    } else {
+        k_values[channel] = k;
+    }
+    __syncthreads();
+    Pair dot0 = 0, dot1 = 0;                           // bit pattern of (0.0f, 0.0f)
+#pragma unroll
+    for (uint32_t g = 0; g < kGroups; ++g) {
+        const ulonglong2 unit = *reinterpret_cast<const ulonglong2*>(u_values + (g * 4 + lane) * 4);
+        dot0 = fma_pair(unit.x, state[2 * g], dot0);
+        dot1 = fma_pair(unit.y, state[2 * g + 1], dot1);
+    }
+    float dot = pair_sum(dot0) + pair_sum(dot1);
+    dot += __shfl_xor_sync(0xffffffffu, dot, 1);
+    dot += __shfl_xor_sync(0xffffffffu, dot, 2);
+    const Pair recalled = pair_of(dot, dot);
+    const Pair values = pair_of(v, v);
+    Pair sum0 = 0, sum1 = 0;
+#pragma unroll
+    for (uint32_t g = 0; g < kGroups; ++g) {
+        const uint32_t at = (g * 4 + lane) * 4;
+        const ulonglong2 rr = *reinterpret_cast<const ulonglong2*>(r_values + at);
+        const ulonglong2 ww = *reinterpret_cast<const ulonglong2*>(w_values + at);
+        const ulonglong2 aa = *reinterpret_cast<const ulonglong2*>(removal_values + at);
+        const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(k_values + at);
+        state[2 * g] = fma_pair(kk.x, values, fma_pair(aa.x, recalled, mul_pair(ww.x, state[2 * g])));
+        state[2 * g + 1] = fma_pair(kk.y, values, fma_pair(aa.y, recalled, mul_pair(ww.y, state[2 * g + 1])));
+        sum0 = fma_pair(rr.x, state[2 * g], sum0);
+        sum1 = fma_pair(rr.y, state[2 * g + 1], sum1);
+        if (live && at < dim) {
+            const float4 value = {low_of(state[2 * g]), high_of(state[2 * g]), low_of(state[2 * g + 1]),
+                                  high_of(state[2 * g + 1])};
+            if (vector_state) {
+                __stcs(reinterpret_cast<float4*>(state_column + at), value);
+            } else {
+                state_column[at] = value.x;
+                if (at + 1 < dim) state_column[at + 1] = value.y;
+                if (at + 2 < dim) state_column[at + 2] = value.z;
+                if (at + 3 < dim) state_column[at + 3] = value.w;
+            }
+        }
+    }
+    float result = pair_sum(sum0) + pair_sum(sum1);
+    result += __shfl_xor_sync(0xffffffffu, result, 1);
+    result += __shfl_xor_sync(0xffffffffu, result, 2);
+    const float o_squares = warp_sum(lane == 0 && live ? result * result : 0.0f);
+    if (threadIdx.x % 32 == 0) partial[kThreads / 32 + warp] = o_squares;
+    __syncthreads();
+    squares = 0.0f;
+#pragma unroll
+    for (uint32_t w = 0; w < kThreads / 32; ++w) squares += partial[kThreads / 32 + w];
+    if (lane == 0 && live) {
+        args.out[token * args.out_pitch + head_base + channel] =
+            from_float<T>(result * inverse_rms(squares, dim, args.eps) * weight * sigmoidf(gate));
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ prompt kernel
+
+// 16-byte copy global -> shared without registers
+__device__ __forceinline__ void copy_async_16(void* target, const void* source) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(target)), "l"(source) : "memory");
+}
+__device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int PENDING>
+__device__ __forceinline__ void copy_async_wait() {
+    asm volatile("cp.async.wait_group %0;" ::"n"(PENDING) : "memory");
+}
+__device__ __forceinline__ void named_barrier(uint32_t id, uint32_t threads) {
+    asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory");
+}
+
+constexpr uint32_t kPromptTokens = 16;       // tokens per tile = rows of one MMA tile
+constexpr uint32_t kHelpers = 128;           // threads that prepare and finish
+constexpr uint32_t kRawStages = 4;           // being finished, in the recurrence, being prepared, arriving
+constexpr uint32_t kPromptMaxRank = 256;
+
+template <uint32_t DP>
+struct PromptLayout {
+    uint32_t rank_pad;        // multiple of 16
+    uint32_t z_stride;        // bf16 elements between rows of z / W2 in shared memory: 16-byte rows, no bank conflicts
+    uint32_t raw_row;         // bf16 elements per token: r | k | v | g | a (DP each) | z
+    size_t raw, vectors, produced, tanh_parts, w2, constants, scale, total;
+    __host__ __device__ explicit PromptLayout(uint32_t rank) {
+        rank_pad = (rank + 15) / 16 * 16;
+        z_stride = rank_pad + 8;
+        raw_row = 5 * DP + rank_pad;
+        size_t at = 0;
+        raw = at;
+        at += static_cast<size_t>(kRawStages) * kPromptTokens * raw_row * 2;
+        vectors = at;                                             // [2][tokens][2][DP] f32: w, removal / |k|
+        at += 2 * kPromptTokens * 2 * DP * 4;
+        produced = at;                                            // [2][tokens][DP] f32
+        at += 2 * kPromptTokens * DP * 4;
+        tanh_parts = at;                                          // [2][tokens][z_stride] bf16: high and low parts
+        at += 2 * kPromptTokens * z_stride * 2;
+        w2 = at;                                                  // [DP][z_stride] bf16
+        at += static_cast<size_t>(DP) * z_stride * 2;
+        constants = at;                                           // [3][DP] f32: w0, removal bias, norm weight
+        at += 3 * DP * 4;
+        scale = at;                                               // [2][tokens] f32: 1 / |k|
+        at += 2 * kPromptTokens * 4;
+        total = at;
+    }
+};
+
+// Where key channel `row` of a prepared f32 vector lies: the 4-channel groups of the eight threads that share a column
+// are interleaved, so that their 16-byte reads are consecutive.
+template <uint32_t DP>
+__device__ __forceinline__ uint32_t interleaved(uint32_t row) {
+    constexpr uint32_t kRows = DP / 8;
+    return row % kRows / 4 * 32 + row / kRows * 4 + row % 4;
+}
+
+// 2 * DP threads run the recurrence: eight per group of four value columns, DP / 8 consecutive key channels each.
+template <uint32_t DP>
+__global__ void __launch_bounds__(2 * DP + kHelpers)
+delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
+    constexpr uint32_t kRows = DP / 8;
+    constexpr uint32_t kScanThreads = 2 * DP;
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) unsigned char prompt_shared[];
+    const PromptLayout<DP> layout(args.rank);
+    const uint32_t dim = args.dim;
+    const uint32_t head = blockIdx.x % args.heads;
+    const uint32_t segment = blockIdx.x / args.heads;
+    const uint32_t begin = args.segments.offsets[segment];
+    uint32_t end = args.segments.offsets[segment + 1];
+    end = end < args.segments.num_tokens ? end : static_cast<uint32_t>(args.segments.num_tokens);
+    const size_t slot = args.segments.slots[segment];
+    if (begin >= end || slot >= args.segments.num_request_slots) {
+        return;
+    }
+    const uint32_t tiles = (end - begin + kPromptTokens - 1) / kPromptTokens;
+    const size_t width = static_cast<size_t>(args.heads) * dim;
+    const size_t head_base = static_cast<size_t>(head) * dim;
+    auto* raw = reinterpret_cast<__nv_bfloat16*>(prompt_shared + layout.raw);
+    auto* vectors = reinterpret_cast<float*>(prompt_shared + layout.vectors);
+    auto* produced = reinterpret_cast<float*>(prompt_shared + layout.produced);
+    auto* tanh_parts = reinterpret_cast<__nv_bfloat16*>(prompt_shared + layout.tanh_parts);
+    auto* w2 = reinterpret_cast<__nv_bfloat16*>(prompt_shared + layout.w2);
+    auto* constants = reinterpret_cast<float*>(prompt_shared + layout.constants);
+    auto* scale = reinterpret_cast<float*>(prompt_shared + layout.scale);
+    float* state_base = reinterpret_cast<float*>(static_cast<unsigned char*>(args.record.base) +
+                                                 slot * args.record.stride + args.record.offset) +
+                        head_base * dim;
+
+    // padding channels and tokens that never arrive stay zero
+    for (uint32_t item = threadIdx.x; item < kRawStages * kPromptTokens * layout.raw_row / 8;
+         item += kScanThreads + kHelpers) {
+        reinterpret_cast<uint4*>(raw)[item] = make_uint4(0, 0, 0, 0);
+    }
+    for (uint32_t item = threadIdx.x; item < DP * layout.z_stride; item += kScanThreads + kHelpers) {
+        const uint32_t channel = item / layout.z_stride;
+        const uint32_t z = item % layout.z_stride;
+        w2[item] = channel < dim && z < args.rank ? args.decay_up[(head_base + channel) * args.rank + z]
+                                                  : __float2bfloat16_rn(0.0f);
+    }
+    for (uint32_t channel = threadIdx.x; channel < DP; channel += kScanThreads + kHelpers) {
+        const bool live = channel < dim;
+        constants[channel] = live ? __bfloat162float(args.decay_base[head_base + channel]) : 0.0f;
+        constants[DP + channel] = live ? __bfloat162float(args.removal_bias[head_base + channel]) : 0.0f;
+        constants[2 * DP + channel] = live ? __bfloat162float(args.norm[head_base + channel]) : 0.0f;
+    }
+    __syncthreads();
+
+    const bool scanner = threadIdx.x < kScanThreads;
+    const uint32_t helper = threadIdx.x - kScanThreads;
+    const uint32_t helper_warp = helper / 32;
+    const uint32_t warp_lane = threadIdx.x % 32;
+
+    auto load_tile = [&](uint32_t tile) {             // helpers only; always one group per call
+        if (tile < tiles) {
+            const uint32_t first = begin + tile * kPromptTokens;
+            const uint32_t tokens = min(kPromptTokens, end - first);
+            const uint32_t per_vector = dim / 8;
+            const uint32_t z_copies = (args.rank + 7) / 8;
+            const uint32_t per_token = 5 * per_vector + z_copies;
+            __nv_bfloat16* stage = raw + tile % kRawStages * kPromptTokens * layout.raw_row;
+            for (uint32_t item = helper; item < tokens * per_token; item += kHelpers) {
+                const uint32_t t = item / per_token;
+                const uint32_t part = item - t * per_token;
+                const __nv_bfloat16* source = args.projected + static_cast<size_t>(first + t) * args.pitch;
+                __nv_bfloat16* target = stage + t * layout.raw_row;
+                if (part < 5 * per_vector) {
+                    const uint32_t vector = part / per_vector;
+                    const uint32_t chunk = part - vector * per_vector;
+                    copy_async_16(target + vector * DP + chunk * 8, source + vector * width + head_base + chunk * 8);
+                } else {
+                    const uint32_t chunk = part - 5 * per_vector;
+                    copy_async_16(target + 5 * DP + chunk * 8, source + 5 * width + chunk * 8);
+                }
+            }
+        }
+        copy_async_commit();
+    };
+
+    auto prepare_tile = [&](uint32_t tile) {          // helpers only; the tile's copies have arrived for all of them
+        const __nv_bfloat16* stage = raw + tile % kRawStages * kPromptTokens * layout.raw_row;
+        float* target = vectors + tile % 2 * kPromptTokens * 2 * DP;
+        float* unit = scale + tile % 2 * kPromptTokens;
+#pragma unroll
+        for (uint32_t i = 0; i < kPromptTokens / 4; ++i) {
+            const uint32_t t = helper_warp * (kPromptTokens / 4) + i;
+            const __nv_bfloat16* k = stage + t * layout.raw_row + DP;
+            float sum = 0.0f;
+#pragma unroll
+            for (uint32_t part = 0; part < DP / 64; ++part) {
+                const float2 both =
+                    __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k + part * 64 + warp_lane * 2));
+                sum = fmaf(both.x, both.x, fmaf(both.y, both.y, sum));
+            }
+            sum = warp_sum(sum);
+            if (warp_lane == 0) unit[t] = 1.0f / sqrtf(sum + kUnitEps);
+        }
+        for (uint32_t item = helper; item < kPromptTokens * layout.rank_pad; item += kHelpers) {
+            const uint32_t t = item / layout.rank_pad;
+            const uint32_t z = item - t * layout.rank_pad;
+            // columns between rank and its multiple of eight arrive with the copy and belong to nobody: W2 is zero there
+            const float value = z < args.rank ? tanhf(__bfloat162float(stage[t * layout.raw_row + 5 * DP + z])) : 0.0f;
+            const __nv_bfloat16 high = __float2bfloat16_rn(value);
+            tanh_parts[t * layout.z_stride + z] = high;
+            tanh_parts[(kPromptTokens + t) * layout.z_stride + z] = __float2bfloat16_rn(value - __bfloat162float(high));
+        }
+        named_barrier(1, kHelpers);
+        // decay logits of 16 tokens x (DP / 4) channels per warp: tanh(z) W2^T with tanh(z) as a sum of two bf16 values
+        constexpr uint32_t kTilesPerWarp = DP / 32;
+        float logits[kTilesPerWarp][4] = {};
+        const uint32_t z_row = warp_lane % 16, z_part = warp_lane / 16 * 8;
+        for (uint32_t step = 0; step < layout.rank_pad; step += 16) {
+            uint32_t high[4], low[4];
+            ldmatrix_x4(smem_u32(tanh_parts + z_row * layout.z_stride + step + z_part), high[0], high[1], high[2], high[3]);
+            ldmatrix_x4(smem_u32(tanh_parts + (kPromptTokens + z_row) * layout.z_stride + step + z_part), low[0], low[1],
+                        low[2], low[3]);
+#pragma unroll
+            for (uint32_t n = 0; n < kTilesPerWarp; n += 2) {
+                const uint32_t channel = helper_warp * (DP / 4) + n * 8 + warp_lane / 16 * 8 + warp_lane % 8;
+                uint32_t b0, b1, b2, b3;
+                ldmatrix_x4(smem_u32(w2 + channel * layout.z_stride + step + warp_lane / 8 % 2 * 8), b0, b1, b2, b3);
+                mma_bf16_16816(logits[n], high[0], high[1], high[2], high[3], b0, b1);
+                mma_bf16_16816(logits[n], low[0], low[1], low[2], low[3], b0, b1);
+                mma_bf16_16816(logits[n + 1], high[0], high[1], high[2], high[3], b2, b3);
+                mma_bf16_16816(logits[n + 1], low[0], low[1], low[2], low[3], b2, b3);
+            }
+        }
+#pragma unroll
+        for (uint32_t n = 0; n < kTilesPerWarp; ++n) {
+            const uint32_t channel = helper_warp * (DP / 4) + n * 8 + warp_lane % 4 * 2;
+#pragma unroll
+            for (uint32_t half = 0; half < 2; ++half) {
+                const uint32_t t = warp_lane / 4 + half * 8;
+                const float2 rate = __bfloat1622float2(
+                    *reinterpret_cast<const __nv_bfloat162*>(stage + t * layout.raw_row + 4 * DP + channel));
+                float2 w, removal;
+                w.x = expf(-kDecayScale * sigmoidf(logits[n][2 * half] + constants[channel]));
+                w.y = expf(-kDecayScale * sigmoidf(logits[n][2 * half + 1] + constants[channel + 1]));
+                // -(a * u) (u^T S) = -(a / |k|) * k * (u^T S): the recurrence multiplies by k anyway
+                removal.x = -sigmoidf(rate.x + constants[DP + channel]) * unit[t];
+                removal.y = -sigmoidf(rate.y + constants[DP + channel + 1]) * unit[t];
+                const uint32_t at = interleaved<DP>(channel);
+                *reinterpret_cast<float2*>(target + t * 2 * DP + at) = w;
+                *reinterpret_cast<float2*>(target + t * 2 * DP + DP + at) = removal;
+            }
+        }
+    };
+
+    auto finish_tile = [&](uint32_t tile) {           // helpers only
+        const __nv_bfloat16* stage = raw + tile % kRawStages * kPromptTokens * layout.raw_row;
+        const float* source = produced + tile % 2 * kPromptTokens * DP;
+        const uint32_t first = begin + tile * kPromptTokens;
+#pragma unroll
+        for (uint32_t i = 0; i < kPromptTokens / 4; ++i) {
+            const uint32_t t = helper_warp * (kPromptTokens / 4) + i;
+            if (first + t >= end) break;
+            float2 value[DP / 64];
+            float sum = 0.0f;
+#pragma unroll
+            for (uint32_t part = 0; part < DP / 64; ++part) {
+                value[part] = *reinterpret_cast<const float2*>(source + t * DP + part * 64 + warp_lane * 2);
+                sum = fmaf(value[part].x, value[part].x, fmaf(value[part].y, value[part].y, sum));
+            }
+            const float factor = inverse_rms(warp_sum(sum), dim, args.eps);
+#pragma unroll
+            for (uint32_t part = 0; part < DP / 64; ++part) {
+                const uint32_t channel = part * 64 + warp_lane * 2;
+                if (channel < dim) {
+                    const float2 gate = __bfloat1622float2(
+                        *reinterpret_cast<const __nv_bfloat162*>(stage + t * layout.raw_row + 3 * DP + channel));
+                    const float2 weight = *reinterpret_cast<const float2*>(constants + 2 * DP + channel);
+                    const uint32_t both = pack_bf16x2(value[part].x * factor * weight.x * sigmoidf(gate.x),
+                                                      value[part].y * factor * weight.y * sigmoidf(gate.y));
+                    *reinterpret_cast<uint32_t*>(args.out + static_cast<size_t>(first + t) * args.out_pitch + head_base +
+                                                 channel) = both;
+                }
+            }
+        }
+    };
+
+    // ---- the state: columns 4 * group .. + 3, key channels lane * kRows .. + kRows - 1
+    const uint32_t lane = threadIdx.x % 8;
+    const uint32_t column0 = threadIdx.x / 8 * 4;
+    Pair state[4][kRows / 2];
+    if (scanner) {
+#pragma unroll
+        for (uint32_t c = 0; c < 4; ++c) {
+#pragma unroll
+            for (uint32_t g = 0; g < kRows / 4; ++g) {
+                const uint32_t row = lane * kRows + g * 4;
+                float4 value = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                if (column0 + c < dim && row < dim) {          // dim is a multiple of 8
+                    value = *reinterpret_cast<const float4*>(state_base + static_cast<size_t>(column0 + c) * dim + row);
+                }
+                state[c][2 * g] = pair_of(value.x, value.y);
+                state[c][2 * g + 1] = pair_of(value.z, value.w);
+            }
+        }
+    } else {
+        load_tile(0);
+        load_tile(1);
+        copy_async_wait<1>();
+        named_barrier(1, kHelpers);
+        prepare_tile(0);
+    }
+    __syncthreads();
+
+    for (uint32_t tile = 0; tile < tiles; ++tile) {
+        if (scanner) {
+            const uint32_t tokens = min(kPromptTokens, end - begin - tile * kPromptTokens);
+            const __nv_bfloat16* stage = raw + tile % kRawStages * kPromptTokens * layout.raw_row;
+            const float* prepared = vectors + tile % 2 * kPromptTokens * 2 * DP;
+            const float* unit = scale + tile % 2 * kPromptTokens;
+            float* target = produced + tile % 2 * kPromptTokens * DP;
+#pragma unroll 2
+            for (uint32_t t = 0; t < tokens; ++t) {
+                const __nv_bfloat16* row = stage + t * layout.raw_row;
+                Pair k[kRows / 2], r[kRows / 2];
+#pragma unroll
+                for (uint32_t part = 0; part < kRows / 8; ++part) {
+                    const uint4 k_raw = *reinterpret_cast<const uint4*>(row + DP + lane * kRows + part * 8);
+                    const uint4 r_raw = *reinterpret_cast<const uint4*>(row + lane * kRows + part * 8);
+                    const uint32_t k_words[4] = {k_raw.x, k_raw.y, k_raw.z, k_raw.w};
+                    const uint32_t r_words[4] = {r_raw.x, r_raw.y, r_raw.z, r_raw.w};
+#pragma unroll
+                    for (uint32_t i = 0; i < 4; ++i) {       // bf16 -> f32 is a shift
+                        k[part * 4 + i] = pair_of(__uint_as_float(k_words[i] << 16),
+                                                  __uint_as_float(k_words[i] & 0xffff0000u));
+                        r[part * 4 + i] = pair_of(__uint_as_float(r_words[i] << 16),
+                                                  __uint_as_float(r_words[i] & 0xffff0000u));
+                    }
+                }
+                const uint2 v_raw = *reinterpret_cast<const uint2*>(row + 2 * DP + column0);
+                const float v[4] = {__uint_as_float(v_raw.x << 16), __uint_as_float(v_raw.x & 0xffff0000u),
+                                    __uint_as_float(v_raw.y << 16), __uint_as_float(v_raw.y & 0xffff0000u)};
+                float dot[4];
+#pragma unroll
+                for (uint32_t c = 0; c < 4; ++c) {
+                    Pair even = mul_pair(k[0], state[c][0]);
+                    Pair odd = mul_pair(k[1], state[c][1]);
+#pragma unroll
+                    for (uint32_t i = 2; i < kRows / 2; i += 2) {
+                        even = fma_pair(k[i], state[c][i], even);
+                        odd = fma_pair(k[i + 1], state[c][i + 1], odd);
+                    }
+                    dot[c] = pair_sum(even) + pair_sum(odd);
+                }
+#pragma unroll
+                for (uint32_t delta = 1; delta < 8; delta <<= 1) {
+#pragma unroll
+                    for (uint32_t c = 0; c < 4; ++c) dot[c] += __shfl_xor_sync(0xffffffffu, dot[c], delta);
+                }
+                const float unit_scale = unit[t];
+                const float* token = prepared + t * 2 * DP;
+                Pair sums[4] = {0, 0, 0, 0};
+                Pair recalled[4], values[4];
+#pragma unroll
+                for (uint32_t c = 0; c < 4; ++c) {
+                    const float product = dot[c] * unit_scale;
+                    recalled[c] = pair_of(product, product);
+                    values[c] = pair_of(v[c], v[c]);
+                }
+#pragma unroll
+                for (uint32_t g = 0; g < kRows / 4; ++g) {
+                    const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(token + g * 32 + lane * 4);
+                    const ulonglong2 removal = *reinterpret_cast<const ulonglong2*>(token + DP + g * 32 + lane * 4);
+#pragma unroll
+                    for (uint32_t c = 0; c < 4; ++c) {
+                        // w S + k (v - (a / |k|) (u^T S))
+                        state[c][2 * g] = fma_pair(k[2 * g], fma_pair(removal.x, recalled[c], values[c]),
+                                                   mul_pair(w.x, state[c][2 * g]));
+                        state[c][2 * g + 1] = fma_pair(k[2 * g + 1], fma_pair(removal.y, recalled[c], values[c]),
+                                                       mul_pair(w.y, state[c][2 * g + 1]));
+                        sums[c] = fma_pair(r[2 * g], state[c][2 * g], sums[c]);
+                        sums[c] = fma_pair(r[2 * g + 1], state[c][2 * g + 1], sums[c]);
+                    }
+                }
+                // the four column sums over the eight threads, each pair of threads keeping half of the columns
+                float result[4];
+#pragma unroll
+                for (uint32_t c = 0; c < 4; ++c) result[c] = pair_sum(sums[c]);
+                const bool upper1 = lane & 1, upper2 = lane & 2;
+                const float keep0 = upper1 ? result[2] : result[0], keep1 = upper1 ? result[3] : result[1];
+                const float give0 = upper1 ? result[0] : result[2], give1 = upper1 ? result[1] : result[3];
+                const float half0 = keep0 + __shfl_xor_sync(0xffffffffu, give0, 1);
+                const float half1 = keep1 + __shfl_xor_sync(0xffffffffu, give1, 1);
+                float total = (upper2 ? half1 : half0) + __shfl_xor_sync(0xffffffffu, upper2 ? half0 : half1, 2);
+                total += __shfl_xor_sync(0xffffffffu, total, 4);
+                if (lane < 4) target[t * DP + column0 + (lane & 1) * 2 + (lane >> 1)] = total;
+            }
+        } else {
+            load_tile(tile + 2);
+            if (tile > 0) finish_tile(tile - 1);
+            copy_async_wait<1>();                     // tile + 1 has arrived for this thread ...
+            named_barrier(1, kHelpers);               // ... and for all helpers
+            if (tile + 1 < tiles) prepare_tile(tile + 1);
+        }
+        __syncthreads();
+    }
+    if (scanner) {
+#pragma unroll
+        for (uint32_t c = 0; c < 4; ++c) {
+#pragma unroll
+            for (uint32_t g = 0; g < kRows / 4; ++g) {
+                const uint32_t row = lane * kRows + g * 4;
+                if (column0 + c < dim && row < dim) {
+                    *reinterpret_cast<float4*>(state_base + static_cast<size_t>(column0 + c) * dim + row) =
+                        make_float4(low_of(state[c][2 * g]), high_of(state[c][2 * g]), low_of(state[c][2 * g + 1]),
+                                    high_of(state[c][2 * g + 1]));
+                }
+            }
+        }
+    } else {
+        finish_tile(tiles - 1);
+    }
+}
+
+template <typename T, uint32_t DP>
+cudaError_t launch_decode(cudaStream_t stream, const DeltaArgs<T>& args) {
+    const size_t shared = (5 * DP + 2 * (DP * 4 / 32) + args.rank) * sizeof(float);
+    if (shared > 48 * 1024) {
+        return cudaErrorInvalidValue;
+    }
+    return launch_kernel(delta_decode_kernel<T, DP>,
+                         static_cast<unsigned int>(args.segments.num_segments * args.heads), DP * 4, shared, stream, 1,
+                         args);
+}
+
+template <uint32_t DP>
+cudaError_t launch_prompt(cudaStream_t stream, const DeltaArgs<__nv_bfloat16>& args) {
+    const size_t shared = PromptLayout<DP>(args.rank).total;
+    const auto kernel = delta_prompt_kernel<DP>;
+    const cudaError_t status = cudaFuncSetAttribute(reinterpret_cast<const void*>(kernel),
+                                                    cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                    static_cast<int>(shared));
+    if (status != cudaSuccess) return status;
+    return launch_kernel(kernel, static_cast<unsigned int>(args.segments.num_segments * args.heads),
+                         2 * DP + kHelpers, shared, stream, 1, args);
+}
+
+bool prompt_kernel_takes(const DeltaArgs<__nv_bfloat16>& args) {
+    const size_t shared = args.dim <= 64 ? PromptLayout<64>(args.rank).total : PromptLayout<128>(args.rank).total;
+    return args.dim % 8 == 0 && args.dim <= 128 && args.rank <= kPromptMaxRank && args.pitch % 8 == 0 &&
+           args.out_pitch % 2 == 0 && aligned_to(args.projected, 16) && aligned_to(args.out, 4) &&
+           shared <= 227 * 1024;
+}
+
 template <typename T, uint32_t DP, uint32_t LANES, uint32_t COLUMNS>
 cudaError_t launch_sized(cudaStream_t stream, DeltaArgs<T> args) {
     args.splits = (args.dim + COLUMNS - 1) / COLUMNS;
@@ -402,6 +996,16 @@ cudaError_t launch_typed(cudaStream_t stream, const DeltaRuleLaunch& launch) {
     args.out_pitch = launch.out_pitch;
     args.eps = launch.eps;
     args.splits = 1;
+    if (launch.segments.offsets == nullptr && launch.dim <= 128 && launch.rank <= 4096) {
+        if (launch.dim <= 32) return launch_decode<T, 32>(stream, args);
+        if (launch.dim <= 64) return launch_decode<T, 64>(stream, args);
+        return launch_decode<T, 128>(stream, args);
+    }
+    if constexpr (std::is_same<T, __nv_bfloat16>::value) {
+        if (launch.segments.offsets != nullptr && prompt_kernel_takes(args)) {
+            return launch.dim <= 64 ? launch_prompt<64>(stream, args) : launch_prompt<128>(stream, args);
+        }
+    }
     if (launch.dim <= 32) return launch_sized<T, 32, 4, 32>(stream, args);
     if (launch.dim <= 64) return launch_sized<T, 64, 4, 64>(stream, args);
     if (launch.dim <= 128) return launch_sized<T, 128, 4, 128>(stream, args);

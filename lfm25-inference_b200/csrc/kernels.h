@@ -191,6 +191,9 @@ bool bf16_gemm_umma_supports(size_t m, size_t n, size_t k);
 cudaError_t launch_bf16_gemm_umma(cudaStream_t stream, const void* x, const void* weight, void* out, size_t m,
                                   size_t n, size_t k, void* exchange, size_t exchange_bytes, unsigned int* status);
 
+// The device status words of the bounded waits on the current device (nullptr when they cannot be reached).
+unsigned int* device_status_words();
+
 // Stores `message` as the calling thread's last error (what lfm25_last_error() returns) and returns `code`.
 int32_t report_error(int32_t code, const char* message);
 

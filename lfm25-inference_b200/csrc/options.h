@@ -16,6 +16,8 @@
 //                                                                        head) instead of through records and a merge kernel
 //   engine_graph         0 | 1                                 1         serving engine replays captured decode steps
 //   hybrid_attention     0 auto | 1 umma | 2 mma               0         kernel of the mixed-step attention
+//   stack_attention      0 auto | 1 scalar                     0         attention of layer-stack models: the tensor-core kernels
+//                                                                        where they take the shape, or always the scalar one
 //   fp8_gemm_path        0 auto | 1 stream | 2 umma | 3 generic | 4 rows   0   kernel of the E4M3 linear
 //   bf16_gemm            0 auto | 1 umma | 2 cublaslt | 3 rows  0         kernel of the BF16 linear
 //   decode_splits        0 auto | 1..8                         0         KV splits of the decode attention
@@ -40,6 +42,7 @@ enum Option : int {
     kOptSplitkClusterMerge,
     kOptEngineGraph,
     kOptHybridAttention,
+    kOptStackAttention,
     kOptFp8GemmPath,
     kOptBf16Gemm,
     kOptDecodeSplits,

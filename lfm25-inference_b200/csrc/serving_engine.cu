@@ -495,8 +495,12 @@ int32_t lfm25_engine_calibrate(lfm25_engine* self) {
     };
     const size_t batches[4] = {1, std::min<size_t>(8, self->config.max_slots), std::min<size_t>(32, self->config.max_slots),
                                self->config.max_slots};
+    std::vector<size_t> contexts;
     for (size_t context : {size_t(512), size_t(2048)}) {
-        if (context + 1 > self->pages_per_slot * kPage) continue;
+        if (context + 1 <= self->pages_per_slot * kPage) contexts.push_back(context);
+    }
+    if (contexts.empty()) contexts.push_back(self->pages_per_slot * kPage - 1);   // an engine for short sequences
+    for (size_t context : contexts) {
         const size_t pages = (context + 1 + kPage - 1) / kPage;
         size_t previous = 0;
         for (size_t sequences : batches) {

@@ -4,6 +4,7 @@
 #include <math.h>
 
 #include "launch.h"
+#include "options.h"
 #include "stack_attention.h"
 #include "stack_common.cuh"
 
@@ -282,8 +283,12 @@ scalar_attention_kernel(const PagedAttentionArgs<T> args) {
 }
 
 template <typename T>
-cudaError_t launch_scalar(cudaStream_t stream, const StackAttentionLaunch& launch) {
-    const PagedAttentionArgs<T> args = paged_attention_args<T>(launch);
+cudaError_t launch_scalar(cudaStream_t stream, const StackAttentionLaunch& launch, size_t first_token, size_t tokens) {
+    PagedAttentionArgs<T> args = paged_attention_args<T>(launch);
+    args.query += first_token * launch.shape.heads * launch.shape.dim;
+    args.request_slots += first_token;
+    args.positions += first_token;
+    args.out += first_token * launch.out_pitch;
     const size_t group = launch.shape.heads / launch.shape.kv_heads;
     const size_t shared = group * (launch.shape.dim + kScalarThreads + launch.shape.vdim + 3) * sizeof(float);
     if (shared > 227 * 1024 - 2048) {
@@ -295,9 +300,8 @@ cudaError_t launch_scalar(cudaStream_t stream, const StackAttentionLaunch& launc
                                                         static_cast<int>(shared));
         if (status != cudaSuccess) return status;
     }
-    return launch_kernel(scalar_attention_kernel<T>,
-                         static_cast<unsigned int>(launch.segments.num_tokens * launch.shape.kv_heads), kScalarThreads,
-                         shared, stream, 1, args);
+    return launch_kernel(scalar_attention_kernel<T>, static_cast<unsigned int>(tokens * launch.shape.kv_heads),
+                         kScalarThreads, shared, stream, 1, args);
 }
 
 }  // namespace
@@ -308,10 +312,29 @@ cudaError_t launch_projection_norm_rope(cudaStream_t stream, const ProjectionNor
 }
 
 cudaError_t launch_stack_attention(cudaStream_t stream, const StackAttentionLaunch& launch) {
+    const size_t tokens = launch.segments.num_tokens;
     if (launch.type == Activation::kF32) {
-        return launch_scalar<float>(stream, launch);
+        return launch_scalar<float>(stream, launch, 0, tokens);
     }
-    return launch_scalar<__nv_bfloat16>(stream, launch);
+    const bool scalar = option(kOptStackAttention) != 0;
+    if (launch.decode_tokens > 0) {
+        const cudaError_t status = !scalar && stack_attention_decode_supports(launch)
+                                       ? launch_stack_attention_decode(stream, launch)
+                                       : launch_scalar<__nv_bfloat16>(stream, launch, 0, launch.decode_tokens);
+        if (status != cudaSuccess) return status;
+    }
+    if (launch.decode_tokens == tokens) {
+        return cudaSuccess;
+    }
+    if (!scalar && stack_attention_umma_supports(launch)) {
+        // segment offsets are absolute token indices, so the remaining segments are simply a later start
+        StackAttentionLaunch prompts = launch;
+        prompts.segments.offsets += launch.decode_tokens;
+        prompts.segments.slots += launch.decode_tokens;
+        prompts.segments.num_segments -= launch.decode_tokens;
+        return launch_stack_attention_umma(stream, prompts);
+    }
+    return launch_scalar<__nv_bfloat16>(stream, launch, launch.decode_tokens, tokens - launch.decode_tokens);
 }
 
 }  // namespace lfm25

@@ -1,6 +1,8 @@
 // Shared by the attention kernels of the layer stack: their argument block and the addressing of the paged cache.
 #pragma once
 
+#include <cuda.h>
+
 #include "common.cuh"
 #include "stack_kernels.h"
 
@@ -62,5 +64,19 @@ __device__ __forceinline__ int64_t cache_row(const PagedAttentionArgs<T>& args, 
     }
     return static_cast<int64_t>((page * args.shape.kv_heads + kv_head) * kPageSize + position % kPageSize);
 }
+
+// Tensor map of the key (value) cache: rows of one head's vector, boxes of 64 dimensions x one page, 128-byte swizzle;
+// dimensions beyond the head's size read as zero.
+bool make_page_map(CUtensorMap* map, const StackAttentionLaunch& launch, bool value);
+// what both tensor-core kernels need of a launch: bf16, 16-byte rows, a positive scale
+bool paged_copies_possible(const StackAttentionLaunch& launch);
+
+bool stack_attention_umma_supports(const StackAttentionLaunch& launch);
+cudaError_t launch_stack_attention_umma(cudaStream_t stream, const StackAttentionLaunch& launch);
+
+// The first decode_tokens tokens (every one a segment of its own).
+uint32_t stack_attention_splits(const StackAttentionShape& shape, size_t tokens, size_t context);
+bool stack_attention_decode_supports(const StackAttentionLaunch& launch);
+cudaError_t launch_stack_attention_decode(cudaStream_t stream, const StackAttentionLaunch& launch);
 
 }  // namespace lfm25

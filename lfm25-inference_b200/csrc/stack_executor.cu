@@ -134,7 +134,7 @@ struct Step {
     lfm25::StackSegments segments;
     const uint32_t* output_rows;   // nullptr: every token, in order
     size_t num_outputs;
-    size_t max_context;
+    size_t decode_tokens, decode_context;   // leading single-token segments, longest context among them
     bool advance;
 };
 
@@ -206,7 +206,9 @@ int32_t enqueue(lfm25_stack_executor* self, const Step& step) {
             attention.request_slots = step.request_slots;
             attention.positions = step.positions;
             attention.segments = step.segments;
-            attention.max_context = step.max_context;
+            attention.decode_tokens = step.decode_tokens;
+            attention.decode_context = step.decode_context;
+            attention.status = lfm25::device_status_words();
             attention.out = self->joined;
             attention.out_pitch = layer.output.k;
             STACK_CUDA(lfm25::launch_stack_attention(stream, attention), "attention launch failed");
@@ -326,7 +328,11 @@ int32_t decode_step(const lfm25_stack_executor* self, const lfm25_decode_batch* 
     step->segments = {nullptr, batch->request_slots, batch->num_tokens, batch->num_tokens, self->model->num_request_slots};
     step->output_rows = nullptr;
     step->num_outputs = batch->num_tokens;
-    step->max_context = batch->max_context_tokens;
+    step->decode_tokens = batch->num_tokens;
+    // rounded up to a power of two: the context decides how the decode attention splits the keys, and a captured step
+    // serves every context of its class
+    step->decode_context = 1;
+    while (step->decode_context < batch->max_context_tokens) step->decode_context *= 2;
     step->advance = advance;
     return LFM25_OK;
 }
@@ -422,7 +428,7 @@ int32_t lfm25_stack_executor_step_graph(lfm25_stack_executor* self, const lfm25_
     STACK_TRY(decode_step(self, batch, advance != 0, &step));
     lfm25::StepKey key;
     key.num_tokens = batch->num_tokens;
-    key.splits = 0;
+    key.splits = step.decode_context;
     key.flags = advance != 0 ? 1u : 0u;
     key.signature = signature(self, batch);
     return self->graphs.run(key, self->blaslt->stream, [&]() -> int32_t { return enqueue(self, step); });
@@ -434,7 +440,8 @@ int32_t lfm25_stack_executor_forward_ragged(lfm25_stack_executor* self, const lf
         return lfm25::report_error(LFM25_ERR_NULL_POINTER, "stack executor received a null argument");
     }
     if (batch->num_tokens == 0 || batch->num_tokens > self->maximum_tokens || num_output_rows > self->maximum_rows ||
-        batch->num_segments == 0 || batch->num_segments > batch->num_tokens) {
+        batch->num_segments == 0 || batch->num_segments > batch->num_tokens ||
+        batch->num_decode_segments > batch->num_segments) {
         return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "ragged step exceeds the stack executor's workspace");
     }
     if (!batch->token_ids || !batch->positions || !batch->request_slots || !batch->physical_slots ||
@@ -454,7 +461,8 @@ int32_t lfm25_stack_executor_forward_ragged(lfm25_stack_executor* self, const lf
                      self->model->num_request_slots};
     step.output_rows = batch->output_rows;
     step.num_outputs = num_output_rows;
-    step.max_context = batch->max_decode_context_tokens;
+    step.decode_tokens = batch->num_decode_segments;
+    step.decode_context = batch->max_decode_context_tokens;
     step.advance = false;
     return enqueue(self, step);
 }

@@ -120,7 +120,11 @@ struct StackAttentionLaunch {
     const uint32_t* request_slots; // [T]
     const uint32_t* positions;     // [T]
     StackSegments segments;
-    size_t max_context;            // longest context of the step, for the split of long key ranges
+    // The first decode_tokens tokens are segments of one token; decode_context is the longest context among them (what
+    // their key range is split by).
+    size_t decode_tokens;
+    size_t decode_context;
+    unsigned int* status;          // device status words of the bounded waits
     void* out;                     // activations, rows out_pitch apart, heads * vdim columns
     size_t out_pitch;
 };

@@ -2,6 +2,8 @@
 // rows, the polynomial activation, and greedy sampling.
 #include <math.h>
 
+#include <algorithm>
+
 #include "launch.h"
 #include "stack_common.cuh"
 
@@ -58,12 +60,15 @@ __device__ __forceinline__ void residual_values(const ResidualNormConvArgs& args
 // first tokens of the segment, the record.  Only the segment's first tile touches the record: it reads it for its own
 // first rows and replaces it afterwards, so no other CTA depends on the order.
 // GROUP threads share a row: the whole CTA when a tile is one row (decode), one warp otherwise.
-template <typename T, int VEC, int GROUP>
+// HELD: a row fits the registers of its threads (8 vectors each), so that it is read once.
+// TAPS: number of taps known at compile time (0 = any), whose weights and window then stay in registers.
+template <typename T, int VEC, int GROUP, bool HELD, int TAPS>
 __global__ void __launch_bounds__(kThreads)
 residual_norm_conv_kernel(const ResidualNormConvArgs args, const T* __restrict__ update, T* __restrict__ mixed_out,
                           T* __restrict__ ff_out) {
     pdl_launch_dependents();
     pdl_wait();
+    constexpr int kHeld = HELD ? (GROUP == 32 ? 8 : 1) : 1;
     extern __shared__ __align__(16) unsigned char shared_raw[];
     __shared__ float scratch[kThreads / 32];
     T* rows = reinterpret_cast<T*>(shared_raw);      // [taps - 1 + tile_rows][width]
@@ -102,29 +107,50 @@ residual_norm_conv_kernel(const ResidualNormConvArgs args, const T* __restrict__
             embedding_row = id < args.vocab ? args.embedding + id * width : nullptr;
         }
         float sum = 0.0f;
-        for (size_t channel = lane * VEC; channel < width; channel += GROUP * VEC) {
-            float value[VEC];
+        float held[kHeld][VEC];           // the row between the two passes, when it fits
+        auto accumulate = [&](size_t channel, float (&value)[VEC]) {
             residual_values<T, VEC>(args, update, embedding_row, token, channel, value);
 #pragma unroll
             for (int i = 0; i < VEC; ++i) sum = fmaf(value[i], value[i], sum);
-            if (own) {
-                store_values<VEC>(args.residual_out + static_cast<size_t>(token) * width + channel, value);
-            }
-        }
-        sum = GROUP == 32 ? warp_sum(sum) : block_sum(sum, scratch);
-        const float scale = inverse_rms(sum, width, args.eps);
-        for (size_t channel = lane * VEC; channel < width; channel += GROUP * VEC) {
-            float value[VEC], weight[VEC], result[VEC];
-            residual_values<T, VEC>(args, update, embedding_row, token, channel, value);
+        };
+        auto emit = [&](size_t channel, const float (&value)[VEC], float scale) {
+            float weight[VEC], result[VEC];
             load_values<VEC>(args.mixer_norm + channel, weight);
 #pragma unroll
             for (int i = 0; i < VEC; ++i) result[i] = value[i] * scale * weight[i];
             store_values<VEC>(rows + index * width + channel, result);
-            if (own && args.ff_norm != nullptr) {
+            if (!own) {
+                return;
+            }
+            store_values<VEC>(args.residual_out + static_cast<size_t>(token) * width + channel, value);
+            if (args.ff_norm != nullptr) {
                 load_values<VEC>(args.ff_norm + channel, weight);
 #pragma unroll
                 for (int i = 0; i < VEC; ++i) result[i] = value[i] * scale * weight[i];
                 store_values<VEC>(ff_out + static_cast<size_t>(token) * width + channel, result);
+            }
+        };
+        if constexpr (HELD) {
+#pragma unroll
+            for (int step = 0; step < kHeld; ++step) {
+                const size_t channel = (step * GROUP + lane) * VEC;
+                if (channel < width) accumulate(channel, held[step]);
+            }
+        } else {
+            for (size_t channel = lane * VEC; channel < width; channel += GROUP * VEC) accumulate(channel, held[0]);
+        }
+        sum = GROUP == 32 ? warp_sum(sum) : block_sum(sum, scratch);
+        const float scale = inverse_rms(sum, width, args.eps);
+        if constexpr (HELD) {
+#pragma unroll
+            for (int step = 0; step < kHeld; ++step) {
+                const size_t channel = (step * GROUP + lane) * VEC;
+                if (channel < width) emit(channel, held[step], scale);
+            }
+        } else {
+            for (size_t channel = lane * VEC; channel < width; channel += GROUP * VEC) {
+                residual_values<T, VEC>(args, update, embedding_row, token, channel, held[0]);
+                emit(channel, held[0], scale);
             }
         }
     }
@@ -133,26 +159,55 @@ residual_norm_conv_kernel(const ResidualNormConvArgs args, const T* __restrict__
     T* record = reinterpret_cast<T*>(static_cast<unsigned char*>(args.record.base) + slot * args.record.stride +
                                      args.record.offset);
     for (size_t channel = threadIdx.x * VEC; channel < width; channel += kThreads * VEC) {
-        for (uint32_t row = 0; row < tile.count; ++row) {
+        // the input `back` tokens before row `row` of the tile: in shared memory, or in the record (whose last row is
+        // the token before the segment)
+        auto load_input = [&](uint32_t row, uint32_t back, float (&value)[VEC]) {
             const uint32_t offset = tile.first - tile.begin + row;     // of the token in its segment
-            float sum[VEC], value[VEC], tap[VEC];
-#pragma unroll
-            for (int i = 0; i < VEC; ++i) sum[i] = 0.0f;
-            for (uint32_t j = 0; j < args.taps; ++j) {
-                const uint32_t back = history - j;
-                if (back > offset) {      // before this segment: the record, whose last row is the token before it
-                    load_values<VEC>(record + (history - (back - offset)) * width + channel, value);
-                } else {
-                    load_values<VEC>(rows + (history + row - back) * width + channel, value);
-                }
-                load_values<VEC>(args.conv + j * width + channel, tap);
-#pragma unroll
-                for (int i = 0; i < VEC; ++i) sum[i] = fmaf(tap[i], value[i], sum[i]);
+            if (back > offset) {
+                load_values<VEC>(record + (history - (back - offset)) * width + channel, value);
+            } else {
+                load_values<VEC>(rows + (history + row - back) * width + channel, value);
             }
-            load_values<VEC>(rows + (history + row) * width + channel, value);
+        };
+        if constexpr (TAPS > 0) {
+            float tap[TAPS][VEC], window[TAPS][VEC];
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) value[i] += sum[i];
-            store_values<VEC>(mixed_out + static_cast<size_t>(tile.first + row) * width + channel, value);
+            for (int j = 0; j < TAPS; ++j) load_values<VEC>(args.conv + j * width + channel, tap[j]);
+#pragma unroll
+            for (int j = 1; j < TAPS; ++j) load_input(0, TAPS - j, window[j]);
+            for (uint32_t row = 0; row < tile.count; ++row) {
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j) {
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) window[j][i] = window[j + 1][i];
+                }
+                load_values<VEC>(rows + (history + row) * width + channel, window[TAPS - 1]);
+                float sum[VEC];
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) {
+                    sum[i] = 0.0f;
+#pragma unroll
+                    for (int j = 0; j < TAPS; ++j) sum[i] = fmaf(tap[j][i], window[j][i], sum[i]);
+                    sum[i] += window[TAPS - 1][i];
+                }
+                store_values<VEC>(mixed_out + static_cast<size_t>(tile.first + row) * width + channel, sum);
+            }
+        } else {
+            for (uint32_t row = 0; row < tile.count; ++row) {
+                float sum[VEC], value[VEC], tap[VEC];
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) sum[i] = 0.0f;
+                for (uint32_t j = 0; j < args.taps; ++j) {
+                    load_input(row, history - j, value);
+                    load_values<VEC>(args.conv + j * width + channel, tap);
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) sum[i] = fmaf(tap[i], value[i], sum[i]);
+                }
+                load_values<VEC>(rows + (history + row) * width + channel, value);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) value[i] += sum[i];
+                store_values<VEC>(mixed_out + static_cast<size_t>(tile.first + row) * width + channel, value);
+            }
         }
         if (first_tile) {
             // the same thread has read this channel's history above; ascending order only reads rows not yet written
@@ -402,11 +457,12 @@ cudaError_t launch_rnc(cudaStream_t stream, const ResidualNormConvLaunch& launch
     const bool single = launch.segments.offsets == nullptr;
     const size_t history = launch.taps - 1;
     const size_t row_bytes = launch.width * sizeof(T);
-    // rows per tile: 8 where the rows of a tile and its history fit, never fewer than the history
+    // rows per tile: 13 where they and their history fit half of an SM's shared memory (with three rows of history that
+    // is two per warp), never fewer than the history
     size_t rows = 1;
     if (!single) {
-        rows = history > 8 ? history : 8;
-        while (rows > 1 && rows > history && (rows + history) * row_bytes > kMaxSharedBytes / 2) --rows;
+        rows = history > 13 ? history : 16 - std::min<size_t>(history, 3);
+        while (rows > 1 && rows > history && (rows + history) * row_bytes > kMaxSharedBytes / 2 - 1024) --rows;
     }
     const size_t shared = (rows + history) * row_bytes;
     if (shared > kMaxSharedBytes) {
@@ -419,9 +475,16 @@ cudaError_t launch_rnc(cudaStream_t stream, const ResidualNormConvLaunch& launch
                         aligned_to(launch.residual_out, 16) && aligned_to(launch.mixed_out, 16) &&
                         aligned_to(launch.ff_out, 16) && aligned_to(launch.record.base, 16) &&
                         launch.record.stride % 16 == 0 && launch.record.offset % 16 == 0;
-    void (*kernel)(const ResidualNormConvArgs, const T*, T*, T*) =
-        vector ? (single ? residual_norm_conv_kernel<T, 8, 256> : residual_norm_conv_kernel<T, 8, 32>)
-               : (single ? residual_norm_conv_kernel<T, 1, 256> : residual_norm_conv_kernel<T, 1, 32>);
+    void (*kernel)(const ResidualNormConvArgs, const T*, T*, T*) = nullptr;
+    if (!vector) {
+        kernel = single ? residual_norm_conv_kernel<T, 1, 256, false, 0> : residual_norm_conv_kernel<T, 1, 32, false, 0>;
+    } else if (launch.width > 2048) {
+        kernel = single ? residual_norm_conv_kernel<T, 8, 256, false, 0> : residual_norm_conv_kernel<T, 8, 32, false, 0>;
+    } else if (launch.taps == 4) {
+        kernel = single ? residual_norm_conv_kernel<T, 8, 256, true, 4> : residual_norm_conv_kernel<T, 8, 32, true, 4>;
+    } else {
+        kernel = single ? residual_norm_conv_kernel<T, 8, 256, true, 0> : residual_norm_conv_kernel<T, 8, 32, true, 0>;
+    }
     if (shared > 48 * 1024) {
         const cudaError_t status = cudaFuncSetAttribute(reinterpret_cast<const void*>(kernel),
                                                         cudaFuncAttributeMaxDynamicSharedMemorySize,
