@@ -44,6 +44,11 @@ __device__ __forceinline__ Pair fma_pair(Pair a, Pair b, Pair c) {
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(out) : "l"(a), "l"(b), "l"(c));
     return out;
 }
+__device__ __forceinline__ Pair add_pair(Pair a, Pair b) {
+    Pair out;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(out) : "l"(a), "l"(b));
+    return out;
+}
 __device__ __forceinline__ Pair mul_pair(Pair a, Pair b) {
     Pair out;
     asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(out) : "l"(a), "l"(b));
@@ -551,25 +556,29 @@ __device__ __forceinline__ void named_barrier(uint32_t id, uint32_t threads) {
     asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory");
 }
 
+// The prompt kernel's decays and rates: the fast f32 exponential and division, a few units in the last place from the
+// correctly rounded ones.
+__device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
+__device__ __forceinline__ float fast_tanh(float z) { return 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * z)); }
+
 constexpr uint32_t kPromptTokens = 16;       // tokens per tile = rows of one MMA tile
-constexpr uint32_t kHelpers = 128;           // threads that prepare and finish
 constexpr uint32_t kRawStages = 4;           // being finished, in the recurrence, being prepared, arriving
 constexpr uint32_t kPromptMaxRank = 256;
 
 template <uint32_t DP>
 struct PromptLayout {
-    uint32_t rank_pad;        // multiple of 16
+    uint32_t rank_pad;        // multiple of 32
     uint32_t z_stride;        // bf16 elements between rows of z / W2 in shared memory: 16-byte rows, no bank conflicts
     uint32_t raw_row;         // bf16 elements per token: r | k | v | g | a (DP each) | z
     size_t raw, vectors, produced, tanh_parts, w2, constants, scale, total;
     __host__ __device__ explicit PromptLayout(uint32_t rank) {
-        rank_pad = (rank + 15) / 16 * 16;
+        rank_pad = (rank + 31) / 32 * 32;
         z_stride = rank_pad + 8;
         raw_row = 5 * DP + rank_pad;
         size_t at = 0;
         raw = at;
         at += static_cast<size_t>(kRawStages) * kPromptTokens * raw_row * 2;
-        vectors = at;                                             // [2][tokens][2][DP] f32: w, removal / |k|
+        vectors = at;                                             // [2][tokens][2][DP] f32: w, removal / |k|^2
         at += 2 * kPromptTokens * 2 * DP * 4;
         produced = at;                                            // [2][tokens][DP] f32
         at += 2 * kPromptTokens * DP * 4;
@@ -579,7 +588,7 @@ struct PromptLayout {
         at += static_cast<size_t>(DP) * z_stride * 2;
         constants = at;                                           // [3][DP] f32: w0, removal bias, norm weight
         at += 3 * DP * 4;
-        scale = at;                                               // [2][tokens] f32: 1 / |k|
+        scale = at;                                               // [2][tokens] f32: 1 / |k|^2
         at += 2 * kPromptTokens * 4;
         total = at;
     }
@@ -593,12 +602,17 @@ __device__ __forceinline__ uint32_t interleaved(uint32_t row) {
     return row % kRows / 4 * 32 + row / kRows * 4 + row % 4;
 }
 
-// 2 * DP threads run the recurrence: eight per group of four value columns, DP / 8 consecutive key channels each.
-template <uint32_t DP>
-__global__ void __launch_bounds__(2 * DP + kHelpers)
+// Eight threads per group of COLUMNS value columns run the recurrence, DP / 8 consecutive key channels each; HELPERS
+// threads prepare and finish.
+template <uint32_t DP, uint32_t COLUMNS, uint32_t HELPERS>
+__global__ void __launch_bounds__(DP / COLUMNS * 8 + HELPERS)
 delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
     constexpr uint32_t kRows = DP / 8;
-    constexpr uint32_t kScanThreads = 2 * DP;
+    constexpr uint32_t kScanThreads = DP / COLUMNS * 8;
+    constexpr uint32_t kHelpers = HELPERS;
+    constexpr uint32_t kHelperWarps = kHelpers / 32;
+    constexpr uint32_t kTokensPerHelper = kPromptTokens / kHelperWarps;   // tokens per helper warp
+    static_assert(COLUMNS == 2 || COLUMNS == 4, "columns per thread");
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ __align__(16) unsigned char prompt_shared[];
@@ -651,26 +665,39 @@ delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
     const uint32_t helper_warp = helper / 32;
     const uint32_t warp_lane = threadIdx.x % 32;
 
+    // the 16-byte pieces of a token's row that this lane copies: offsets in the row and in the stage
+    constexpr uint32_t kPieces = (5 * DP / 8 + kPromptMaxRank / 8 + 31) / 32;
+    const uint32_t per_vector = dim / 8;
+    const uint32_t pieces = 5 * per_vector + (args.rank + 7) / 8;
+    auto piece_offsets = [&](uint32_t piece, uint32_t& source, uint32_t& target) {
+        if (piece < 5 * per_vector) {
+            const uint32_t vector = piece / per_vector;
+            const uint32_t chunk = piece - vector * per_vector;
+            source = static_cast<uint32_t>(vector * width + head_base) + chunk * 8;
+            target = vector * DP + chunk * 8;
+        } else {
+            const uint32_t chunk = piece - 5 * per_vector;
+            source = static_cast<uint32_t>(5 * width) + chunk * 8;
+            target = 5 * DP + chunk * 8;
+        }
+    };
+    uint32_t first_source = 0, first_target = 0, second_source = 0, second_target = 0;
+    piece_offsets(warp_lane, first_source, first_target);
+    piece_offsets(warp_lane + 32, second_source, second_target);
     auto load_tile = [&](uint32_t tile) {             // helpers only; always one group per call
-        if (tile < tiles) {
-            const uint32_t first = begin + tile * kPromptTokens;
-            const uint32_t tokens = min(kPromptTokens, end - first);
-            const uint32_t per_vector = dim / 8;
-            const uint32_t z_copies = (args.rank + 7) / 8;
-            const uint32_t per_token = 5 * per_vector + z_copies;
-            __nv_bfloat16* stage = raw + tile % kRawStages * kPromptTokens * layout.raw_row;
-            for (uint32_t item = helper; item < tokens * per_token; item += kHelpers) {
-                const uint32_t t = item / per_token;
-                const uint32_t part = item - t * per_token;
+        const uint32_t first = begin + tile * kPromptTokens;
+#pragma unroll
+        for (uint32_t i = 0; i < kTokensPerHelper; ++i) {
+            const uint32_t t = helper_warp * kTokensPerHelper + i;
+            if (tile < tiles && first + t < end) {
                 const __nv_bfloat16* source = args.projected + static_cast<size_t>(first + t) * args.pitch;
-                __nv_bfloat16* target = stage + t * layout.raw_row;
-                if (part < 5 * per_vector) {
-                    const uint32_t vector = part / per_vector;
-                    const uint32_t chunk = part - vector * per_vector;
-                    copy_async_16(target + vector * DP + chunk * 8, source + vector * width + head_base + chunk * 8);
-                } else {
-                    const uint32_t chunk = part - 5 * per_vector;
-                    copy_async_16(target + 5 * DP + chunk * 8, source + 5 * width + chunk * 8);
+                __nv_bfloat16* target = raw + (tile % kRawStages * kPromptTokens + t) * layout.raw_row;
+                if (warp_lane < pieces) copy_async_16(target + first_target, source + first_source);
+                if (warp_lane + 32 < pieces) copy_async_16(target + second_target, source + second_source);
+                for (uint32_t piece = warp_lane + 64; kPieces > 2 && piece < pieces; piece += 32) {
+                    uint32_t from, to;
+                    piece_offsets(piece, from, to);
+                    copy_async_16(target + to, source + from);
                 }
             }
         }
@@ -681,67 +708,90 @@ delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
         const __nv_bfloat16* stage = raw + tile % kRawStages * kPromptTokens * layout.raw_row;
         float* target = vectors + tile % 2 * kPromptTokens * 2 * DP;
         float* unit = scale + tile % 2 * kPromptTokens;
+        float squares[kTokensPerHelper];
 #pragma unroll
-        for (uint32_t i = 0; i < kPromptTokens / 4; ++i) {
-            const uint32_t t = helper_warp * (kPromptTokens / 4) + i;
-            const __nv_bfloat16* k = stage + t * layout.raw_row + DP;
-            float sum = 0.0f;
+        for (uint32_t i = 0; i < kTokensPerHelper; ++i) {
+            const __nv_bfloat16* row = stage + (helper_warp * kTokensPerHelper + i) * layout.raw_row;
+            squares[i] = 0.0f;
 #pragma unroll
             for (uint32_t part = 0; part < DP / 64; ++part) {
                 const float2 both =
-                    __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k + part * 64 + warp_lane * 2));
-                sum = fmaf(both.x, both.x, fmaf(both.y, both.y, sum));
+                    __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + DP + part * 64 + warp_lane * 2));
+                squares[i] = fmaf(both.x, both.x, fmaf(both.y, both.y, squares[i]));
             }
-            sum = warp_sum(sum);
-            if (warp_lane == 0) unit[t] = 1.0f / sqrtf(sum + kUnitEps);
         }
-        for (uint32_t item = helper; item < kPromptTokens * layout.rank_pad; item += kHelpers) {
-            const uint32_t t = item / layout.rank_pad;
-            const uint32_t z = item - t * layout.rank_pad;
-            // columns between rank and its multiple of eight arrive with the copy and belong to nobody: W2 is zero there
-            const float value = z < args.rank ? tanhf(__bfloat162float(stage[t * layout.raw_row + 5 * DP + z])) : 0.0f;
-            const __nv_bfloat16 high = __float2bfloat16_rn(value);
-            tanh_parts[t * layout.z_stride + z] = high;
-            tanh_parts[(kPromptTokens + t) * layout.z_stride + z] = __float2bfloat16_rn(value - __bfloat162float(high));
+        for (uint32_t z = warp_lane * 2; z < layout.rank_pad; z += 64) {
+#pragma unroll
+            for (uint32_t i = 0; i < kTokensPerHelper; ++i) {
+                const uint32_t t = helper_warp * kTokensPerHelper + i;
+                const float2 both = __bfloat1622float2(
+                    *reinterpret_cast<const __nv_bfloat162*>(stage + t * layout.raw_row + 5 * DP + z));
+                // columns between rank and the end of its last copy belong to nobody
+                const float a = z < args.rank ? fast_tanh(both.x) : 0.0f;
+                const float b = z + 1 < args.rank ? fast_tanh(both.y) : 0.0f;
+                const __nv_bfloat162 high = __floats2bfloat162_rn(a, b);
+                const float2 rounded = __bfloat1622float2(high);
+                *reinterpret_cast<__nv_bfloat162*>(tanh_parts + t * layout.z_stride + z) = high;
+                *reinterpret_cast<__nv_bfloat162*>(tanh_parts + (kPromptTokens + t) * layout.z_stride + z) =
+                    __floats2bfloat162_rn(a - rounded.x, b - rounded.y);
+            }
+        }
+#pragma unroll
+        for (uint32_t i = 0; i < kTokensPerHelper; ++i) squares[i] = warp_sum(squares[i]);
+        if (warp_lane == 0) {
+#pragma unroll
+            for (uint32_t i = 0; i < kTokensPerHelper; ++i) {
+                unit[helper_warp * kTokensPerHelper + i] = 1.0f / (squares[i] + kUnitEps);
+            }
         }
         named_barrier(1, kHelpers);
-        // decay logits of 16 tokens x (DP / 4) channels per warp: tanh(z) W2^T with tanh(z) as a sum of two bf16 values
-        constexpr uint32_t kTilesPerWarp = DP / 32;
-        float logits[kTilesPerWarp][4] = {};
-        const uint32_t z_row = warp_lane % 16, z_part = warp_lane / 16 * 8;
-        for (uint32_t step = 0; step < layout.rank_pad; step += 16) {
-            uint32_t high[4], low[4];
-            ldmatrix_x4(smem_u32(tanh_parts + z_row * layout.z_stride + step + z_part), high[0], high[1], high[2], high[3]);
-            ldmatrix_x4(smem_u32(tanh_parts + (kPromptTokens + z_row) * layout.z_stride + step + z_part), low[0], low[1],
-                        low[2], low[3]);
+        // decay logits of 16 tokens x 8 channels at a time: tanh(z) W2^T with tanh(z) as a sum of two bf16 values
 #pragma unroll
-            for (uint32_t n = 0; n < kTilesPerWarp; n += 2) {
-                const uint32_t channel = helper_warp * (DP / 4) + n * 8 + warp_lane / 16 * 8 + warp_lane % 8;
+        for (uint32_t n = 0; n < DP / 8 / kHelperWarps; ++n) {
+            const uint32_t channel0 = (n * kHelperWarps + helper_warp) * 8;
+            float logits[4] = {};
+            const uint32_t z_row = warp_lane % 16, z_part = warp_lane / 16 * 8;
+            for (uint32_t step = 0; step < layout.rank_pad; step += 32) {
                 uint32_t b0, b1, b2, b3;
-                ldmatrix_x4(smem_u32(w2 + channel * layout.z_stride + step + warp_lane / 8 % 2 * 8), b0, b1, b2, b3);
-                mma_bf16_16816(logits[n], high[0], high[1], high[2], high[3], b0, b1);
-                mma_bf16_16816(logits[n], low[0], low[1], low[2], low[3], b0, b1);
-                mma_bf16_16816(logits[n + 1], high[0], high[1], high[2], high[3], b2, b3);
-                mma_bf16_16816(logits[n + 1], low[0], low[1], low[2], low[3], b2, b3);
-            }
-        }
+                ldmatrix_x4(smem_u32(w2 + (channel0 + warp_lane % 8) * layout.z_stride + step + warp_lane / 8 * 8), b0, b1,
+                            b2, b3);
 #pragma unroll
-        for (uint32_t n = 0; n < kTilesPerWarp; ++n) {
-            const uint32_t channel = helper_warp * (DP / 4) + n * 8 + warp_lane % 4 * 2;
+                for (uint32_t part = 0; part < 2; ++part) {
+                    uint32_t high[4], low[4];
+                    const __nv_bfloat16* source = tanh_parts + z_row * layout.z_stride + step + part * 16 + z_part;
+                    ldmatrix_x4(smem_u32(source), high[0], high[1], high[2], high[3]);
+                    ldmatrix_x4(smem_u32(source + kPromptTokens * layout.z_stride), low[0], low[1], low[2], low[3]);
+                    mma_bf16_16816(logits, high[0], high[1], high[2], high[3], part ? b2 : b0, part ? b3 : b1);
+                    mma_bf16_16816(logits, low[0], low[1], low[2], low[3], part ? b2 : b0, part ? b3 : b1);
+                }
+            }
+            const uint32_t channel = channel0 + warp_lane % 4 * 2;
+            const uint32_t t0 = warp_lane / 4;
+            const float2 base = *reinterpret_cast<const float2*>(constants + channel);
+            const float2 bias = *reinterpret_cast<const float2*>(constants + DP + channel);
+            float2 rate[2];
+            float factor[2];
 #pragma unroll
             for (uint32_t half = 0; half < 2; ++half) {
-                const uint32_t t = warp_lane / 4 + half * 8;
-                const float2 rate = __bfloat1622float2(
-                    *reinterpret_cast<const __nv_bfloat162*>(stage + t * layout.raw_row + 4 * DP + channel));
-                float2 w, removal;
-                w.x = expf(-kDecayScale * sigmoidf(logits[n][2 * half] + constants[channel]));
-                w.y = expf(-kDecayScale * sigmoidf(logits[n][2 * half + 1] + constants[channel + 1]));
-                // -(a * u) (u^T S) = -(a / |k|) * k * (u^T S): the recurrence multiplies by k anyway
-                removal.x = -sigmoidf(rate.x + constants[DP + channel]) * unit[t];
-                removal.y = -sigmoidf(rate.y + constants[DP + channel + 1]) * unit[t];
-                const uint32_t at = interleaved<DP>(channel);
-                *reinterpret_cast<float2*>(target + t * 2 * DP + at) = w;
-                *reinterpret_cast<float2*>(target + t * 2 * DP + DP + at) = removal;
+                rate[half] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(
+                    stage + (t0 + half * 8) * layout.raw_row + 4 * DP + channel));
+                factor[half] = unit[t0 + half * 8];
+            }
+            float2 w[2], removal[2];
+#pragma unroll
+            for (uint32_t half = 0; half < 2; ++half) {
+                w[half].x = __expf(-kDecayScale * fast_sigmoid(logits[2 * half] + base.x));
+                w[half].y = __expf(-kDecayScale * fast_sigmoid(logits[2 * half + 1] + base.y));
+                // -(a * u) (u^T S) = -(a / |k|^2) * k * (k^T S): the recurrence multiplies by k anyway
+                removal[half].x = -fast_sigmoid(rate[half].x + bias.x) * factor[half];
+                removal[half].y = -fast_sigmoid(rate[half].y + bias.y) * factor[half];
+            }
+            const uint32_t at = interleaved<DP>(channel);
+#pragma unroll
+            for (uint32_t half = 0; half < 2; ++half) {
+                float* row = target + (t0 + half * 8) * 2 * DP + at;
+                *reinterpret_cast<float2*>(row) = w[half];
+                *reinterpret_cast<float2*>(row + DP) = removal[half];
             }
         }
     };
@@ -750,27 +800,36 @@ delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
         const __nv_bfloat16* stage = raw + tile % kRawStages * kPromptTokens * layout.raw_row;
         const float* source = produced + tile % 2 * kPromptTokens * DP;
         const uint32_t first = begin + tile * kPromptTokens;
+        float2 value[kTokensPerHelper][DP / 64], gate[kTokensPerHelper][DP / 64];
+        float squares[kTokensPerHelper];
 #pragma unroll
-        for (uint32_t i = 0; i < kPromptTokens / 4; ++i) {
-            const uint32_t t = helper_warp * (kPromptTokens / 4) + i;
-            if (first + t >= end) break;
-            float2 value[DP / 64];
-            float sum = 0.0f;
-#pragma unroll
-            for (uint32_t part = 0; part < DP / 64; ++part) {
-                value[part] = *reinterpret_cast<const float2*>(source + t * DP + part * 64 + warp_lane * 2);
-                sum = fmaf(value[part].x, value[part].x, fmaf(value[part].y, value[part].y, sum));
-            }
-            const float factor = inverse_rms(warp_sum(sum), dim, args.eps);
+        for (uint32_t i = 0; i < kTokensPerHelper; ++i) {
+            const uint32_t t = helper_warp * kTokensPerHelper + i;
+            squares[i] = 0.0f;
 #pragma unroll
             for (uint32_t part = 0; part < DP / 64; ++part) {
                 const uint32_t channel = part * 64 + warp_lane * 2;
-                if (channel < dim) {
-                    const float2 gate = __bfloat1622float2(
-                        *reinterpret_cast<const __nv_bfloat162*>(stage + t * layout.raw_row + 3 * DP + channel));
-                    const float2 weight = *reinterpret_cast<const float2*>(constants + 2 * DP + channel);
-                    const uint32_t both = pack_bf16x2(value[part].x * factor * weight.x * sigmoidf(gate.x),
-                                                      value[part].y * factor * weight.y * sigmoidf(gate.y));
+                value[i][part] = *reinterpret_cast<const float2*>(source + t * DP + channel);
+                gate[i][part] = __bfloat1622float2(
+                    *reinterpret_cast<const __nv_bfloat162*>(stage + t * layout.raw_row + 3 * DP + channel));
+                squares[i] = fmaf(value[i][part].x, value[i][part].x,
+                                  fmaf(value[i][part].y, value[i][part].y, squares[i]));
+            }
+        }
+#pragma unroll
+        for (uint32_t i = 0; i < kTokensPerHelper; ++i) squares[i] = warp_sum(squares[i]);
+#pragma unroll
+        for (uint32_t i = 0; i < kTokensPerHelper; ++i) {
+            const uint32_t t = helper_warp * kTokensPerHelper + i;
+            const float factor = rsqrtf(squares[i] / static_cast<float>(dim) + args.eps);
+#pragma unroll
+            for (uint32_t part = 0; part < DP / 64; ++part) {
+                const uint32_t channel = part * 64 + warp_lane * 2;
+                const float2 weight = *reinterpret_cast<const float2*>(constants + 2 * DP + channel);
+                const uint32_t both =
+                    pack_bf16x2(value[i][part].x * factor * weight.x * fast_sigmoid(gate[i][part].x),
+                                value[i][part].y * factor * weight.y * fast_sigmoid(gate[i][part].y));
+                if (channel < dim && first + t < end) {
                     *reinterpret_cast<uint32_t*>(args.out + static_cast<size_t>(first + t) * args.out_pitch + head_base +
                                                  channel) = both;
                 }
@@ -778,13 +837,13 @@ delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
         }
     };
 
-    // ---- the state: columns 4 * group .. + 3, key channels lane * kRows .. + kRows - 1
+    // ---- the state: columns COLUMNS * group .. + COLUMNS - 1, key channels lane * kRows .. + kRows - 1
     const uint32_t lane = threadIdx.x % 8;
-    const uint32_t column0 = threadIdx.x / 8 * 4;
-    Pair state[4][kRows / 2];
+    const uint32_t column0 = threadIdx.x / 8 * COLUMNS;
+    Pair state[COLUMNS][kRows / 2];
     if (scanner) {
 #pragma unroll
-        for (uint32_t c = 0; c < 4; ++c) {
+        for (uint32_t c = 0; c < COLUMNS; ++c) {
 #pragma unroll
             for (uint32_t g = 0; g < kRows / 4; ++g) {
                 const uint32_t row = lane * kRows + g * 4;
@@ -810,18 +869,69 @@ delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
             const uint32_t tokens = min(kPromptTokens, end - begin - tile * kPromptTokens);
             const __nv_bfloat16* stage = raw + tile % kRawStages * kPromptTokens * layout.raw_row;
             const float* prepared = vectors + tile % 2 * kPromptTokens * 2 * DP;
-            const float* unit = scale + tile % 2 * kPromptTokens;
             float* target = produced + tile % 2 * kPromptTokens * DP;
-#pragma unroll 2
-            for (uint32_t t = 0; t < tokens; ++t) {
+            // software pipeline: a token's vectors are read one token ahead, and the sums over the eight threads of a
+            // column group run for o of the previous token beside those for u^T S of this one
+            struct Vectors {
+                uint4 k[kRows / 8], r[kRows / 8];
+                uint32_t v[COLUMNS / 2];
+            };
+            auto read = [&](uint32_t t) {
+                Vectors out;
                 const __nv_bfloat16* row = stage + t * layout.raw_row;
+#pragma unroll
+                for (uint32_t part = 0; part < kRows / 8; ++part) {
+                    out.k[part] = *reinterpret_cast<const uint4*>(row + DP + lane * kRows + part * 8);
+                    out.r[part] = *reinterpret_cast<const uint4*>(row + lane * kRows + part * 8);
+                }
+                if constexpr (COLUMNS == 4) {
+                    const uint2 both = *reinterpret_cast<const uint2*>(row + 2 * DP + column0);
+                    out.v[0] = both.x;
+                    out.v[1] = both.y;
+                } else {
+                    out.v[0] = *reinterpret_cast<const uint32_t*>(row + 2 * DP + column0);
+                }
+                return out;
+            };
+            Vectors next = read(0);
+            float result[COLUMNS] = {};
+            const bool upper1 = lane & 1, upper2 = lane & 2;
+            float* slot_of_lane = target + column0 + (COLUMNS == 4 ? (lane & 1) * 2 + (lane >> 1 & 1) : (lane & 1));
+            // column sums of o over the eight threads, each pair of threads keeping half of the columns
+            auto total_of = [&](const float (&share)[COLUMNS]) {
+                if constexpr (COLUMNS == 2) {
+                    float total = (upper1 ? share[1] : share[0]) +
+                                  __shfl_xor_sync(0xffffffffu, upper1 ? share[0] : share[1], 1);
+                    total += __shfl_xor_sync(0xffffffffu, total, 2);
+                    return total + __shfl_xor_sync(0xffffffffu, total, 4);
+                } else {
+                const float keep0 = upper1 ? share[2] : share[0], keep1 = upper1 ? share[3] : share[1];
+                const float give0 = upper1 ? share[0] : share[2], give1 = upper1 ? share[1] : share[3];
+                const float half0 = keep0 + __shfl_xor_sync(0xffffffffu, give0, 1);
+                const float half1 = keep1 + __shfl_xor_sync(0xffffffffu, give1, 1);
+                float total = (upper2 ? half1 : half0) + __shfl_xor_sync(0xffffffffu, upper2 ? half0 : half1, 2);
+                return total + __shfl_xor_sync(0xffffffffu, total, 4);
+                }
+            };
+            for (uint32_t t = 0; t < tokens; ++t) {
+                const Vectors now = next;
+                next = read(t + 1 < tokens ? t + 1 : t);
+                Pair w[kRows / 2], removal[kRows / 2];
+#pragma unroll
+                for (uint32_t g = 0; g < kRows / 4; ++g) {
+                    const float* token = prepared + t * 2 * DP + g * 32 + lane * 4;
+                    const ulonglong2 w_pair = *reinterpret_cast<const ulonglong2*>(token);
+                    const ulonglong2 removal_pair = *reinterpret_cast<const ulonglong2*>(token + DP);
+                    w[2 * g] = w_pair.x;
+                    w[2 * g + 1] = w_pair.y;
+                    removal[2 * g] = removal_pair.x;
+                    removal[2 * g + 1] = removal_pair.y;
+                }
                 Pair k[kRows / 2], r[kRows / 2];
 #pragma unroll
                 for (uint32_t part = 0; part < kRows / 8; ++part) {
-                    const uint4 k_raw = *reinterpret_cast<const uint4*>(row + DP + lane * kRows + part * 8);
-                    const uint4 r_raw = *reinterpret_cast<const uint4*>(row + lane * kRows + part * 8);
-                    const uint32_t k_words[4] = {k_raw.x, k_raw.y, k_raw.z, k_raw.w};
-                    const uint32_t r_words[4] = {r_raw.x, r_raw.y, r_raw.z, r_raw.w};
+                    const uint32_t k_words[4] = {now.k[part].x, now.k[part].y, now.k[part].z, now.k[part].w};
+                    const uint32_t r_words[4] = {now.r[part].x, now.r[part].y, now.r[part].z, now.r[part].w};
 #pragma unroll
                     for (uint32_t i = 0; i < 4; ++i) {       // bf16 -> f32 is a shift
                         k[part * 4 + i] = pair_of(__uint_as_float(k_words[i] << 16),
@@ -830,12 +940,14 @@ delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
                                                   __uint_as_float(r_words[i] & 0xffff0000u));
                     }
                 }
-                const uint2 v_raw = *reinterpret_cast<const uint2*>(row + 2 * DP + column0);
-                const float v[4] = {__uint_as_float(v_raw.x << 16), __uint_as_float(v_raw.x & 0xffff0000u),
-                                    __uint_as_float(v_raw.y << 16), __uint_as_float(v_raw.y & 0xffff0000u)};
-                float dot[4];
+                float v[COLUMNS], dot[COLUMNS];
 #pragma unroll
-                for (uint32_t c = 0; c < 4; ++c) {
+                for (uint32_t c = 0; c < COLUMNS; c += 2) {
+                    v[c] = __uint_as_float(now.v[c / 2] << 16);
+                    v[c + 1] = __uint_as_float(now.v[c / 2] & 0xffff0000u);
+                }
+#pragma unroll
+                for (uint32_t c = 0; c < COLUMNS; ++c) {
                     Pair even = mul_pair(k[0], state[c][0]);
                     Pair odd = mul_pair(k[1], state[c][1]);
 #pragma unroll
@@ -843,51 +955,41 @@ delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
                         even = fma_pair(k[i], state[c][i], even);
                         odd = fma_pair(k[i + 1], state[c][i + 1], odd);
                     }
-                    dot[c] = pair_sum(even) + pair_sum(odd);
+                    dot[c] = pair_sum(add_pair(even, odd));
                 }
 #pragma unroll
                 for (uint32_t delta = 1; delta < 8; delta <<= 1) {
 #pragma unroll
-                    for (uint32_t c = 0; c < 4; ++c) dot[c] += __shfl_xor_sync(0xffffffffu, dot[c], delta);
+                    for (uint32_t c = 0; c < COLUMNS; ++c) dot[c] += __shfl_xor_sync(0xffffffffu, dot[c], delta);
                 }
-                const float unit_scale = unit[t];
-                const float* token = prepared + t * 2 * DP;
-                Pair sums[4] = {0, 0, 0, 0};
-                Pair recalled[4], values[4];
+                const float before = total_of(result);
+                Pair sums[COLUMNS];
+                // w S does not depend on the sums above
 #pragma unroll
-                for (uint32_t c = 0; c < 4; ++c) {
-                    const float product = dot[c] * unit_scale;
-                    recalled[c] = pair_of(product, product);
-                    values[c] = pair_of(v[c], v[c]);
+                for (uint32_t c = 0; c < COLUMNS; ++c) {
+#pragma unroll
+                    for (uint32_t i = 0; i < kRows / 2; ++i) state[c][i] = mul_pair(w[i], state[c][i]);
                 }
 #pragma unroll
-                for (uint32_t g = 0; g < kRows / 4; ++g) {
-                    const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(token + g * 32 + lane * 4);
-                    const ulonglong2 removal = *reinterpret_cast<const ulonglong2*>(token + DP + g * 32 + lane * 4);
+                for (uint32_t c = 0; c < COLUMNS; ++c) {
+                    const Pair recalled = pair_of(dot[c], dot[c]);
+                    const Pair values = pair_of(v[c], v[c]);
+                    Pair even = 0, odd = 0;
 #pragma unroll
-                    for (uint32_t c = 0; c < 4; ++c) {
-                        // w S + k (v - (a / |k|) (u^T S))
-                        state[c][2 * g] = fma_pair(k[2 * g], fma_pair(removal.x, recalled[c], values[c]),
-                                                   mul_pair(w.x, state[c][2 * g]));
-                        state[c][2 * g + 1] = fma_pair(k[2 * g + 1], fma_pair(removal.y, recalled[c], values[c]),
-                                                       mul_pair(w.y, state[c][2 * g + 1]));
-                        sums[c] = fma_pair(r[2 * g], state[c][2 * g], sums[c]);
-                        sums[c] = fma_pair(r[2 * g + 1], state[c][2 * g + 1], sums[c]);
+                    for (uint32_t i = 0; i < kRows / 2; i += 2) {      // w S + k (v - (a / |k|^2) (k^T S))
+                        state[c][i] = fma_pair(k[i], fma_pair(removal[i], recalled, values), state[c][i]);
+                        state[c][i + 1] = fma_pair(k[i + 1], fma_pair(removal[i + 1], recalled, values), state[c][i + 1]);
+                        even = fma_pair(r[i], state[c][i], even);
+                        odd = fma_pair(r[i + 1], state[c][i + 1], odd);
                     }
+                    sums[c] = add_pair(even, odd);
                 }
-                // the four column sums over the eight threads, each pair of threads keeping half of the columns
-                float result[4];
 #pragma unroll
-                for (uint32_t c = 0; c < 4; ++c) result[c] = pair_sum(sums[c]);
-                const bool upper1 = lane & 1, upper2 = lane & 2;
-                const float keep0 = upper1 ? result[2] : result[0], keep1 = upper1 ? result[3] : result[1];
-                const float give0 = upper1 ? result[0] : result[2], give1 = upper1 ? result[1] : result[3];
-                const float half0 = keep0 + __shfl_xor_sync(0xffffffffu, give0, 1);
-                const float half1 = keep1 + __shfl_xor_sync(0xffffffffu, give1, 1);
-                float total = (upper2 ? half1 : half0) + __shfl_xor_sync(0xffffffffu, upper2 ? half0 : half1, 2);
-                total += __shfl_xor_sync(0xffffffffu, total, 4);
-                if (lane < 4) target[t * DP + column0 + (lane & 1) * 2 + (lane >> 1)] = total;
+                for (uint32_t c = 0; c < COLUMNS; ++c) result[c] = pair_sum(sums[c]);
+                if (lane < COLUMNS && t > 0) slot_of_lane[(t - 1) * DP] = before;
             }
+            const float last = total_of(result);
+            if (lane < COLUMNS) slot_of_lane[(tokens - 1) * DP] = last;
         } else {
             load_tile(tile + 2);
             if (tile > 0) finish_tile(tile - 1);
@@ -899,7 +1001,7 @@ delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
     }
     if (scanner) {
 #pragma unroll
-        for (uint32_t c = 0; c < 4; ++c) {
+        for (uint32_t c = 0; c < COLUMNS; ++c) {
 #pragma unroll
             for (uint32_t g = 0; g < kRows / 4; ++g) {
                 const uint32_t row = lane * kRows + g * 4;
@@ -926,16 +1028,16 @@ cudaError_t launch_decode(cudaStream_t stream, const DeltaArgs<T>& args) {
                          args);
 }
 
-template <uint32_t DP>
+template <uint32_t DP, uint32_t COLUMNS, uint32_t HELPERS>
 cudaError_t launch_prompt(cudaStream_t stream, const DeltaArgs<__nv_bfloat16>& args) {
     const size_t shared = PromptLayout<DP>(args.rank).total;
-    const auto kernel = delta_prompt_kernel<DP>;
+    const auto kernel = delta_prompt_kernel<DP, COLUMNS, HELPERS>;
     const cudaError_t status = cudaFuncSetAttribute(reinterpret_cast<const void*>(kernel),
                                                     cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                     static_cast<int>(shared));
     if (status != cudaSuccess) return status;
     return launch_kernel(kernel, static_cast<unsigned int>(args.segments.num_segments * args.heads),
-                         2 * DP + kHelpers, shared, stream, 1, args);
+                         DP / COLUMNS * 8 + HELPERS, shared, stream, 1, args);
 }
 
 bool prompt_kernel_takes(const DeltaArgs<__nv_bfloat16>& args) {
@@ -1003,7 +1105,7 @@ cudaError_t launch_typed(cudaStream_t stream, const DeltaRuleLaunch& launch) {
     }
     if constexpr (std::is_same<T, __nv_bfloat16>::value) {
         if (launch.segments.offsets != nullptr && prompt_kernel_takes(args)) {
-            return launch.dim <= 64 ? launch_prompt<64>(stream, args) : launch_prompt<128>(stream, args);
+            return launch.dim <= 64 ? launch_prompt<64, 4, 128>(stream, args) : launch_prompt<128, 4, 128>(stream, args);
         }
     }
     if (launch.dim <= 32) return launch_sized<T, 32, 4, 32>(stream, args);

@@ -11,6 +11,7 @@ left; a step in which places are wanted leaves their logits in DIR/<step>.f32 (l
 from __future__ import annotations
 
 import argparse
+import itertools
 import json
 import os
 import sys
@@ -34,14 +35,17 @@ def build_engine(model_dir: str, dtype: str, max_tokens: int, device):
 
 
 def replay(engine, vocab: int, lines, out_dir: str, answer=sys.stdout) -> None:
-    numbers = {}                       # request name -> the engine's request id
+    numbers = {}                       # name of a live request -> the engine's request id, never used twice
+    fresh = itertools.count()
     for line in lines:
         if not line.strip():
             continue
         step = json.loads(line)
         entries, order = [], []
         for entry in step["entries"]:
-            number = numbers.setdefault(entry["id"], len(numbers))
+            if entry["id"] not in numbers:
+                numbers[entry["id"]] = next(fresh)
+            number = numbers[entry["id"]]
             wanted = sorted(set(entry["want"]))
             order.append([wanted.index(place) for place in entry["want"]])
             entries.append((number, entry["tokens"], wanted))
@@ -54,7 +58,8 @@ def replay(engine, vocab: int, lines, out_dir: str, answer=sys.stdout) -> None:
             path = os.path.join(out_dir, f"{step['step']}.f32")
             np.ascontiguousarray(logits[rows], dtype="<f4").tofile(path)
         for name in step.get("end", []):
-            engine.end_forced(numbers.pop(name))
+            if name in numbers:
+                engine.end_forced(numbers.pop(name))
         print(f"done {step['step']}", file=answer, flush=True)
 
 
