@@ -6,19 +6,21 @@
 //
 // A column of S (one value channel) never meets another one, so a CTA takes the columns of one head of one sequence and
 // keeps them in registers over the whole segment: the state is read from and written to memory once per step however
-// long the segment is.  Three kernels:
+// long the segment is.  Four kernels:
 //   decode    one token per sequence: every load is issued up front, then three barriers
-//   prompt    bf16 segments: half of the warps prepare a tile of 16 tokens (decays with one small tensor-core product,
+//   chunk     bf16 segments, heads up to 64: tiles of 16 tokens as matrix products on the tensor cores
+//   prompt    bf16 segments, larger heads: half of the warps prepare a tile of 16 tokens (decays with one small tensor-core product,
 //             removal rates, unit scales) and finish the previous one (norm, gate), the others run the recurrence over
 //             the tile between them; projections arrive through cp.async two tiles ahead
 //   general   any activation type and head size
-// All arithmetic on the state is f32 multiply-adds, two-wide where the sm_100 packed instructions take it (each half
+// Outside the chunk kernel (see there) all arithmetic on the state is f32 multiply-adds, two-wide where the sm_100 packed instructions take it (each half
 // rounds like the scalar one).
 #include <math.h>
 
 #include <type_traits>
 
 #include "launch.h"
+#include "options.h"
 #include "stack_common.cuh"
 
 namespace lfm25 {
@@ -1017,6 +1019,613 @@ delta_prompt_kernel(const DeltaArgs<__nv_bfloat16> args) {
     }
 }
 
+
+// ------------------------------------------------------------------------------------------------ chunk kernel
+//
+// The recurrence over a tile of 16 tokens as matrix products.  With P_t the product of the decays of the tile's tokens
+// up to t, S_t = diag(P_t) Q_t, and
+//     U_t = u_t P_(t-1),   R_t = r_t P_t,   K_t = k_t / P_t,   B_t = -(a_t u_t) / P_t          (per key channel)
+// the update is Q_t = Q_(t-1) + B_t (U_t^T Q_(t-1)) + K_t v_t^T, so with Y_t = Q_(t-1)^T U_t
+//     (I - tril(U B^T, -1)) Y = U Q_0 + tril(U K^T, -1) V
+//     O = R Q_0 + tril(R B^T) Y + tril(R K^T) V,      Q_16 = Q_0 + B^T Y + K^T V.
+// A decay is at least exp(-exp(-1/2)), so 1 / P_t stays below 17000 and every product keeps its relative accuracy.
+// The products run on the tensor cores in TF32 with both operands split into two parts (three products), which
+// leaves errors of the size of f32 rounding; v is bf16 and needs no second part.
+//
+// A CTA owns one head of one segment and works as a pipeline over tiles, one barrier per step; in step i
+//     copies       load tile i + 4, finish tile i - 1 (norm, gate, output), tanh(z) and |k| of tile i + 3
+//     elements     decay logits (a small product), prefix sums over the tokens, U, R, K, B of tile i + 2
+//     triangles    the four masked 16 x 16 products and the inverse of the unit triangle of tile i + 1
+//     matrices     everything that meets the state, for tile i; a warp owns 16 value columns and their state
+
+constexpr uint32_t kChunkDim = 64;                // padded head size
+constexpr uint32_t kChunkStages = 6;              // tiles i - 1 .. i + 4 of raw projections
+constexpr uint32_t kRowStride = kChunkDim + 4;    // U, R: A operands, [token][channel]
+constexpr uint32_t kTransposedStride = kChunkDim + 8;   // K, B: also read as [channel][token]
+constexpr uint32_t kProducedStride = kChunkDim + 8;
+constexpr uint32_t kTriangleStride = 20;
+constexpr uint32_t kColumnStride = 24;            // a warp's 16 columns: state, right-hand side, Y
+
+struct ChunkLayout {
+    uint32_t rank_pad, z_stride, raw_row;
+    size_t raw, operands, triangles, decay_end, tanh_parts, w2, constants, scale, produced, state, columns, total;
+    __host__ __device__ explicit ChunkLayout(uint32_t rank) {
+        rank_pad = (rank + 31) / 32 * 32;
+        z_stride = rank_pad + 8;
+        raw_row = 5 * kChunkDim + rank_pad;
+        size_t at = 0;
+        raw = at;
+        at += static_cast<size_t>(kChunkStages) * kPromptTokens * raw_row * 2;
+        operands = at;                            // [3][U | R | K | B]
+        at += 3 * kPromptTokens * 2 * (kRowStride + kTransposedStride) * 4;
+        triangles = at;                           // [2][inverse | U K^T | R B^T | R K^T | U B^T]
+        at += 2 * 5 * kPromptTokens * kTriangleStride * 4;
+        decay_end = at;                           // [3][channel]: P of the tile's last token
+        at += 3 * kChunkDim * 4;
+        tanh_parts = at;                          // [2][high | low][token][z_stride]
+        at += 2 * 2 * kPromptTokens * z_stride * 2;
+        w2 = at;
+        at += kChunkDim * z_stride * 2;
+        constants = at;                           // w0, removal bias, norm weight
+        at += 3 * kChunkDim * 4;
+        scale = at;                               // [2][token]: 1 / |k|
+        at += 2 * kPromptTokens * 4;
+        produced = at;                            // [2][token][kProducedStride]
+        at += 2 * kPromptTokens * kProducedStride * 4;
+        state = at;                               // [warp][channel][kColumnStride]
+        at += 4 * kChunkDim * kColumnStride * 4;
+        columns = at;                             // [warp][token][kColumnStride]
+        at += 4 * kPromptTokens * kColumnStride * 4;
+        total = at;
+    }
+};
+
+// D(16x8) += A(16x8, tf32) * B(8x8, tf32), f32 accumulation
+__device__ __forceinline__ void mma_tf32(float (&d)[4], const float (&a)[4], const float (&b)[2]) {
+    asm volatile(
+        "mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+        "{%0, %1, %2, %3};"
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])),
+          "r"(__float_as_uint(b[0])), "r"(__float_as_uint(b[1])));
+}
+
+// An operand fragment as high + low: the high part is what TF32 keeps of the value (10 mantissa bits), the low part the
+// rest, of which TF32 keeps another 10.
+template <int N>
+struct SplitFragment {
+    float high[N], low[N];
+    __device__ __forceinline__ void set(int index, float value) {
+        high[index] = __uint_as_float(__float_as_uint(value) & 0xffffe000u);
+        low[index] = value - high[index];
+    }
+};
+using FragmentA = SplitFragment<4>;
+using FragmentB = SplitFragment<2>;
+
+__device__ __forceinline__ void mma_split(float (&d)[4], const FragmentA& a, const FragmentB& b) {
+    mma_tf32(d, a.low, b.high);
+    mma_tf32(d, a.high, b.low);
+    mma_tf32(d, a.high, b.high);
+}
+// B is exact in TF32
+__device__ __forceinline__ void mma_split(float (&d)[4], const FragmentA& a, const float (&b)[2]) {
+    mma_tf32(d, a.low, b);
+    mma_tf32(d, a.high, b);
+}
+
+// rows `source[row * stride + column]` of a 16 x 8 operand
+__device__ __forceinline__ FragmentA load_a(const float* source, uint32_t stride, uint32_t lane) {
+    FragmentA out;
+    const float* at = source + (lane >> 2) * stride + (lane & 3);
+    out.set(0, at[0]);
+    out.set(1, at[8 * stride]);
+    out.set(2, at[4]);
+    out.set(3, at[8 * stride + 4]);
+    return out;
+}
+// the same operand stored transposed: `source[column * stride + row]`
+__device__ __forceinline__ FragmentA load_a_transposed(const float* source, uint32_t stride, uint32_t lane) {
+    FragmentA out;
+    const float* at = source + (lane & 3) * stride + (lane >> 2);
+    out.set(0, at[0]);
+    out.set(1, at[8]);
+    out.set(2, at[4 * stride]);
+    out.set(3, at[4 * stride + 8]);
+    return out;
+}
+// an 8 x 8 operand B[k][n] stored as `source[k * stride + n]`, or transposed as `source[n * stride + k]`
+__device__ __forceinline__ FragmentB load_b(const float* source, uint32_t stride, uint32_t lane) {
+    FragmentB out;
+    const float* at = source + (lane & 3) * stride + (lane >> 2);
+    out.set(0, at[0]);
+    out.set(1, at[4 * stride]);
+    return out;
+}
+__device__ __forceinline__ FragmentB load_b_transposed(const float* source, uint32_t stride, uint32_t lane) {
+    FragmentB out;
+    const float* at = source + (lane >> 2) * stride + (lane & 3);
+    out.set(0, at[0]);
+    out.set(1, at[4]);
+    return out;
+}
+// a 16 x 8 result to `target[row * stride + column]`
+__device__ __forceinline__ void store_c(float* target, uint32_t stride, uint32_t lane, const float (&c)[4]) {
+    float* at = target + (lane >> 2) * stride + (lane & 3) * 2;
+    *reinterpret_cast<float2*>(at) = make_float2(c[0], c[1]);
+    *reinterpret_cast<float2*>(at + 8 * stride) = make_float2(c[2], c[3]);
+}
+
+constexpr uint32_t kChunkThreads = 512;           // four groups of four warps
+
+__global__ void __launch_bounds__(kChunkThreads)
+delta_chunk_kernel(const DeltaArgs<__nv_bfloat16> args) {
+    constexpr uint32_t DP = kChunkDim;
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) unsigned char chunk_shared[];
+    const ChunkLayout layout(args.rank);
+    const uint32_t dim = args.dim;
+    const uint32_t head = blockIdx.x % args.heads;
+    const uint32_t segment = blockIdx.x / args.heads;
+    const uint32_t begin = args.segments.offsets[segment];
+    uint32_t end = args.segments.offsets[segment + 1];
+    end = end < args.segments.num_tokens ? end : static_cast<uint32_t>(args.segments.num_tokens);
+    const size_t slot = args.segments.slots[segment];
+    if (begin >= end || slot >= args.segments.num_request_slots) {
+        return;
+    }
+    const int tiles = static_cast<int>((end - begin + kPromptTokens - 1) / kPromptTokens);
+    const size_t width = static_cast<size_t>(args.heads) * dim;
+    const size_t head_base = static_cast<size_t>(head) * dim;
+    auto* raw = reinterpret_cast<__nv_bfloat16*>(chunk_shared + layout.raw);
+    auto* tanh_parts = reinterpret_cast<__nv_bfloat16*>(chunk_shared + layout.tanh_parts);
+    auto* w2 = reinterpret_cast<__nv_bfloat16*>(chunk_shared + layout.w2);
+    auto* constants = reinterpret_cast<float*>(chunk_shared + layout.constants);
+    float* state_base = reinterpret_cast<float*>(static_cast<unsigned char*>(args.record.base) +
+                                                 slot * args.record.stride + args.record.offset) +
+                        head_base * dim;
+    auto stage_of = [&](int tile) { return raw + tile % kChunkStages * kPromptTokens * layout.raw_row; };
+    auto unit_of = [&](int tile) {
+        return reinterpret_cast<float*>(chunk_shared + layout.scale) + tile % 2 * kPromptTokens;
+    };
+    auto tanh_of = [&](int tile) { return tanh_parts + tile % 2 * 2 * kPromptTokens * layout.z_stride; };
+    auto operands_of = [&](int tile) {
+        return reinterpret_cast<float*>(chunk_shared + layout.operands) +
+               tile % 3 * kPromptTokens * 2 * (kRowStride + kTransposedStride);
+    };
+    constexpr uint32_t kOperandR = kPromptTokens * kRowStride, kOperandK = 2 * kPromptTokens * kRowStride,
+                       kOperandB = kOperandK + kPromptTokens * kTransposedStride;
+    auto decay_end_of = [&](int tile) {
+        return reinterpret_cast<float*>(chunk_shared + layout.decay_end) + tile % 3 * DP;
+    };
+    constexpr uint32_t kTriangle = kPromptTokens * kTriangleStride;
+    auto triangles_of = [&](int tile) {
+        return reinterpret_cast<float*>(chunk_shared + layout.triangles) + tile % 2 * 5 * kTriangle;
+    };
+    auto produced_of = [&](int tile) {
+        return reinterpret_cast<float*>(chunk_shared + layout.produced) + tile % 2 * kPromptTokens * kProducedStride;
+    };
+
+    for (uint32_t item = threadIdx.x; item < kChunkStages * kPromptTokens * layout.raw_row / 8; item += kChunkThreads) {
+        reinterpret_cast<uint4*>(raw)[item] = make_uint4(0, 0, 0, 0);
+    }
+    for (uint32_t item = threadIdx.x; item < DP * layout.z_stride; item += kChunkThreads) {
+        const uint32_t channel = item / layout.z_stride;
+        const uint32_t z = item - channel * layout.z_stride;
+        w2[item] = channel < dim && z < args.rank ? args.decay_up[(head_base + channel) * args.rank + z]
+                                                  : __float2bfloat16_rn(0.0f);
+    }
+    if (threadIdx.x < DP) {
+        const uint32_t channel = threadIdx.x;
+        const bool live = channel < dim;
+        constants[channel] = live ? __bfloat162float(args.decay_base[head_base + channel]) : 0.0f;
+        constants[DP + channel] = live ? __bfloat162float(args.removal_bias[head_base + channel]) : 0.0f;
+        constants[2 * DP + channel] = live ? __bfloat162float(args.norm[head_base + channel]) : 0.0f;
+    }
+
+    const uint32_t group = threadIdx.x / 128;          // 0 matrices, 1 copies, 2 elements, 3 triangles
+    const uint32_t warp = threadIdx.x / 32 % 4;        // of the group
+    const uint32_t lane = threadIdx.x % 32;
+
+    // ---- matrices: state of 16 value columns, as the accumulators of the update product
+    const uint32_t column0 = warp * 16;
+    float* state = reinterpret_cast<float*>(chunk_shared + layout.state) + warp * DP * kColumnStride;
+    float* columns = reinterpret_cast<float*>(chunk_shared + layout.columns) + warp * kPromptTokens * kColumnStride;
+    float accumulator[4][2][4];                        // [16 key channels][8 columns]
+    if (group == 0) {
+#pragma unroll
+        for (uint32_t m = 0; m < 4; ++m) {
+#pragma unroll
+            for (uint32_t n = 0; n < 2; ++n) {
+#pragma unroll
+                for (uint32_t i = 0; i < 4; ++i) {
+                    const uint32_t row = m * 16 + (lane >> 2) + (i >> 1) * 8;
+                    const uint32_t column = column0 + n * 8 + (lane & 3) * 2 + (i & 1);
+                    accumulator[m][n][i] =
+                        row < dim && column < dim ? state_base[static_cast<size_t>(column) * dim + row] : 0.0f;
+                }
+                store_c(state + m * 16 * kColumnStride + n * 8, kColumnStride, lane, accumulator[m][n]);
+            }
+        }
+    }
+    // ---- copies: the 16-byte pieces of a token's row that this lane moves
+    const uint32_t per_vector = dim / 8;
+    const uint32_t pieces = 5 * per_vector + (args.rank + 7) / 8;
+    auto piece_offsets = [&](uint32_t piece, uint32_t& source, uint32_t& target) {
+        if (piece < 5 * per_vector) {
+            const uint32_t vector = piece / per_vector;
+            const uint32_t chunk = piece - vector * per_vector;
+            source = static_cast<uint32_t>(vector * width + head_base) + chunk * 8;
+            target = vector * DP + chunk * 8;
+        } else {
+            const uint32_t chunk = piece - 5 * per_vector;
+            source = static_cast<uint32_t>(5 * width) + chunk * 8;
+            target = 5 * DP + chunk * 8;
+        }
+    };
+    uint32_t first_source = 0, first_target = 0, second_source = 0, second_target = 0;
+    piece_offsets(lane, first_source, first_target);
+    piece_offsets(lane + 32, second_source, second_target);
+    __syncthreads();
+
+    for (int step = -4; step <= tiles; ++step) {
+        if (group == 0) {
+            const int tile = step;
+            if (tile >= 0 && tile < tiles) {
+                const float* operands = operands_of(tile);
+                const float* triangles = triangles_of(tile);
+                // U Q_0 and R Q_0
+                float from_state[2][2][4] = {};        // [U, R][8 columns]
+#pragma unroll
+                for (uint32_t k = 0; k < DP / 8; ++k) {
+                    const FragmentB b0 = load_b(state + k * 8 * kColumnStride, kColumnStride, lane);
+                    const FragmentB b1 = load_b(state + k * 8 * kColumnStride + 8, kColumnStride, lane);
+#pragma unroll
+                    for (uint32_t m = 0; m < 2; ++m) {
+                        const FragmentA a = load_a(operands + m * kOperandR + k * 8, kRowStride, lane);
+                        mma_split(from_state[m][0], a, b0);
+                        mma_split(from_state[m][1], a, b1);
+                    }
+                }
+                // v of the tile: B operand [token][column], exact in TF32
+                float v[2][2][2];                      // [8 tokens][8 columns]
+                const __nv_bfloat16* values = stage_of(tile) + 2 * DP + column0;
+#pragma unroll
+                for (uint32_t k = 0; k < 2; ++k) {
+#pragma unroll
+                    for (uint32_t n = 0; n < 2; ++n) {
+#pragma unroll
+                        for (uint32_t i = 0; i < 2; ++i) {
+                            v[k][n][i] = __bfloat162float(
+                                values[(k * 8 + (lane & 3) + i * 4) * layout.raw_row + n * 8 + (lane >> 2)]);
+                        }
+                    }
+                }
+                // right-hand side, then Y
+#pragma unroll
+                for (uint32_t k = 0; k < 2; ++k) {
+                    const FragmentA a = load_a(triangles + 1 * kTriangle + k * 8, kTriangleStride, lane);
+                    mma_split(from_state[0][0], a, v[k][0]);
+                    mma_split(from_state[0][1], a, v[k][1]);
+                }
+                store_c(columns, kColumnStride, lane, from_state[0][0]);
+                store_c(columns + 8, kColumnStride, lane, from_state[0][1]);
+                __syncwarp();
+                float solved[2][4] = {};
+#pragma unroll
+                for (uint32_t k = 0; k < 2; ++k) {
+                    const FragmentA a = load_a(triangles + k * 8, kTriangleStride, lane);
+#pragma unroll
+                    for (uint32_t n = 0; n < 2; ++n) {
+                        mma_split(solved[n], a, load_b(columns + k * 8 * kColumnStride + n * 8, kColumnStride, lane));
+                    }
+                }
+                __syncwarp();
+                store_c(columns, kColumnStride, lane, solved[0]);
+                store_c(columns + 8, kColumnStride, lane, solved[1]);
+                __syncwarp();
+                FragmentB y[2][2];
+#pragma unroll
+                for (uint32_t k = 0; k < 2; ++k) {
+#pragma unroll
+                    for (uint32_t n = 0; n < 2; ++n) {
+                        y[k][n] = load_b(columns + k * 8 * kColumnStride + n * 8, kColumnStride, lane);
+                    }
+                }
+                // O
+#pragma unroll
+                for (uint32_t k = 0; k < 2; ++k) {
+                    const FragmentA with_y = load_a(triangles + 2 * kTriangle + k * 8, kTriangleStride, lane);
+                    const FragmentA with_v = load_a(triangles + 3 * kTriangle + k * 8, kTriangleStride, lane);
+#pragma unroll
+                    for (uint32_t n = 0; n < 2; ++n) {
+                        mma_split(from_state[1][n], with_y, y[k][n]);
+                        mma_split(from_state[1][n], with_v, v[k][n]);
+                    }
+                }
+                store_c(produced_of(tile) + column0, kProducedStride, lane, from_state[1][0]);
+                store_c(produced_of(tile) + column0 + 8, kProducedStride, lane, from_state[1][1]);
+                // the state behind the tile
+                const float* decay = decay_end_of(tile);
+#pragma unroll
+                for (uint32_t m = 0; m < 4; ++m) {
+#pragma unroll
+                    for (uint32_t k = 0; k < 2; ++k) {
+                        const uint32_t at = k * 8 * kTransposedStride + m * 16;
+                        const FragmentA with_v = load_a_transposed(operands + kOperandK + at, kTransposedStride, lane);
+                        const FragmentA with_y = load_a_transposed(operands + kOperandB + at, kTransposedStride, lane);
+#pragma unroll
+                        for (uint32_t n = 0; n < 2; ++n) {
+                            mma_split(accumulator[m][n], with_v, v[k][n]);
+                            mma_split(accumulator[m][n], with_y, y[k][n]);
+                        }
+                    }
+                    const float upper = decay[m * 16 + (lane >> 2)], lower = decay[m * 16 + (lane >> 2) + 8];
+#pragma unroll
+                    for (uint32_t n = 0; n < 2; ++n) {
+                        accumulator[m][n][0] *= upper;
+                        accumulator[m][n][1] *= upper;
+                        accumulator[m][n][2] *= lower;
+                        accumulator[m][n][3] *= lower;
+                        store_c(state + m * 16 * kColumnStride + n * 8, kColumnStride, lane, accumulator[m][n]);
+                    }
+                }
+            }
+        } else if (group == 1) {
+            // ---- load tile step + 4
+            {
+                const int tile = step + 4;
+                const uint32_t first = begin + static_cast<uint32_t>(tile) * kPromptTokens;
+                if (tile < tiles) {
+#pragma unroll
+                    for (uint32_t i = 0; i < 4; ++i) {
+                        const uint32_t t = warp * 4 + i;
+                        if (first + t < end) {
+                            const __nv_bfloat16* source = args.projected + static_cast<size_t>(first + t) * args.pitch;
+                            __nv_bfloat16* target = stage_of(tile) + t * layout.raw_row;
+                            if (lane < pieces) copy_async_16(target + first_target, source + first_source);
+                            if (lane + 32 < pieces) copy_async_16(target + second_target, source + second_source);
+                            for (uint32_t piece = lane + 64; piece < pieces; piece += 32) {
+                                uint32_t from, to;
+                                piece_offsets(piece, from, to);
+                                copy_async_16(target + to, source + from);
+                            }
+                        }
+                    }
+                }
+                copy_async_commit();
+            }
+            // ---- finish tile step - 1
+            if (step >= 1) {
+                const int tile = step - 1;
+                const __nv_bfloat16* stage = stage_of(tile);
+                const float* source = produced_of(tile);
+                const uint32_t first = begin + static_cast<uint32_t>(tile) * kPromptTokens;
+                float2 value[4], gate[4];
+                float squares[4];
+#pragma unroll
+                for (uint32_t i = 0; i < 4; ++i) {
+                    const uint32_t t = warp * 4 + i;
+                    value[i] = *reinterpret_cast<const float2*>(source + t * kProducedStride + lane * 2);
+                    gate[i] = __bfloat1622float2(
+                        *reinterpret_cast<const __nv_bfloat162*>(stage + t * layout.raw_row + 3 * DP + lane * 2));
+                    squares[i] = fmaf(value[i].x, value[i].x, value[i].y * value[i].y);
+                }
+#pragma unroll
+                for (uint32_t i = 0; i < 4; ++i) squares[i] = warp_sum(squares[i]);
+                const float2 weight = *reinterpret_cast<const float2*>(constants + 2 * DP + lane * 2);
+#pragma unroll
+                for (uint32_t i = 0; i < 4; ++i) {
+                    const uint32_t t = warp * 4 + i;
+                    const float factor = rsqrtf(squares[i] / static_cast<float>(dim) + args.eps);
+                    const uint32_t both = pack_bf16x2(value[i].x * factor * weight.x * fast_sigmoid(gate[i].x),
+                                                      value[i].y * factor * weight.y * fast_sigmoid(gate[i].y));
+                    if (lane * 2 < dim && first + t < end) {
+                        *reinterpret_cast<uint32_t*>(args.out + static_cast<size_t>(first + t) * args.out_pitch +
+                                                     head_base + lane * 2) = both;
+                    }
+                }
+            }
+            // ---- tanh(z) and 1 / |k| of tile step + 3, whose copies were issued one step ago
+            copy_async_wait<1>();
+            named_barrier(1, 128);
+            const int tile = step + 3;
+            if (tile >= 0 && tile < tiles) {
+                const __nv_bfloat16* stage = stage_of(tile);
+                __nv_bfloat16* parts = tanh_of(tile);
+                float squares[4];
+#pragma unroll
+                for (uint32_t i = 0; i < 4; ++i) {
+                    const float2 both = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(
+                        stage + (warp * 4 + i) * layout.raw_row + DP + lane * 2));
+                    squares[i] = fmaf(both.x, both.x, both.y * both.y);
+                }
+                for (uint32_t z = lane * 2; z < layout.rank_pad; z += 64) {
+                    float2 both[4];
+#pragma unroll
+                    for (uint32_t i = 0; i < 4; ++i) {
+                        both[i] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(
+                            stage + (warp * 4 + i) * layout.raw_row + 5 * DP + z));
+                        // columns between rank and the end of its last copy belong to nobody
+                        both[i].x = z < args.rank ? fast_tanh(both[i].x) : 0.0f;
+                        both[i].y = z + 1 < args.rank ? fast_tanh(both[i].y) : 0.0f;
+                    }
+#pragma unroll
+                    for (uint32_t i = 0; i < 4; ++i) {
+                        const __nv_bfloat162 high = __floats2bfloat162_rn(both[i].x, both[i].y);
+                        const float2 rounded = __bfloat1622float2(high);
+                        __nv_bfloat16* target = parts + (warp * 4 + i) * layout.z_stride + z;
+                        *reinterpret_cast<__nv_bfloat162*>(target) = high;
+                        *reinterpret_cast<__nv_bfloat162*>(target + kPromptTokens * layout.z_stride) =
+                            __floats2bfloat162_rn(both[i].x - rounded.x, both[i].y - rounded.y);
+                    }
+                }
+#pragma unroll
+                for (uint32_t i = 0; i < 4; ++i) squares[i] = warp_sum(squares[i]);
+                if (lane < 4) {
+                    const float mine = lane == 0 ? squares[0] : (lane == 1 ? squares[1] : (lane == 2 ? squares[2] : squares[3]));
+                    unit_of(tile)[warp * 4 + lane] = rsqrtf(mine + kUnitEps);
+                }
+            }
+        } else if (group == 2) {
+            const int tile = step + 2;
+            if (tile >= 0 && tile < tiles) {
+                const uint32_t tokens = min(kPromptTokens, end - begin - static_cast<uint32_t>(tile) * kPromptTokens);
+                const __nv_bfloat16* stage = stage_of(tile);
+                const __nv_bfloat16* parts = tanh_of(tile);
+                const float* unit = unit_of(tile);
+                float* operands = operands_of(tile);
+                // decay logits of 16 tokens x 16 channels per warp
+                float logits[2][4] = {};
+                const uint32_t z_row = lane % 16, z_part = lane / 16 * 8;
+                for (uint32_t z = 0; z < layout.rank_pad; z += 16) {
+                    uint32_t b0, b1, b2, b3, high[4], low[4];
+                    const uint32_t channel = warp * 16 + lane / 16 * 8 + lane % 8;
+                    ldmatrix_x4(smem_u32(w2 + channel * layout.z_stride + z + lane / 8 % 2 * 8), b0, b1, b2, b3);
+                    const __nv_bfloat16* source = parts + z_row * layout.z_stride + z + z_part;
+                    ldmatrix_x4(smem_u32(source), high[0], high[1], high[2], high[3]);
+                    ldmatrix_x4(smem_u32(source + kPromptTokens * layout.z_stride), low[0], low[1], low[2], low[3]);
+                    mma_bf16_16816(logits[0], high[0], high[1], high[2], high[3], b0, b1);
+                    mma_bf16_16816(logits[1], high[0], high[1], high[2], high[3], b2, b3);
+                    mma_bf16_16816(logits[0], low[0], low[1], low[2], low[3], b0, b1);
+                    mma_bf16_16816(logits[1], low[0], low[1], low[2], low[3], b2, b3);
+                }
+                const uint32_t t0 = lane >> 2;
+                // log decay per token, then its prefix sums: over the eight lanes that hold tokens 0..7, and over
+                // those that hold 8..15 in the other half of the fragment
+                float own[2][4], prefix[2][4];
+#pragma unroll
+                for (uint32_t n = 0; n < 2; ++n) {
+                    const uint32_t channel = warp * 16 + n * 8 + (lane & 3) * 2;
+#pragma unroll
+                    for (uint32_t i = 0; i < 4; ++i) {
+                        own[n][i] = t0 + (i >> 1) * 8 < tokens
+                                        ? -kDecayScale * fast_sigmoid(logits[n][i] + constants[channel + (i & 1)])
+                                        : 0.0f;
+                        prefix[n][i] = own[n][i];
+                    }
+                }
+#pragma unroll
+                for (uint32_t delta = 4; delta < 32; delta <<= 1) {
+#pragma unroll
+                    for (uint32_t n = 0; n < 2; ++n) {
+#pragma unroll
+                        for (uint32_t i = 0; i < 4; ++i) {
+                            const float other = __shfl_up_sync(0xffffffffu, prefix[n][i], delta);
+                            if (lane >= delta) prefix[n][i] += other;
+                        }
+                    }
+                }
+#pragma unroll
+                for (uint32_t n = 0; n < 2; ++n) {
+#pragma unroll
+                    for (uint32_t i = 0; i < 2; ++i) {
+                        prefix[n][2 + i] += __shfl_sync(0xffffffffu, prefix[n][i], 28 + (lane & 3));
+                    }
+                }
+#pragma unroll
+                for (uint32_t n = 0; n < 2; ++n) {
+                    const uint32_t channel = warp * 16 + n * 8 + (lane & 3) * 2;
+                    const float2 bias = *reinterpret_cast<const float2*>(constants + DP + channel);
+#pragma unroll
+                    for (uint32_t half = 0; half < 2; ++half) {
+                        const uint32_t t = t0 + half * 8;
+                        const __nv_bfloat16* row = stage + t * layout.raw_row + channel;
+                        float2 r = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row));
+                        float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + DP));
+                        const float2 rate = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + 4 * DP));
+                        if (t >= tokens) r = k = make_float2(0.0f, 0.0f);      // left over from an earlier tile
+                        const float scale = unit[t];
+                        const float px = __expf(prefix[n][2 * half]), py = __expf(prefix[n][2 * half + 1]);
+                        const float bx = __expf(prefix[n][2 * half] - own[n][2 * half]);
+                        const float by = __expf(prefix[n][2 * half + 1] - own[n][2 * half + 1]);
+                        const float ix = __expf(-prefix[n][2 * half]), iy = __expf(-prefix[n][2 * half + 1]);
+                        float* row_target = operands + t * kRowStride + channel;
+                        *reinterpret_cast<float2*>(row_target) = make_float2(k.x * scale * bx, k.y * scale * by);
+                        *reinterpret_cast<float2*>(row_target + kOperandR) = make_float2(r.x * px, r.y * py);
+                        float* transposed_target = operands + kOperandK + t * kTransposedStride + channel;
+                        *reinterpret_cast<float2*>(transposed_target) = make_float2(k.x * ix, k.y * iy);
+                        *reinterpret_cast<float2*>(transposed_target + kOperandB - kOperandK) =
+                            make_float2(-fast_sigmoid(rate.x + bias.x) * k.x * scale * ix,
+                                        -fast_sigmoid(rate.y + bias.y) * k.y * scale * iy);
+                        if (t == kPromptTokens - 1) {
+                            *reinterpret_cast<float2*>(decay_end_of(tile) + channel) = make_float2(px, py);
+                        }
+                    }
+                }
+            }
+        } else {
+            const int tile = step + 1;
+            if (tile >= 0 && tile < tiles) {
+                const float* operands = operands_of(tile);
+                float* triangles = triangles_of(tile);
+                // warps 0, 1: rows of U; 2, 3: rows of R; even warps against B, odd ones against K
+                const float* rows = operands + (warp >> 1) * kOperandR;
+                const float* against = operands + (warp & 1 ? kOperandK : kOperandB);
+                float product[2][4] = {};
+#pragma unroll
+                for (uint32_t k = 0; k < DP / 8; ++k) {
+                    const FragmentA a = load_a(rows + k * 8, kRowStride, lane);
+#pragma unroll
+                    for (uint32_t n = 0; n < 2; ++n) {
+                        mma_split(product[n],
+                                  a, load_b_transposed(against + n * 8 * kTransposedStride + k * 8, kTransposedStride, lane));
+                    }
+                }
+                // U B^T goes behind the four results, U K^T, R B^T and R K^T to places 1, 2 and 3
+                float* target = triangles + (warp == 0 ? 4 : warp) * kTriangle;
+#pragma unroll
+                for (uint32_t n = 0; n < 2; ++n) {
+#pragma unroll
+                    for (uint32_t i = 0; i < 4; ++i) {
+                        const uint32_t row = (lane >> 2) + (i >> 1) * 8;
+                        const uint32_t column = n * 8 + (lane & 3) * 2 + (i & 1);
+                        const bool kept = warp < 2 ? column < row : column <= row;     // U meets the state before s = t
+                        if (!kept) product[n][i] = 0.0f;
+                    }
+                    store_c(target + n * 8, kTriangleStride, lane, product[n]);
+                }
+                if (warp == 0) {
+                    __syncwarp();
+                    // column `lane` of the inverse of I - L: x_t = e_t + sum over s < t of L[t][s] x_s
+                    const float* lower = triangles + 4 * kTriangle;
+                    float x[kPromptTokens];
+#pragma unroll
+                    for (uint32_t t = 0; t < kPromptTokens; ++t) {
+                        float even = t == lane ? 1.0f : 0.0f, odd = 0.0f;
+#pragma unroll
+                        for (uint32_t s = 0; s < t; s += 2) {
+                            const float2 pair = *reinterpret_cast<const float2*>(lower + t * kTriangleStride + s);
+                            even = fmaf(pair.x, x[s], even);
+                            if (s + 1 < t) odd = fmaf(pair.y, x[s + 1], odd);
+                        }
+                        x[t] = even + odd;
+                        if (lane < kPromptTokens) triangles[t * kTriangleStride + lane] = x[t];
+                    }
+                }
+            }
+        }
+        __syncthreads();
+    }
+    if (group == 0) {
+#pragma unroll
+        for (uint32_t m = 0; m < 4; ++m) {
+#pragma unroll
+            for (uint32_t n = 0; n < 2; ++n) {
+#pragma unroll
+                for (uint32_t i = 0; i < 4; ++i) {
+                    const uint32_t row = m * 16 + (lane >> 2) + (i >> 1) * 8;
+                    const uint32_t column = column0 + n * 8 + (lane & 3) * 2 + (i & 1);
+                    if (row < dim && column < dim) {
+                        state_base[static_cast<size_t>(column) * dim + row] = accumulator[m][n][i];
+                    }
+                }
+            }
+        }
+    }
+}
+
 template <typename T, uint32_t DP>
 cudaError_t launch_decode(cudaStream_t stream, const DeltaArgs<T>& args) {
     const size_t shared = (5 * DP + 2 * (DP * 4 / 32) + args.rank) * sizeof(float);
@@ -1038,6 +1647,16 @@ cudaError_t launch_prompt(cudaStream_t stream, const DeltaArgs<__nv_bfloat16>& a
     if (status != cudaSuccess) return status;
     return launch_kernel(kernel, static_cast<unsigned int>(args.segments.num_segments * args.heads),
                          DP / COLUMNS * 8 + HELPERS, shared, stream, 1, args);
+}
+
+cudaError_t launch_chunk(cudaStream_t stream, const DeltaArgs<__nv_bfloat16>& args) {
+    const size_t shared = ChunkLayout(args.rank).total;
+    const cudaError_t status = cudaFuncSetAttribute(reinterpret_cast<const void*>(delta_chunk_kernel),
+                                                    cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                    static_cast<int>(shared));
+    if (status != cudaSuccess) return status;
+    return launch_kernel(delta_chunk_kernel, static_cast<unsigned int>(args.segments.num_segments * args.heads),
+                         kChunkThreads, shared, stream, 1, args);
 }
 
 bool prompt_kernel_takes(const DeltaArgs<__nv_bfloat16>& args) {
@@ -1104,7 +1723,10 @@ cudaError_t launch_typed(cudaStream_t stream, const DeltaRuleLaunch& launch) {
         return launch_decode<T, 128>(stream, args);
     }
     if constexpr (std::is_same<T, __nv_bfloat16>::value) {
-        if (launch.segments.offsets != nullptr && prompt_kernel_takes(args)) {
+        if (launch.segments.offsets != nullptr && option(kOptDeltaPrompt) != 2 && prompt_kernel_takes(args)) {
+            if (launch.dim <= kChunkDim && ChunkLayout(launch.rank).total <= 227 * 1024 && option(kOptDeltaPrompt) == 0) {
+                return launch_chunk(stream, args);
+            }
             return launch.dim <= 64 ? launch_prompt<64, 4, 128>(stream, args) : launch_prompt<128, 4, 128>(stream, args);
         }
     }

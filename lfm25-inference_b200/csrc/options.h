@@ -18,6 +18,9 @@
 //   hybrid_attention     0 auto | 1 umma | 2 mma               0         kernel of the mixed-step attention
 //   stack_attention      0 auto | 1 scalar                     0         attention of layer-stack models: the tensor-core kernels
 //                                                                        where they take the shape, or always the scalar one
+//   delta_prompt         0 auto | 1 scan | 2 general           0         delta rule over bf16 segments: tensor-core chunks where they
+//                                                                        take the head size, the token-by-token prompt kernel,
+//                                                                        or the general kernel
 //   fp8_gemm_path        0 auto | 1 stream | 2 umma | 3 generic | 4 rows   0   kernel of the E4M3 linear
 //   bf16_gemm            0 auto | 1 umma | 2 cublaslt | 3 rows  0         kernel of the BF16 linear
 //   decode_splits        0 auto | 1..8                         0         KV splits of the decode attention
@@ -43,6 +46,7 @@ enum Option : int {
     kOptEngineGraph,
     kOptHybridAttention,
     kOptStackAttention,
+    kOptDeltaPrompt,
     kOptFp8GemmPath,
     kOptBf16Gemm,
     kOptDecodeSplits,

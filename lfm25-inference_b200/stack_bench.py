@@ -111,7 +111,7 @@ def _bytes_and_flops(node: dict, tokens: int, keys: float, segments: int) -> dic
         "projection_norm_rope_kernel": (tokens * projected * 4, 0.0),
         "attention": (keys * groups * (dim + vdim) * 2 if segments == tokens else 0.0,
                       2.0 * keys * heads * (dim + vdim)),
-        "delta_rule_kernel": (tokens * (6 * inner + RANK) * 2 + segments * state * 2,
+        "delta": (tokens * (6 * inner + RANK) * 2 + segments * state * 2,
                               tokens * delta["heads"] * delta["dim"] ** 2 * 10.0),
     }
 
@@ -121,11 +121,11 @@ def rooflines(node, times, tokens, keys, segments, hbm_gbs, tensor_tflops, fp32_
     at the nominal rate)."""
     out = {}
     for kernel, (launches, micros) in times.items():
-        key = "attention" if "attention" in kernel else kernel
+        key = next((word for word in ("attention", "delta") if word in kernel), kernel)
         work = _bytes_and_flops(node, tokens, keys, segments).get(key)
         if work is None:
             continue
-        peak = fp32_tflops if key == "delta_rule_kernel" else tensor_tflops
+        peak = fp32_tflops if key == "delta" else tensor_tflops
         ideal = max(work[0] / (hbm_gbs * 1e9), work[1] / (peak * 1e12)) * 1e6
         out[kernel] = {"us": round(micros, 2), "roofline_us": round(ideal, 2), "frac": round(ideal / micros, 3)}
     return out

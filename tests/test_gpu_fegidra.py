@@ -82,6 +82,22 @@ def test_delta_rule_layer(device, dtype, heads, dim, rank):
     check_layer(config, 13, device, dtype, [37, 2, 1, 16, 1, 5], rank)
 
 
+@pytest.mark.parametrize("heads,dim,rank", [(3, 16, 5), (2, 64, 16), (1, 24, 1), (2, 48, 70), (1, 128, 40), (2, 64, 250)])
+def test_delta_rule_prompt_kernels_agree(device, library_option, heads, dim, rank):
+    """The tensor-core chunks, the token-by-token prompt kernel and the general kernel on the same bf16 inputs: all keep
+    32-bit accuracy in the recurrence, so they differ by rounding of the bf16 output only.  Strong decays (the chunks
+    divide by their product) and weak ones side by side, portions that end inside a tile."""
+    config = cases.config_of([cases.delta_layer(heads, dim, ff=0)])
+    tensors = cases.random_tensors(config, 83, rank)
+    tensors["l0.mix.w0"][::2] = 9.0                # decay exp(-exp(-1/2)) throughout
+    results = []
+    for forced in (0, 1, 2):
+        library_option("delta_prompt", forced)
+        results.append(run_layer(config, tensors, device, "bfloat16", [200, 33, 2, 16, 3])[0])
+    for other in results[1:]:
+        assert cases.relative_error(other, results[0]).max() < 4e-3
+
+
 @pytest.mark.parametrize("dtype", TYPES)
 @pytest.mark.parametrize("width,ff", [(48, 40), (256, 72), (64, 1000), (50, 30), (96, 9)])
 def test_feed_forward(device, dtype, width, ff):
