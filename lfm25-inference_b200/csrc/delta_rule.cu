@@ -1082,8 +1082,7 @@ struct ChunkLayout {
 
 // D(16x8) += A(16x8, tf32) * B(8x8, tf32), f32 accumulation
 __device__ __forceinline__ void mma_tf32(float (&d)[4], const float (&a)[4], const float (&b)[2]) {
-    asm volatile(
-        "mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+    asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
         "{%0, %1, %2, %3};"
         : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
         : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])),
@@ -1112,6 +1111,21 @@ __device__ __forceinline__ void mma_split(float (&d)[4], const FragmentA& a, con
 __device__ __forceinline__ void mma_split(float (&d)[4], const FragmentA& a, const float (&b)[2]) {
     mma_tf32(d, a.low, b);
     mma_tf32(d, a.high, b);
+}
+// The same for two accumulators, whose products alternate so that none waits for the one before it.
+__device__ __forceinline__ void mma_split(float (&d)[2][4], const FragmentA& a, const FragmentB& b0, const FragmentB& b1) {
+    mma_tf32(d[0], a.low, b0.high);
+    mma_tf32(d[1], a.low, b1.high);
+    mma_tf32(d[0], a.high, b0.low);
+    mma_tf32(d[1], a.high, b1.low);
+    mma_tf32(d[0], a.high, b0.high);
+    mma_tf32(d[1], a.high, b1.high);
+}
+__device__ __forceinline__ void mma_split(float (&d)[2][4], const FragmentA& a, const float (&b0)[2], const float (&b1)[2]) {
+    mma_tf32(d[0], a.low, b0);
+    mma_tf32(d[1], a.low, b1);
+    mma_tf32(d[0], a.high, b0);
+    mma_tf32(d[1], a.high, b1);
 }
 
 // rows `source[row * stride + column]` of a 16 x 8 operand
@@ -1157,6 +1171,7 @@ __device__ __forceinline__ void store_c(float* target, uint32_t stride, uint32_t
 }
 
 constexpr uint32_t kChunkThreads = 512;           // four groups of four warps
+static_assert(kChunkThreads == 8 * kChunkDim, "eight threads per channel stage W2");
 
 __global__ void __launch_bounds__(kChunkThreads)
 delta_chunk_kernel(const DeltaArgs<__nv_bfloat16> args) {
@@ -1210,11 +1225,23 @@ delta_chunk_kernel(const DeltaArgs<__nv_bfloat16> args) {
     for (uint32_t item = threadIdx.x; item < kChunkStages * kPromptTokens * layout.raw_row / 8; item += kChunkThreads) {
         reinterpret_cast<uint4*>(raw)[item] = make_uint4(0, 0, 0, 0);
     }
-    for (uint32_t item = threadIdx.x; item < DP * layout.z_stride; item += kChunkThreads) {
-        const uint32_t channel = item / layout.z_stride;
-        const uint32_t z = item - channel * layout.z_stride;
-        w2[item] = channel < dim && z < args.rank ? args.decay_up[(head_base + channel) * args.rank + z]
-                                                  : __float2bfloat16_rn(0.0f);
+    {
+        // eight threads per channel
+        const uint32_t channel = threadIdx.x / 8;
+        const __nv_bfloat16* source = args.decay_up + (head_base + channel) * args.rank;
+        const bool vector_rank = args.rank % 8 == 0;
+        for (uint32_t z = threadIdx.x % 8 * 8; z < layout.z_stride; z += 64) {
+            uint4 value = make_uint4(0, 0, 0, 0);
+            if (channel < dim && z < args.rank) {
+                if (vector_rank) {
+                    value = *reinterpret_cast<const uint4*>(source + z);
+                } else {
+                    auto* elements = reinterpret_cast<__nv_bfloat16*>(&value);
+                    for (uint32_t i = 0; i < 8 && z + i < args.rank; ++i) elements[i] = source[z + i];
+                }
+            }
+            *reinterpret_cast<uint4*>(w2 + channel * layout.z_stride + z) = value;
+        }
     }
     if (threadIdx.x < DP) {
         const uint32_t channel = threadIdx.x;
@@ -1284,8 +1311,7 @@ delta_chunk_kernel(const DeltaArgs<__nv_bfloat16> args) {
 #pragma unroll
                     for (uint32_t m = 0; m < 2; ++m) {
                         const FragmentA a = load_a(operands + m * kOperandR + k * 8, kRowStride, lane);
-                        mma_split(from_state[m][0], a, b0);
-                        mma_split(from_state[m][1], a, b1);
+                        mma_split(from_state[m], a, b0, b1);
                     }
                 }
                 // v of the tile: B operand [token][column], exact in TF32
@@ -1306,8 +1332,7 @@ delta_chunk_kernel(const DeltaArgs<__nv_bfloat16> args) {
 #pragma unroll
                 for (uint32_t k = 0; k < 2; ++k) {
                     const FragmentA a = load_a(triangles + 1 * kTriangle + k * 8, kTriangleStride, lane);
-                    mma_split(from_state[0][0], a, v[k][0]);
-                    mma_split(from_state[0][1], a, v[k][1]);
+                    mma_split(from_state[0], a, v[k][0], v[k][1]);
                 }
                 store_c(columns, kColumnStride, lane, from_state[0][0]);
                 store_c(columns + 8, kColumnStride, lane, from_state[0][1]);
@@ -1316,10 +1341,8 @@ delta_chunk_kernel(const DeltaArgs<__nv_bfloat16> args) {
 #pragma unroll
                 for (uint32_t k = 0; k < 2; ++k) {
                     const FragmentA a = load_a(triangles + k * 8, kTriangleStride, lane);
-#pragma unroll
-                    for (uint32_t n = 0; n < 2; ++n) {
-                        mma_split(solved[n], a, load_b(columns + k * 8 * kColumnStride + n * 8, kColumnStride, lane));
-                    }
+                    mma_split(solved, a, load_b(columns + k * 8 * kColumnStride, kColumnStride, lane),
+                              load_b(columns + k * 8 * kColumnStride + 8, kColumnStride, lane));
                 }
                 __syncwarp();
                 store_c(columns, kColumnStride, lane, solved[0]);
@@ -1338,11 +1361,8 @@ delta_chunk_kernel(const DeltaArgs<__nv_bfloat16> args) {
                 for (uint32_t k = 0; k < 2; ++k) {
                     const FragmentA with_y = load_a(triangles + 2 * kTriangle + k * 8, kTriangleStride, lane);
                     const FragmentA with_v = load_a(triangles + 3 * kTriangle + k * 8, kTriangleStride, lane);
-#pragma unroll
-                    for (uint32_t n = 0; n < 2; ++n) {
-                        mma_split(from_state[1][n], with_y, y[k][n]);
-                        mma_split(from_state[1][n], with_v, v[k][n]);
-                    }
+                    mma_split(from_state[1], with_v, v[k][0], v[k][1]);
+                    mma_split(from_state[1], with_y, y[k][0], y[k][1]);
                 }
                 store_c(produced_of(tile) + column0, kProducedStride, lane, from_state[1][0]);
                 store_c(produced_of(tile) + column0 + 8, kProducedStride, lane, from_state[1][1]);
@@ -1355,11 +1375,8 @@ delta_chunk_kernel(const DeltaArgs<__nv_bfloat16> args) {
                         const uint32_t at = k * 8 * kTransposedStride + m * 16;
                         const FragmentA with_v = load_a_transposed(operands + kOperandK + at, kTransposedStride, lane);
                         const FragmentA with_y = load_a_transposed(operands + kOperandB + at, kTransposedStride, lane);
-#pragma unroll
-                        for (uint32_t n = 0; n < 2; ++n) {
-                            mma_split(accumulator[m][n], with_v, v[k][n]);
-                            mma_split(accumulator[m][n], with_y, y[k][n]);
-                        }
+                        mma_split(accumulator[m], with_v, v[k][0], v[k][1]);
+                        mma_split(accumulator[m], with_y, y[k][0], y[k][1]);
                     }
                     const float upper = decay[m * 16 + (lane >> 2)], lower = decay[m * 16 + (lane >> 2) + 8];
 #pragma unroll
@@ -1567,11 +1584,8 @@ delta_chunk_kernel(const DeltaArgs<__nv_bfloat16> args) {
 #pragma unroll
                 for (uint32_t k = 0; k < DP / 8; ++k) {
                     const FragmentA a = load_a(rows + k * 8, kRowStride, lane);
-#pragma unroll
-                    for (uint32_t n = 0; n < 2; ++n) {
-                        mma_split(product[n],
-                                  a, load_b_transposed(against + n * 8 * kTransposedStride + k * 8, kTransposedStride, lane));
-                    }
+                    mma_split(product, a, load_b_transposed(against + k * 8, kTransposedStride, lane),
+                              load_b_transposed(against + 8 * kTransposedStride + k * 8, kTransposedStride, lane));
                 }
                 // U B^T goes behind the four results, U K^T, R B^T and R K^T to places 1, 2 and 3
                 float* target = triangles + (warp == 0 ? 4 : warp) * kTriangle;
@@ -1663,6 +1677,7 @@ bool prompt_kernel_takes(const DeltaArgs<__nv_bfloat16>& args) {
     const size_t shared = args.dim <= 64 ? PromptLayout<64>(args.rank).total : PromptLayout<128>(args.rank).total;
     return args.dim % 8 == 0 && args.dim <= 128 && args.rank <= kPromptMaxRank && args.pitch % 8 == 0 &&
            args.out_pitch % 2 == 0 && aligned_to(args.projected, 16) && aligned_to(args.out, 4) &&
+           aligned_to(args.decay_up, 16) &&
            shared <= 227 * 1024;
 }
 
@@ -1742,8 +1757,26 @@ cudaError_t launch_typed(cudaStream_t stream, const DeltaRuleLaunch& launch) {
 bool delta_rule_needs_scratch(uint32_t dim) { return dim > 128; }
 
 cudaError_t launch_delta_rule(cudaStream_t stream, const DeltaRuleLaunch& launch) {
-    return launch.type == Activation::kF32 ? launch_typed<float>(stream, launch)
-                                           : launch_typed<__nv_bfloat16>(stream, launch);
+    const auto run = [&](const DeltaRuleLaunch& part) {
+        return part.type == Activation::kF32 ? launch_typed<float>(stream, part)
+                                             : launch_typed<__nv_bfloat16>(stream, part);
+    };
+    if (launch.segments.offsets == nullptr || launch.decode_tokens == 0) {
+        return run(launch);
+    }
+    DeltaRuleLaunch decodes = launch;
+    decodes.segments.offsets = nullptr;
+    decodes.segments.num_segments = launch.decode_tokens;
+    decodes.segments.num_tokens = launch.decode_tokens;
+    const cudaError_t status = run(decodes);
+    if (status != cudaSuccess || launch.decode_tokens == launch.segments.num_segments) {
+        return status;
+    }
+    DeltaRuleLaunch prompts = launch;      // segment offsets are absolute token indices
+    prompts.segments.offsets += launch.decode_tokens;
+    prompts.segments.slots += launch.decode_tokens;
+    prompts.segments.num_segments -= launch.decode_tokens;
+    return run(prompts);
 }
 
 }  // namespace lfm25

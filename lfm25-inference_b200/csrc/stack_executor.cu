@@ -216,6 +216,7 @@ int32_t enqueue(lfm25_stack_executor* self, const Step& step) {
             lfm25::DeltaRuleLaunch delta;
             delta.type = self->type;
             delta.segments = step.segments;
+            delta.decode_tokens = step.segments.offsets != nullptr ? step.decode_tokens : 0;
             delta.heads = layer.heads;
             delta.dim = layer.dim;
             delta.rank = layer.rank;

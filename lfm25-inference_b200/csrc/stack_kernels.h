@@ -138,6 +138,7 @@ cudaError_t launch_stack_attention(cudaStream_t stream, const StackAttentionLaun
 struct DeltaRuleLaunch {
     Activation type;
     StackSegments segments;
+    size_t decode_tokens;          // the first decode_tokens segments hold one token each
     uint32_t heads, dim, rank;
     const void* projected;
     size_t pitch;
