@@ -60,15 +60,16 @@ __device__ __forceinline__ void residual_values(const ResidualNormConvArgs& args
 // first tokens of the segment, the record.  Only the segment's first tile touches the record: it reads it for its own
 // first rows and replaces it afterwards, so no other CTA depends on the order.
 // GROUP threads share a row: the whole CTA when a tile is one row (decode), one warp otherwise.
-// HELD: a row fits the registers of its threads (8 vectors each), so that it is read once.
+// HELD: a row fits the registers of its threads (one vector each), so that it is read once.
 // TAPS: number of taps known at compile time (0 = any), whose weights and window then stay in registers.
 template <typename T, int VEC, int GROUP, bool HELD, int TAPS>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, GROUP == 32 ? 3 : 1)
 residual_norm_conv_kernel(const ResidualNormConvArgs args, const T* __restrict__ update, T* __restrict__ mixed_out,
                           T* __restrict__ ff_out) {
     pdl_launch_dependents();
     pdl_wait();
-    constexpr int kHeld = HELD ? (GROUP == 32 ? 8 : 1) : 1;
+    static_assert(!HELD || GROUP == kThreads, "a row is held by a whole CTA");
+    constexpr int kHeld = 1;
     extern __shared__ __align__(16) unsigned char shared_raw[];
     __shared__ float scratch[kThreads / 32];
     T* rows = reinterpret_cast<T*>(shared_raw);      // [taps - 1 + tile_rows][width]
@@ -457,11 +458,11 @@ cudaError_t launch_rnc(cudaStream_t stream, const ResidualNormConvLaunch& launch
     const bool single = launch.segments.offsets == nullptr;
     const size_t history = launch.taps - 1;
     const size_t row_bytes = launch.width * sizeof(T);
-    // rows per tile: 13 where they and their history fit half of an SM's shared memory (with three rows of history that
-    // is two per warp), never fewer than the history
+    // rows per tile: with their history one row per warp (measured best at three CTAs per SM, more in flight than with
+    // rows held in registers), never fewer than the history
     size_t rows = 1;
     if (!single) {
-        rows = history > 13 ? history : 16 - std::min<size_t>(history, 3);
+        rows = history >= 4 ? std::max<size_t>(history, 8) : 8 - history;
         while (rows > 1 && rows > history && (rows + history) * row_bytes > kMaxSharedBytes / 2 - 1024) --rows;
     }
     const size_t shared = (rows + history) * row_bytes;
@@ -481,9 +482,9 @@ cudaError_t launch_rnc(cudaStream_t stream, const ResidualNormConvLaunch& launch
     } else if (launch.width > 2048) {
         kernel = single ? residual_norm_conv_kernel<T, 8, 256, false, 0> : residual_norm_conv_kernel<T, 8, 32, false, 0>;
     } else if (launch.taps == 4) {
-        kernel = single ? residual_norm_conv_kernel<T, 8, 256, true, 4> : residual_norm_conv_kernel<T, 8, 32, true, 4>;
+        kernel = single ? residual_norm_conv_kernel<T, 8, 256, true, 4> : residual_norm_conv_kernel<T, 8, 32, false, 4>;
     } else {
-        kernel = single ? residual_norm_conv_kernel<T, 8, 256, true, 0> : residual_norm_conv_kernel<T, 8, 32, true, 0>;
+        kernel = single ? residual_norm_conv_kernel<T, 8, 256, true, 0> : residual_norm_conv_kernel<T, 8, 32, false, 0>;
     }
     if (shared > 48 * 1024) {
         const cudaError_t status = cudaFuncSetAttribute(reinterpret_cast<const void*>(kernel),
