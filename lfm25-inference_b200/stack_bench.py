@@ -131,11 +131,12 @@ def rooflines(node, times, tokens, keys, segments, hbm_gbs, tensor_tflops, fp32_
     return out
 
 
-def decode_case(device, stream, sequences: int, contexts, steps: int, node: dict, hbm: float, tensor: float) -> dict:
-    """Decode steps of both models replayed from their graphs on the same batch."""
+def decode_case(device, sequences: int, contexts, steps: int, node: dict, hbm: float, tensor: float,
+                beside_lfm2: bool = True) -> dict:
+    """Decode steps replayed from their graphs, of the stack and, on the same batch, of the LFM2 model."""
     batch = workloads.ragged_decode_batch(1, sequences, contexts[0], contexts[1],
                                           sequences * (contexts[1] // 16 + 8) + 64, 64)
-    token_ids = np.random.default_rng(3).integers(0, lfm_model.VOCAB, size=sequences).astype(np.uint32)
+    token_ids = np.random.default_rng(3).integers(0, node["vocab"], size=sequences).astype(np.uint32)
     context = int(batch.contexts.max()) + 64
     out = {"sequences": sequences, "contexts": list(contexts)}
 
@@ -150,13 +151,18 @@ def decode_case(device, stream, sequences: int, contexts, steps: int, node: dict
     device_batch = fixed_batch()
     milliseconds = timed_ms(lambda: executor.step_graph(device_batch, advance=False), steps)
     times = kernel_times(lambda: executor.step_graph(device_batch, advance=False))
-    keys = float((batch.positions(0).astype(np.float64) + 1).sum())
+    limit = next(layer["mixer"]["mask"]["size"] for layer in node["layers"] if layer["type"] == "attention")
+    keys = float((batch.positions(0).astype(np.float64) % limit + 1).sum())
     out["stack"] = {"ms_per_step": milliseconds, "tok_s": sequences / milliseconds * 1e3,
                     "kernels": {name: [count, round(micros, 2)] for name, (count, micros) in times.items()},
                     "rooflines": rooflines(node, times, sequences, keys, sequences, hbm, tensor),
                     "launches": executor.graph_kernels(), "weight_bytes": model.weight_bytes()}
     executor.close()
     del model
+    if not beside_lfm2:
+        blaslt.close()
+        torch.cuda.empty_cache()
+        return out
     reference = lfm_model.RandomModel(7, device, batch.num_pages, sequences, fp8_policy=False)
     closest = lfm_model.DecodeExecutor(blaslt, sequences)
     device_batch = fixed_batch()
@@ -186,13 +192,13 @@ def _lfm2_rooflines(times, tokens, keys, segments, hbm, tensor) -> dict:
     return out
 
 
-def prefill_case(device, stream, prefixes, chunk: int, steps: int, node: dict, hbm: float, tensor: float) -> dict:
+def prefill_case(device, prefixes, chunk: int, steps: int, node: dict, hbm: float, tensor: float,
+                 beside_lfm2: bool = True) -> dict:
     """Mixed steps of `chunk` new tokens behind each of `prefixes` cached ones."""
     pages = sum((prefix + chunk + 15) // 16 for prefix in prefixes)
     batch = workloads.mixed_step_batch(5, prefixes, [chunk] * len(prefixes), pages)
-    token_ids = np.random.default_rng(5).integers(0, lfm_model.VOCAB, size=batch.num_tokens).astype(np.uint32)
-    size = node["layers"][next(i for i, layer in enumerate(node["layers"]) if layer["type"] == "attention")]
-    limit = size["mixer"]["mask"]["size"]
+    token_ids = np.random.default_rng(5).integers(0, node["vocab"], size=batch.num_tokens).astype(np.uint32)
+    limit = next(layer["mixer"]["mask"]["size"] for layer in node["layers"] if layer["type"] == "attention")
     positions = batch.positions.astype(np.float64)
     out = {"prefixes": list(prefixes), "chunk": chunk, "attention_chunk": limit}
     blaslt = ops.BlasLt()
@@ -208,6 +214,10 @@ def prefill_case(device, stream, prefixes, chunk: int, steps: int, node: dict, h
                     "rooflines": rooflines(node, times, batch.num_tokens, keys, batch.num_segments, hbm, tensor)}
     executor.close()
     del model
+    if not beside_lfm2:
+        blaslt.close()
+        torch.cuda.empty_cache()
+        return out
     reference = lfm_model.RandomModel(7, device, pages, batch.num_segments, fp8_policy=False)
     closest = lfm_model.DecodeExecutor(blaslt, batch.num_tokens, maximum_segments=batch.num_segments)
     device_batch = lfm_model.RaggedBatch(device, batch, token_ids)
@@ -224,13 +234,27 @@ def prefill_case(device, stream, prefixes, chunk: int, steps: int, node: dict, h
     return out
 
 
+# Other sizes, without a counterpart: heads of 128 with chunks shorter than the contexts, one smaller and one larger width.
+OTHER_SIZES = {
+    "width 1024": dict(width=1024, num_layers=8, attention_layers=(2, 5), heads=8, kv_heads=2, dim=128, delta_heads=16,
+                       ff=6144, vocab=32768, chunk=512),
+    "width 4096": dict(width=4096, num_layers=8, attention_layers=(2, 5), heads=32, kv_heads=8, dim=128, delta_heads=32,
+                       delta_dim=128, ff=24576, vocab=65536, chunk=1024),
+}
+
+
 def run(device, steps: int, hbm: float, tensor: float) -> dict:
     node = config()
-    stream = torch.cuda.Stream(device=device)
-    with torch.cuda.stream(stream):
-        decode = [decode_case(device, stream, sequences, contexts, steps, node, hbm, tensor)
+    few = max(steps // 8, 4)
+    with torch.cuda.stream(torch.cuda.Stream(device=device)):
+        decode = [decode_case(device, sequences, contexts, steps, node, hbm, tensor)
                   for sequences, contexts in ((1, (1024, 1024)), (32, (128, 4096)), (128, (128, 4096)))]
-        prefill = [prefill_case(device, stream, [0] * 8, 512, max(steps // 8, 4), node, hbm, tensor),
-                   prefill_case(device, stream, [0], 4096, max(steps // 8, 4), node, hbm, tensor),
-                   prefill_case(device, stream, [1024] * 8, 512, max(steps // 8, 4), node, hbm, tensor)]
-    return {"decode": decode, "prefill": prefill}
+        prefill = [prefill_case(device, [0] * 8, 512, few, node, hbm, tensor),
+                   prefill_case(device, [0], 4096, few, node, hbm, tensor),
+                   prefill_case(device, [1024] * 8, 512, few, node, hbm, tensor)]
+        others = {}
+        for name, sizes in OTHER_SIZES.items():
+            other = config(**sizes)
+            others[name] = {"decode": decode_case(device, 64, (128, 4096), steps, other, hbm, tensor, False),
+                            "prefill": prefill_case(device, [0] * 8, 512, few, other, hbm, tensor, False)}
+    return {"decode": decode, "prefill": prefill, "other_sizes": others}

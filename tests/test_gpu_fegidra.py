@@ -399,3 +399,43 @@ def test_captured_steps_match_eager_ones(device, mixed_case):
             executor.close()
             blaslt.close()
     assert np.array_equal(produced[0], produced[1])
+
+
+def test_command_line_and_trace_replay(device, mixed_case, tmp_path):
+    """A model folder through the two programs, each in a process of its own."""
+    import json
+    import os
+    import subprocess
+    import sys
+
+    import torch
+
+    from lfm25_inference_b200 import checkpoint
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    config, tensors, tokens, want = mixed_case
+    (tmp_path / "config.json").write_text(json.dumps(config))
+    checkpoint.write(str(tmp_path / "model.safetensors"),
+                     {name: torch.from_numpy(values).to(torch.bfloat16) for name, values in tensors.items()})
+
+    def run(program, *arguments, **options):
+        done = subprocess.run([sys.executable, os.path.join(root, "bin", program), *arguments], capture_output=True,
+                              text=True, timeout=300, **options)
+        assert done.returncode == 0, done.stderr[-2000:]
+        return done.stdout
+
+    prompts = [tokens[:9], tokens[20:61]]
+    produced = run("lfm25", "generate", "--model", str(tmp_path), "--dtype", "float32", "--max-new-tokens", "8",
+                   *[word for prompt in prompts for word in ("--tokens", ",".join(map(str, prompt)))]).split()
+    for prompt, line in zip(prompts, produced):
+        expected, margins = greedy_with_margin(config, tensors, prompt, 8)
+        sure = next((i for i, margin in enumerate(margins) if margin < 1e-3), len(expected))
+        assert [int(word) for word in line.split(",")][:sure] == expected[:sure] and sure > 2
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": tokens[:70].tolist(), "want": [3, 69]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": tokens[70:71].tolist(), "want": [0]}], "end": ["a"]},
+             {"step": 2, "entries": [{"id": "a", "tokens": tokens[:2].tolist(), "want": [1]}], "end": ["a"]}]
+    out = run("trace_run", "--model", str(tmp_path), "--dtype", "float32", "--out", str(tmp_path), "--max-tokens", "80",
+              input="".join(json.dumps(step) + "\n" for step in steps))
+    assert [line for line in out.splitlines() if line.startswith("done")] == ["done 0", "done 1", "done 2"]
+    for step, places in ((0, [3, 69]), (1, [70]), (2, [1])):
+        got = np.fromfile(tmp_path / f"{step}.f32", dtype="<f4").reshape(len(places), config["vocab"])
+        assert cases.relative_error(got, want[places]).max() <= cases.LIMITS["float32"]
