@@ -572,7 +572,12 @@ typedef struct lfm25_ragged_batch {
      * context among them) and only the remaining segments in the hybrid kernel.  0: everything in the hybrid kernel. */
     size_t num_decode_segments;
     size_t max_decode_context_tokens;
+    /* Extension: the context lengths (last position + 1) of the segments behind the decode ones, each rounded up to
+     * LFM25_CONTEXT_ROWS and added up; 0 = not known.  Attention that lays a prompt's whole context out in scratch needs
+     * it to size its launches. */
+    size_t prompt_context_rows;
 } lfm25_ragged_batch;
+#define LFM25_CONTEXT_ROWS 64
 /* An executor for steps of up to maximum_tokens tokens (<= 8192) in up to maximum_segments sequences (<= 256):
  * lfm25_decode_executor_create is the case maximum_tokens == maximum_segments. */
 int32_t lfm25_decode_executor_create_ragged(lfm25_blaslt* blaslt, size_t maximum_tokens, size_t maximum_segments,
@@ -632,9 +637,12 @@ const void* lfm25_decode_executor_logits(const lfm25_decode_executor* executor);
 /* ------------------------------------------------------------------------------------------
  * Layer-stack models: a decoder described layer by layer, for designs other than the one above
  * ------------------------------------------------------------------------------------------
- * A layer is x <- x + (mixer(h + conv(h)) + ff(n)) with h = norm(x) * mixer_norm, n = norm(x) * ff_norm and conv a causal
- * per-channel convolution over time; the mixer is attention over the paged cache or a recurrence over a state that
- * every request slot carries.  Every size and constant is a field; bf16 weights, activations in bf16 or f32, and the
+ * The layers of a model have one of two arrangements.  With N(x) = x / sqrt(mean(x^2) + eps) and N(x; w) =
+ * N(x) * (norm_shift + w):
+ *   parallel   x <- x + (mixer(h + conv(h)) + ff(n)),  h = N(x; mixer_norm), n = N(x; ff_norm), conv a causal
+ *              per-channel convolution over time
+ *   sandwich   x <- x + N(mixer(N(x; mixer_norm)); mixer_post_norm),  then  x <- x + N(ff(N(x; ff_norm)); ff_post_norm)
+ * The mixer is attention over the paged cache or a recurrence over a state that every request slot carries.  Every size and constant is a field; bf16 weights, activations in bf16 or f32, and the
  * residual stream, norms, rotation, softmax and recurrent state in f32 in both.  Unlike lfm25_model, which fixes the
  * LFM2 shapes, nothing here is a compile-time constant except the page size (16 tokens). */
 
@@ -642,6 +650,12 @@ const void* lfm25_decode_executor_logits(const lfm25_decode_executor* executor);
 #define LFM25_ACTIVATION_F32 1u
 #define LFM25_MIXER_ATTENTION 0u
 #define LFM25_MIXER_GENERAL_DELTA 1u
+#define LFM25_MIXER_LATENT_ATTENTION 2u
+#define LFM25_MIXER_STATE_SPACE 3u
+#define LFM25_BLOCK_PARALLEL 0u
+#define LFM25_BLOCK_SANDWICH 1u
+#define LFM25_FEED_FORWARD_POLY_NORM 0u
+#define LFM25_FEED_FORWARD_SQUARED_RELU 1u
 
 /* Matrix [n, k] in bf16; rows beyond the layer's own columns (up to n) are zero. */
 typedef struct lfm25_stack_linear {
@@ -654,14 +668,24 @@ typedef struct lfm25_stack_layer {
     uint32_t mixer;                    /* LFM25_MIXER_* */
     const void* mixer_norm;            /* bf16 [width] */
     const void* ff_norm;               /* bf16 [width]; NULL with ff == 0 */
-    const void* conv;                  /* bf16 [conv_taps, width], tap-major, last row = current token */
-    size_t conv_offset;                /* of [conv_taps - 1, width] activations in a request slot's record (bytes) */
-    /* projections of the mixer input, one matrix: attention q | k | v; delta rule r | k | v | g | a | z */
+    /* parallel arrangement: the input convolution, bf16 [conv_taps, width]; state-space mixer: the convolution of x | B |
+     * C, bf16 [conv_taps, channels].  Tap-major, last row = current token. */
+    const void* conv;
+    size_t conv_offset;                /* of its last conv_taps - 1 inputs (activations) in a request slot's record */
+    uint32_t conv_taps;
+    /* projections of the mixer input, one matrix: attention q | k | v; delta rule r | k | v | g | a | z; latent attention
+     * query latent | key/value latent and rotated key | gate, each section starting at a multiple of 8 columns (the
+     * second one missing with shared_cache); state space z | x | B | C | dt */
     lfm25_stack_linear projection;
-    /* output projection of the mixer beside that of the feed-forward: [width, mixer columns + ff] */
+    /* output projection of the mixer; parallel arrangement: beside that of the feed-forward, [width, mixer columns + ff] */
     lfm25_stack_linear output;
-    /* feed-forward: up -> PolyNorm a N(z) + b N(z^2) + c N(z^3) + e -> (part of output); ff == 0: none */
+    /* feed-forward, ff == 0: none.  PolyNorm a N(z) + b N(z^2) + c N(z^3) + e or relu(z)^2 between up and down (parallel
+     * arrangement: the part of output) */
     uint32_t ff;
+    uint32_t ff_activation;            /* LFM25_FEED_FORWARD_* */
+    lfm25_stack_linear down;           /* sandwich arrangement: [width, up.n] */
+    const void* mixer_post_norm;       /* sandwich arrangement: bf16 [width] */
+    const void* ff_post_norm;
     lfm25_stack_linear up;
     float poly[4];
     uint32_t heads;
@@ -685,16 +709,37 @@ typedef struct lfm25_stack_layer {
     const void* removal_bias;          /* bf16 [heads * dim] */
     const void* head_norm;             /* bf16 [heads * dim] */
     size_t state_offset;               /* of f32 [heads, dim (value), dim (key)] in a request slot's record (bytes) */
+    /* latent attention: queries of heads x (dim + rot_dim), the last rot_dim rotated on their first rot_dims entries; the
+     * cache holds the normed latent, activations [num_pages, 16, kv_rank] in value_cache, and the rotated key part that
+     * all heads share, [num_pages, 16, rot_dim] in key_cache.  The output is gated by sigmoid of the gate section. */
+    uint32_t q_rank;
+    uint32_t kv_rank;
+    uint32_t rot_dim;
+    uint32_t shared_cache;             /* 1: the caches are another layer's, filled earlier in the step */
+    const void* query_latent_norm;     /* bf16 [q_rank] */
+    const void* latent_norm;           /* bf16 [kv_rank] */
+    lfm25_stack_linear query_up;       /* [heads * (dim + rot_dim), q_rank] */
+    lfm25_stack_linear latent_up;      /* [heads * dim key rows, then heads * vdim value rows, kv_rank] */
+    /* state-space mixer (heads, vdim, state_offset of f32 [heads, state_size, vdim], head_norm [heads * vdim]) */
+    uint32_t groups;                   /* of B and C; head h uses group h / (heads / groups) */
+    uint32_t state_size;
+    uint32_t norm_groups;              /* equal parts of the gated output that are normed on their own */
+    const void* conv_bias;             /* bf16 [channels] */
+    const void* step_bias;             /* bf16 [heads]: dt = softplus(raw + bias) */
+    const void* log_rate;              /* bf16 [heads]: the state decays by exp(-exp(log_rate) dt) */
+    const void* skip;                  /* bf16 [heads] */
 } lfm25_stack_layer;
 
 typedef struct lfm25_stack_model {
     uint32_t num_layers;
     const lfm25_stack_layer* layers;   /* host array */
     uint32_t activation;               /* LFM25_ACTIVATION_* */
-    uint32_t conv_taps;
+    uint32_t block;                    /* LFM25_BLOCK_* */
     size_t vocab;
     size_t width;
     float norm_eps;
+    float norm_shift;                  /* sandwich arrangement: added to the stored weights of norms over the width */
+    float logit_softcap;               /* logits <- cap * tanh(logits / cap); 0 = none */
     const void* embedding;             /* bf16 [vocab, width] */
     const void* final_norm;            /* bf16 [width] */
     lfm25_stack_linear head;           /* [>= vocab, width] */

@@ -97,7 +97,10 @@ class RaggedBatch(ctypes.Structure):
                 ("block_tables", ctypes.c_void_p), ("block_table_stride", ctypes.c_size_t),
                 ("block_table_rows", ctypes.c_size_t), ("num_tokens", ctypes.c_size_t),
                 ("num_segments", ctypes.c_size_t), ("num_decode_segments", ctypes.c_size_t),
-                ("max_decode_context_tokens", ctypes.c_size_t)]
+                ("max_decode_context_tokens", ctypes.c_size_t), ("prompt_context_rows", ctypes.c_size_t)]
+
+
+CONTEXT_ROWS = 64
 
 
 class PrefixCacheSnapshot(ctypes.Structure):
@@ -200,7 +203,9 @@ HybridAttentionLaunch = _launch_struct("HybridAttentionLaunch", [
     "#query_token_stride", "#kv_token_stride"])
 
 ACTIVATION_BF16, ACTIVATION_F32 = 0, 1
-MIXER_ATTENTION, MIXER_GENERAL_DELTA = 0, 1
+MIXER_ATTENTION, MIXER_GENERAL_DELTA, MIXER_LATENT_ATTENTION, MIXER_STATE_SPACE = 0, 1, 2, 3
+BLOCK_PARALLEL, BLOCK_SANDWICH = 0, 1
+FEED_FORWARD_POLY_NORM, FEED_FORWARD_SQUARED_RELU = 0, 1
 
 
 class StackLinear(ctypes.Structure):
@@ -209,21 +214,29 @@ class StackLinear(ctypes.Structure):
 
 class StackLayer(ctypes.Structure):
     _fields_ = ([("mixer", ctypes.c_uint32), ("mixer_norm", ctypes.c_void_p), ("ff_norm", ctypes.c_void_p),
-                 ("conv", ctypes.c_void_p), ("conv_offset", ctypes.c_size_t), ("projection", StackLinear),
-                 ("output", StackLinear), ("ff", ctypes.c_uint32), ("up", StackLinear), ("poly", ctypes.c_float * 4)]
+                 ("conv", ctypes.c_void_p), ("conv_offset", ctypes.c_size_t), ("conv_taps", ctypes.c_uint32),
+                 ("projection", StackLinear), ("output", StackLinear), ("ff", ctypes.c_uint32),
+                 ("ff_activation", ctypes.c_uint32), ("down", StackLinear), ("mixer_post_norm", ctypes.c_void_p),
+                 ("ff_post_norm", ctypes.c_void_p), ("up", StackLinear), ("poly", ctypes.c_float * 4)]
                 + [(name, ctypes.c_uint32) for name in ("heads", "dim", "kv_heads", "vdim", "rot_dims", "chunk")]
                 + [("scale", ctypes.c_float)]
                 + [(name, ctypes.c_void_p) for name in ("inv_freq", "bias", "query_norm", "key_norm", "key_cache",
                                                         "value_cache")]
                 + [("rank", ctypes.c_uint32)]
                 + [(name, ctypes.c_void_p) for name in ("decay_up", "decay_base", "removal_bias", "head_norm")]
-                + [("state_offset", ctypes.c_size_t)])
+                + [("state_offset", ctypes.c_size_t)]
+                + [(name, ctypes.c_uint32) for name in ("q_rank", "kv_rank", "rot_dim", "shared_cache")]
+                + [("query_latent_norm", ctypes.c_void_p), ("latent_norm", ctypes.c_void_p), ("query_up", StackLinear),
+                   ("latent_up", StackLinear)]
+                + [(name, ctypes.c_uint32) for name in ("groups", "state_size", "norm_groups")]
+                + [(name, ctypes.c_void_p) for name in ("conv_bias", "step_bias", "log_rate", "skip")])
 
 
 class StackModel(ctypes.Structure):
     _fields_ = [("num_layers", ctypes.c_uint32), ("layers", _P(StackLayer)), ("activation", ctypes.c_uint32),
-                ("conv_taps", ctypes.c_uint32), ("vocab", ctypes.c_size_t), ("width", ctypes.c_size_t),
-                ("norm_eps", ctypes.c_float), ("embedding", ctypes.c_void_p), ("final_norm", ctypes.c_void_p),
+                ("block", ctypes.c_uint32), ("vocab", ctypes.c_size_t), ("width", ctypes.c_size_t),
+                ("norm_eps", ctypes.c_float), ("norm_shift", ctypes.c_float), ("logit_softcap", ctypes.c_float),
+                ("embedding", ctypes.c_void_p), ("final_norm", ctypes.c_void_p),
                 ("head", StackLinear), ("records", ctypes.c_void_p), ("record_bytes", ctypes.c_size_t),
                 ("num_request_slots", ctypes.c_size_t), ("num_pages", ctypes.c_size_t)]
 

@@ -137,6 +137,7 @@ int32_t enqueue_step(lfm25_engine* self, const StepShape& shape) {
     size_t tokens = 0;
     size_t decode_segments = 0;
     size_t decode_context = 0;
+    size_t prompt_rows = 0;
     bool leading = true;
     uint32_t* meta = self->h_meta;
     uint32_t* h_positions = meta + self->max_tokens;
@@ -158,6 +159,8 @@ int32_t enqueue_step(lfm25_engine* self, const StepShape& shape) {
             decode_context = std::max(decode_context, shape.prefixes[segment] + 1);
         } else {
             leading = false;
+            const size_t context = shape.prefixes[segment] + shape.chunks[segment];
+            prompt_rows += (context + LFM25_CONTEXT_ROWS - 1) / LFM25_CONTEXT_ROWS * LFM25_CONTEXT_ROWS;
         }
     }
     h_offsets[segments] = static_cast<uint32_t>(tokens);
@@ -198,6 +201,7 @@ int32_t enqueue_step(lfm25_engine* self, const StepShape& shape) {
     batch.num_segments = segments;
     batch.num_decode_segments = decode_segments;
     batch.max_decode_context_tokens = decode_context;
+    batch.prompt_context_rows = prompt_rows;
     return self->backend->mixed(batch, num_rows);
 }
 

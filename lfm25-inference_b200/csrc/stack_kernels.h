@@ -61,20 +61,64 @@ cudaError_t launch_residual_norm_rows(cudaStream_t stream, Activation type, cons
                                       const void* weight, const uint32_t* rows, void* out, size_t num_rows,
                                       size_t num_tokens, size_t width, float eps);
 
+// With N(x; w) = x / sqrt(mean(x^2) + eps) * (shift + w), per row:
+//   x = residual (or the embedding row of token_ids), plus N(update; post_norm) when there is an update
+//   residual_out = x,  out = N(x; norm)            -- either may be left out
+// Row i reads row rows[i] (rows == nullptr: i) of residual and update; residual_out may be the buffer of residual.
+struct ResidualPostNormLaunch {
+    Activation type;
+    const float* residual;         // [T, width]; unused with an embedding
+    const void* update;            // [T, width] activations, or nullptr
+    const void* post_norm;         // bf16 [width]
+    const uint32_t* token_ids;     // [T] with `embedding`, else nullptr
+    const void* embedding;         // bf16 [vocab, width] or nullptr
+    size_t vocab;
+    const void* norm;              // bf16 [width]
+    const uint32_t* rows;
+    float* residual_out;           // [num_rows, width] or nullptr
+    void* out;                     // [num_rows, width] activations or nullptr
+    size_t num_rows;
+    size_t num_tokens;
+    size_t width;
+    float shift;
+    float eps;
+};
+cudaError_t launch_residual_post_norm(cudaStream_t stream, const ResidualPostNormLaunch& launch);
+
+// z <- relu(z)^2 in place
+cudaError_t launch_squared_relu(cudaStream_t stream, Activation type, void* z, size_t count);
+
 // out[t, c] = a N(z)[c] + b N(z^2)[c] + c N(z^3)[c] + e with N the unweighted RMS norm of the row; columns
 // width .. width + pad - 1 of `out` are set to zero.
 cudaError_t launch_poly_norm(cudaStream_t stream, Activation type, const void* z, size_t z_pitch, void* out,
                              size_t out_pitch, size_t rows, size_t width, size_t pad, const float coefficients[4],
                              float eps);
 
-// Greedy choice: index of the row's largest logit, the lowest index among equals; NaN never wins.
-cudaError_t launch_argmax_rows(cudaStream_t stream, Activation type, const void* logits, size_t pitch,
-                               uint32_t* sampled, size_t rows, size_t vocab);
+// Greedy choice: index of the row's largest logit, the lowest index among equals; NaN never wins.  softcap > 0: the
+// logits become softcap * tanh(logits / softcap) first, in place.
+cudaError_t launch_argmax_rows(cudaStream_t stream, Activation type, void* logits, size_t pitch, uint32_t* sampled,
+                               size_t rows, size_t vocab, float softcap);
 
 // y[m, n] = sum_k x[m, k] w[n, k] with plain 32-bit multiply-adds: the matrix product of the f32 activation type and
 // of bf16 shapes that the tensor-core paths cannot take.
 cudaError_t launch_linear_simt(cudaStream_t stream, Activation type, const void* x, const void* weight, void* y,
                                size_t m, size_t n, size_t k);
+
+// One matrix product per head: y[t, h, n] = sum_k x[t, h, k] w[h, n, k] (gate: times sigmoid(gate[t, h * n_size + n])).
+struct HeadLinearLaunch {
+    Activation type;
+    const void* x;                 // activations: token t, head h at x + t * x_pitch + h * x_head
+    size_t x_pitch, x_head;
+    const void* weight;            // bf16: head h, output n, input k at weight + h * w_head + n * w_n + k * w_k
+    size_t w_head, w_n, w_k;       // w_n or w_k is 1
+    void* y;                       // activations: y + t * y_pitch + h * n
+    size_t y_pitch;
+    const void* gate;              // activations, token t at gate + t * gate_pitch, or nullptr
+    size_t gate_pitch;
+    size_t tokens, n, k;
+    uint32_t heads;
+};
+cudaError_t launch_head_linear(cudaStream_t stream, const HeadLinearLaunch& launch);
 
 // ---------------------------------------------------------------------------------------------------- attention
 
@@ -129,6 +173,169 @@ struct StackAttentionLaunch {
     size_t out_pitch;
 };
 cudaError_t launch_stack_attention(cudaStream_t stream, const StackAttentionLaunch& launch);
+
+// -------------------------------------------------------------------------------------------- latent attention
+
+struct LatentAttentionShape {
+    uint32_t heads, dim, rot_dim, vdim, kv_rank;
+    float scale;
+};
+
+// The projections of latent attention: out = N(query latent) * query_norm; N(latent) * latent_norm and the rotated key
+// part into the paged cache.  `projected` rows hold query latent | latent | key part, the latter two from `latent_column`.
+struct LatentProjectionLaunch {
+    Activation type;
+    const void* projected;
+    size_t pitch;
+    uint32_t q_rank, kv_rank, rot_dim, rot_dims;
+    size_t latent_column;
+    bool append;                   // false: the cache is another layer's, only the query latent is wanted
+    const void* query_norm;        // bf16 [q_rank]
+    const void* latent_norm;       // bf16 [kv_rank]
+    const float* inv_freq;         // f32 [rot_dims / 2]
+    const uint32_t* positions;
+    const int64_t* physical_slots; // negative = do not append
+    void* query_out;               // [T, q_rank]
+    void* latent_cache;            // [pages, 16, kv_rank]
+    void* key_cache;               // [pages, 16, rot_dim]
+    size_t num_tokens;
+    size_t num_pages;
+    float eps;
+};
+cudaError_t launch_latent_projection(cudaStream_t stream, const LatentProjectionLaunch& launch);
+
+// Rotates entries 0 .. rot_dims - 1 behind the first `dim` of every head, in place; query [T, heads, dim + rot_dim] in rows
+// `pitch` apart.
+cudaError_t launch_rotate_queries(cudaStream_t stream, Activation type, void* query, size_t pitch, const float* inv_freq,
+                                  const uint32_t* positions, size_t tokens, uint32_t heads, uint32_t dim,
+                                  uint32_t rot_dim, uint32_t rot_dims);
+
+// Attention against the latents themselves: the key up-projection has been moved to the query side, so one latent vector
+// and one rotated key per token serve all heads, and the output is the weighted latent of every head.
+struct LatentAttentionLaunch {
+    Activation type;
+    LatentAttentionShape shape;
+    const void* absorbed;          // [T, heads, kv_rank]
+    const void* query;             // [T, heads, dim + rot_dim], rows query_pitch apart: the last rot_dim, rotated
+    size_t query_pitch;
+    const void* latent_cache;
+    const void* key_cache;
+    const uint32_t* block_tables;
+    size_t block_table_stride;
+    size_t block_table_rows;
+    size_t num_pages;
+    const uint32_t* request_slots; // [T]
+    const uint32_t* positions;     // [T]
+    size_t tokens;
+    size_t context;                // longest context among them when known, else 0
+    unsigned int* status;
+    void* out;                     // [T, heads, kv_rank]
+};
+cudaError_t launch_latent_attention(cudaStream_t stream, const LatentAttentionLaunch& launch);
+
+// Row of a step's context scratch at which each segment's keys start: segment s takes ceil(context / 64) * 64 rows in
+// order; the segments from `first_segment` on.  bases has num_segments + 1 entries.
+cudaError_t launch_context_bases(cudaStream_t stream, const StackSegments& segments, const uint32_t* positions,
+                                 size_t first_segment, uint32_t* bases);
+
+// Copies the cached latents and rotated keys of those segments' contexts into contiguous rows; rows behind a context are
+// cleared.
+struct GatherContextLaunch {
+    Activation type;
+    StackSegments segments;
+    size_t first_segment;
+    const uint32_t* bases;
+    const uint32_t* positions;
+    const uint32_t* block_tables;
+    size_t block_table_stride;
+    size_t block_table_rows;
+    size_t num_pages;
+    uint32_t kv_rank, rot_dim;
+    const void* latent_cache;
+    const void* key_cache;
+    void* latents;                 // [rows, kv_rank]
+    void* keys;                    // [rows, rot_dim]
+    size_t rows;
+};
+cudaError_t launch_gather_context(cudaStream_t stream, const GatherContextLaunch& launch);
+
+// Prompt attention over keys and values that were formed from the gathered latents: `expanded` rows hold heads * dim key
+// columns, then heads * vdim value columns.
+struct ExpandedAttentionLaunch {
+    Activation type;
+    LatentAttentionShape shape;
+    const void* query;             // [T, heads, dim + rot_dim], rows query_pitch apart
+    size_t query_pitch;
+    const void* expanded;
+    size_t expanded_pitch;
+    const void* keys;              // [rows, rot_dim]
+    const uint32_t* bases;
+    size_t rows;
+    size_t first_segment;
+    StackSegments segments;
+    const uint32_t* positions;
+    const void* gate;              // activations, token t at gate + t * gate_pitch, heads * vdim columns
+    size_t gate_pitch;
+    unsigned int* status;
+    void* out;                     // activations, rows out_pitch apart, heads * vdim columns
+    size_t out_pitch;
+};
+bool expanded_attention_supports(Activation type, const LatentAttentionShape& shape, size_t out_pitch, size_t gate_pitch,
+                                 size_t expanded_pitch);
+cudaError_t launch_expanded_attention(cudaStream_t stream, const ExpandedAttentionLaunch& launch);
+
+// ---------------------------------------------------------------------------------------------- state-space mixer
+
+// out[t, c] = silu(sum_j conv[j, c] x[t - taps + 1 + j, c] + bias[c]) over `channels` columns of x; the last taps - 1
+// inputs live in `record` as [taps - 1, channels] activations, oldest first.
+struct ChannelConvLaunch {
+    Activation type;
+    StackSegments segments;
+    const void* x;
+    size_t pitch;
+    const void* conv;              // bf16 [taps, channels]
+    const void* bias;              // bf16 [channels]
+    uint32_t taps;
+    StackRecord record;
+    void* out;                     // [T, channels]
+    size_t channels;
+};
+cudaError_t launch_channel_conv(cudaStream_t stream, const ChannelConvLaunch& launch);
+
+// Per head S <- exp(-exp(log_rate) dt) S + dt B x^T, y = S^T C + skip x with dt = softplus(raw + step_bias); `mixed` rows
+// hold x [heads, vdim] | B [groups, size] | C [groups, size].  State: f32 [heads, size, vdim] in `record`.
+struct StateSpaceLaunch {
+    Activation type;
+    StackSegments segments;
+    size_t decode_tokens;          // the first decode_tokens segments hold one token each
+    uint32_t heads, groups, size, vdim;
+    const void* mixed;
+    size_t mixed_pitch;
+    const void* raw_step;          // activations: token t at raw_step + t * step_pitch, heads columns
+    size_t step_pitch;
+    const void* step_bias;         // bf16 [heads]
+    const void* log_rate;
+    const void* skip;
+    StackRecord record;
+    void* out;                     // [T, heads * vdim]
+};
+constexpr uint32_t kStateSpaceMaxSize = 512;
+cudaError_t launch_state_space(cudaStream_t stream, const StateSpaceLaunch& launch);
+
+// out = N(y silu(z)) * norm, N over each of `groups` equal parts of the row on its own.
+struct GatedGroupNormLaunch {
+    Activation type;
+    const void* y;                 // [T, width]
+    const void* z;                 // activations, rows z_pitch apart
+    size_t z_pitch;
+    const void* norm;              // bf16 [width]
+    void* out;                     // activations, rows out_pitch apart
+    size_t out_pitch;
+    size_t tokens, width;
+    uint32_t groups;
+    float eps;
+};
+cudaError_t launch_gated_group_norm(cudaStream_t stream, const GatedGroupNormLaunch& launch);
 
 // ---------------------------------------------------------------------------------------------------- delta rule
 

@@ -264,6 +264,169 @@ residual_norm_rows_kernel(const float* __restrict__ residual, const T* __restric
     }
 }
 
+struct PostNormArgs {
+    const float* residual;
+    const __nv_bfloat16* post_norm;
+    const uint32_t* token_ids;
+    const __nv_bfloat16* embedding;
+    size_t vocab;
+    const __nv_bfloat16* norm;
+    const uint32_t* rows;
+    float* residual_out;
+    size_t num_tokens;
+    size_t width;
+    float shift;
+    float eps;
+};
+
+// One CTA per row.  HELD: vectors of the row that each thread keeps in registers, so that everything is read once; 0: any
+// width, the row is read again for every pass (residual_out then holds the sum between the passes).
+template <typename T, int VEC, int HELD>
+__global__ void __launch_bounds__(512)
+residual_post_norm_kernel(const PostNormArgs args, const T* __restrict__ update, T* __restrict__ out) {
+    pdl_launch_dependents();
+    __shared__ float scratch[16];
+    pdl_wait();
+    const size_t row = args.rows != nullptr ? args.rows[blockIdx.x] : blockIdx.x;
+    if (row >= args.num_tokens) {
+        return;
+    }
+    const size_t width = args.width;
+    const size_t step = static_cast<size_t>(blockDim.x) * VEC;
+    const __nv_bfloat16* embedding_row = nullptr;
+    if (args.embedding != nullptr) {
+        const size_t id = args.token_ids[row];
+        embedding_row = id < args.vocab ? args.embedding + id * width : nullptr;
+    }
+    auto load_residual = [&](size_t channel, float (&value)[VEC]) {
+        if (args.embedding == nullptr) {
+            load_values<VEC>(args.residual + row * width + channel, value);
+        } else if (embedding_row != nullptr) {
+            load_values<VEC>(embedding_row + channel, value);
+        } else {
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) value[i] = 0.0f;
+        }
+    };
+    auto load_weight = [&](const __nv_bfloat16* weight, size_t channel, float (&value)[VEC]) {
+        load_values<VEC>(weight + channel, value);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) value[i] += args.shift;
+    };
+    auto add_squares = [](const float (&value)[VEC], float& sum) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) sum = fmaf(value[i], value[i], sum);
+    };
+    auto write_residual = [&](size_t channel, const float (&value)[VEC]) {
+        if (args.residual_out != nullptr) store_values<VEC>(args.residual_out + blockIdx.x * width + channel, value);
+    };
+    auto write_out = [&](size_t channel, float (&value)[VEC], float scale) {
+        float weight[VEC];
+        load_weight(args.norm, channel, weight);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) value[i] *= scale * weight[i];
+        store_values<VEC>(out + blockIdx.x * width + channel, value);
+    };
+    if constexpr (HELD > 0) {
+        float held[HELD][VEC];
+#pragma unroll
+        for (int part = 0; part < HELD; ++part) {
+            const size_t channel = part * step + threadIdx.x * VEC;
+            if (channel < width) load_residual(channel, held[part]);
+        }
+        if (update != nullptr) {
+            float add[HELD][VEC], sum = 0.0f;
+#pragma unroll
+            for (int part = 0; part < HELD; ++part) {
+                const size_t channel = part * step + threadIdx.x * VEC;
+                if (channel < width) {
+                    load_values<VEC>(update + row * width + channel, add[part]);
+                    add_squares(add[part], sum);
+                }
+            }
+            const float scale = inverse_rms(block_sum(sum, scratch), width, args.eps);
+#pragma unroll
+            for (int part = 0; part < HELD; ++part) {
+                const size_t channel = part * step + threadIdx.x * VEC;
+                if (channel < width) {
+                    float weight[VEC];
+                    load_weight(args.post_norm, channel, weight);
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) held[part][i] += add[part][i] * scale * weight[i];
+                }
+            }
+        }
+        float sum = 0.0f;
+#pragma unroll
+        for (int part = 0; part < HELD; ++part) {
+            const size_t channel = part * step + threadIdx.x * VEC;
+            if (channel < width) {
+                write_residual(channel, held[part]);
+                add_squares(held[part], sum);
+            }
+        }
+        if (out == nullptr) {
+            return;
+        }
+        const float scale = inverse_rms(block_sum(sum, scratch), width, args.eps);
+#pragma unroll
+        for (int part = 0; part < HELD; ++part) {
+            const size_t channel = part * step + threadIdx.x * VEC;
+            if (channel < width) write_out(channel, held[part], scale);
+        }
+    } else {
+        float post = 0.0f;
+        if (update != nullptr) {
+            float sum = 0.0f;
+            for (size_t channel = threadIdx.x * VEC; channel < width; channel += step) {
+                float add[VEC];
+                load_values<VEC>(update + row * width + channel, add);
+                add_squares(add, sum);
+            }
+            post = inverse_rms(block_sum(sum, scratch), width, args.eps);
+        }
+        auto sum_of = [&](size_t channel, float (&value)[VEC]) {
+            load_residual(channel, value);
+            if (update != nullptr) {
+                float add[VEC], weight[VEC];
+                load_values<VEC>(update + row * width + channel, add);
+                load_weight(args.post_norm, channel, weight);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) value[i] += add[i] * post * weight[i];
+            }
+        };
+        float sum = 0.0f, value[VEC];
+        for (size_t channel = threadIdx.x * VEC; channel < width; channel += step) {
+            sum_of(channel, value);
+            add_squares(value, sum);
+        }
+        const float scale = inverse_rms(block_sum(sum, scratch), width, args.eps);
+        for (size_t channel = threadIdx.x * VEC; channel < width; channel += step) {
+            sum_of(channel, value);
+            write_residual(channel, value);       // the thread that reads this channel again is this one
+            if (out != nullptr) write_out(channel, value, scale);
+        }
+    }
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kThreads)
+squared_relu_kernel(T* __restrict__ z, size_t count) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t at = (static_cast<size_t>(blockIdx.x) * kThreads + threadIdx.x) * VEC;
+    if (at < count) {
+        float value[VEC];
+        load_values<VEC>(z + at, value);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+            const float positive = fmaxf(value[i], 0.0f);
+            value[i] = positive * positive;
+        }
+        store_values<VEC>(z + at, value);
+    }
+}
+
 struct PolyCoefficients {
     float a, b, c, e;
 };
@@ -346,15 +509,22 @@ __device__ __forceinline__ Candidate warp_best(Candidate best) {
 constexpr uint32_t kArgmaxThreads = 512;
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kArgmaxThreads)
-argmax_kernel(const T* __restrict__ logits, size_t pitch, uint32_t* __restrict__ sampled, uint32_t vocab) {
+argmax_kernel(T* __restrict__ logits, size_t pitch, uint32_t* __restrict__ sampled, uint32_t vocab, float softcap) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ Candidate held[kArgmaxThreads / 32];
-    const T* row = logits + blockIdx.x * pitch;
+    T* row = logits + blockIdx.x * pitch;
     Candidate best = {-INFINITY, 0xffffffffu};
     for (uint32_t column = threadIdx.x * VEC; column < vocab; column += kArgmaxThreads * VEC) {
         float value[VEC];
         load_values<VEC>(row + column, value);
+        if (softcap > 0.0f) {
+            // the choice is made among the uncapped logits: tanh keeps the order but not small differences
+            float capped[VEC];
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) capped[i] = softcap * tanhf(value[i] / softcap);
+            store_values<VEC>(row + column, capped);
+        }
 #pragma unroll
         for (int i = 0; i < VEC; ++i) {
             if (value[i] > best.value || (value[i] == best.value && column + i < best.index)) {
@@ -543,13 +713,66 @@ cudaError_t launch_poly_norm(cudaStream_t stream, Activation type, const void* z
     return vector ? go(tag, poly_norm_kernel<__nv_bfloat16, 8>) : go(tag, poly_norm_kernel<__nv_bfloat16, 1>);
 }
 
-cudaError_t launch_argmax_rows(cudaStream_t stream, Activation type, const void* logits, size_t pitch,
-                               uint32_t* sampled, size_t rows, size_t vocab) {
+cudaError_t launch_residual_post_norm(cudaStream_t stream, const ResidualPostNormLaunch& launch) {
+    PostNormArgs args;
+    args.residual = launch.residual;
+    args.post_norm = static_cast<const __nv_bfloat16*>(launch.post_norm);
+    args.token_ids = launch.token_ids;
+    args.embedding = static_cast<const __nv_bfloat16*>(launch.embedding);
+    args.vocab = launch.vocab;
+    args.norm = static_cast<const __nv_bfloat16*>(launch.norm);
+    args.rows = launch.rows;
+    args.residual_out = launch.residual_out;
+    args.num_tokens = launch.num_tokens;
+    args.width = launch.width;
+    args.shift = launch.shift;
+    args.eps = launch.eps;
+    const bool vector = launch.width % 8 == 0 && aligned_to(launch.residual, 16) && aligned_to(launch.update, 16) &&
+                        aligned_to(launch.post_norm, 16) && aligned_to(launch.embedding, 16) &&
+                        aligned_to(launch.norm, 16) && aligned_to(launch.residual_out, 16) && aligned_to(launch.out, 16);
+    const size_t vectors = launch.width / 8;
+    const unsigned int threads =
+        vector ? static_cast<unsigned int>(std::min<size_t>((vectors + 31) / 32 * 32, 512)) : kThreads;
+    const size_t held = (vectors + threads - 1) / threads;
+    auto go = [&](auto* typed, auto kernel) {
+        using T = std::remove_pointer_t<decltype(typed)>;
+        return launch_kernel(kernel, static_cast<unsigned int>(launch.num_rows), threads, 0, stream, 1, args,
+                             static_cast<const T*>(launch.update), static_cast<T*>(launch.out));
+    };
+    auto sized = [&](auto* typed) {
+        using T = std::remove_pointer_t<decltype(typed)>;
+        if (!vector) return go(typed, residual_post_norm_kernel<T, 1, 0>);
+        if (held == 1) return go(typed, residual_post_norm_kernel<T, 8, 1>);
+        if (held == 2) return go(typed, residual_post_norm_kernel<T, 8, 2>);
+        return go(typed, residual_post_norm_kernel<T, 8, 0>);
+    };
+    return launch.type == Activation::kF32 ? sized(static_cast<float*>(nullptr))
+                                           : sized(static_cast<__nv_bfloat16*>(nullptr));
+}
+
+cudaError_t launch_squared_relu(cudaStream_t stream, Activation type, void* z, size_t count) {
+    const bool vector = count % 8 == 0 && aligned_to(z, 16);
+    const size_t per_cta = static_cast<size_t>(kThreads) * (vector ? 8 : 1);
+    auto go = [&](auto* typed, auto kernel) {
+        using T = std::remove_pointer_t<decltype(typed)>;
+        return launch_kernel(kernel, static_cast<unsigned int>((count + per_cta - 1) / per_cta), kThreads, 0, stream, 1,
+                             static_cast<T*>(z), count);
+    };
+    if (type == Activation::kF32) {
+        float* tag = nullptr;
+        return vector ? go(tag, squared_relu_kernel<float, 8>) : go(tag, squared_relu_kernel<float, 1>);
+    }
+    __nv_bfloat16* tag = nullptr;
+    return vector ? go(tag, squared_relu_kernel<__nv_bfloat16, 8>) : go(tag, squared_relu_kernel<__nv_bfloat16, 1>);
+}
+
+cudaError_t launch_argmax_rows(cudaStream_t stream, Activation type, void* logits, size_t pitch, uint32_t* sampled,
+                               size_t rows, size_t vocab, float softcap) {
     const bool vector = vocab % 8 == 0 && pitch % 8 == 0 && aligned_to(logits, 16);
     auto go = [&](auto* typed, auto kernel) {
         using T = std::remove_pointer_t<decltype(typed)>;
         return launch_kernel(kernel, static_cast<unsigned int>(rows), kArgmaxThreads, 0, stream, 1,
-                             static_cast<const T*>(logits), pitch, sampled, static_cast<uint32_t>(vocab));
+                             static_cast<T*>(logits), pitch, sampled, static_cast<uint32_t>(vocab), softcap);
     };
     if (type == Activation::kF32) {
         float* tag = nullptr;

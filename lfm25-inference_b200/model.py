@@ -232,6 +232,12 @@ def leading_decode_segments(batch) -> tuple[int, int]:
     return count, context
 
 
+def prompt_context_rows(batch, decode_segments: int) -> int:
+    """Context lengths of the segments behind the decode ones, each rounded up to whole blocks."""
+    contexts = np.asarray(batch.prefixes[decode_segments:]) + np.asarray(batch.chunks[decode_segments:])
+    return int((-(-contexts // _abi.CONTEXT_ROWS)).sum()) * _abi.CONTEXT_ROWS
+
+
 class RaggedBatch:
     """Device-resident metadata of a step that mixes prefill chunks and decode tokens
     (a `workloads.MixedStepBatch` plus the token ids)."""
@@ -255,7 +261,8 @@ class RaggedBatch:
             self.token_ids.data_ptr(), self.positions.data_ptr(), self.request_slots.data_ptr(),
             self.physical_slots.data_ptr(), self.segment_offsets.data_ptr(), self.segment_slots.data_ptr(),
             self.output_rows.data_ptr(), self.block_tables.data_ptr(), batch.block_tables.shape[1],
-            batch.block_tables.shape[0], self.num_tokens, self.num_segments, decode_segments, decode_context)
+            batch.block_tables.shape[0], self.num_tokens, self.num_segments, decode_segments, decode_context,
+            prompt_context_rows(batch, decode_segments))
 
 
 class DecodeExecutor:

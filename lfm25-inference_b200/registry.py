@@ -10,7 +10,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable
 
-from . import fegidra
+from . import fegidra, ribivik
 
 
 class UnknownModel(ValueError):
@@ -37,6 +37,7 @@ def _load_lfm2_random(folder: str, config: dict, device, num_pages: int, num_req
 
 FAMILIES = {family.architecture: family for family in (
     Family(fegidra.ARCHITECTURE, fegidra.load, ("bfloat16", "float32")),
+    Family(ribivik.ARCHITECTURE, ribivik.load, ("bfloat16", "float32")),
     Family("Lfm2Random", _load_lfm2_random, ("bfloat16",)),
 )}
 

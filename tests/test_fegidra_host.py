@@ -219,9 +219,10 @@ def test_stack_executor_rejects_bad_models_before_touching_the_device():
     layer.mixer, layer.mixer_norm, layer.conv, layer.heads, layer.dim = _abi.MIXER_GENERAL_DELTA, fake, fake, 2, 300
     layer.projection = _abi.StackLinear(fake, 3200, 64)
     layer.output = _abi.StackLinear(fake, 64, 600)
+    layer.conv_taps = 2
     layers = (_abi.StackLayer * 1)(layer)
-    model = _abi.StackModel(1, layers, _abi.ACTIVATION_BF16, 2, 10, 64, 1e-5, fake, fake, _abi.StackLinear(fake, 16, 64),
-                            fake, 1 << 20, 1, 1)
+    model = _abi.StackModel(1, layers, _abi.ACTIVATION_BF16, _abi.BLOCK_PARALLEL, 10, 64, 1e-5, 0.0, 0.0, fake, fake,
+                            _abi.StackLinear(fake, 16, 64), fake, 1 << 20, 1, 1)
 
     def create(tokens=8, rows=8):
         code = library.lfm25_stack_executor_create(fake, ctypes.byref(model), tokens, rows, ctypes.byref(out))
