@@ -34,7 +34,8 @@ enum StatusTag : uint32_t {
     kTagHybridAttention = 4,
     kTagGemmRows = 5,
     kTagStackAttention = 6,
-    kTagStackDecode = 7
+    kTagStackDecode = 7,
+    kTagLatentAttention = 8
 };
 __device__ __forceinline__ void record_wait_timeout(unsigned int* status, uint32_t tag, uint32_t detail) {
     atomicAdd(&status[0], 1u);

@@ -33,6 +33,7 @@ Entry g_options[kOptCount] = {
     {"hybrid_attention", "LFM25_HYBRID_ATTENTION", 0, 0, 2},
     {"stack_attention", "LFM25_STACK_ATTENTION", 0, 0, 1},
     {"delta_prompt", "LFM25_DELTA_PROMPT", 0, 0, 2},
+    {"state_space_prompt", "LFM25_STATE_SPACE_PROMPT", 0, 0, 1},
     {"fp8_gemm_path", "LFM25_FP8_GEMM_PATH", 0, 0, 4},
     {"bf16_gemm", "LFM25_BF16_GEMM", 0, 0, 3},
     {"decode_splits", "LFM25_DECODE_SPLITS", 0, 0, 8},

@@ -21,6 +21,9 @@
 //   delta_prompt         0 auto | 1 scan | 2 general           0         delta rule over bf16 segments: tensor-core chunks where they
 //                                                                        take the head size, the token-by-token prompt kernel,
 //                                                                        or the general kernel
+//   state_space_prompt   0 auto | 1 scan                       0         state-space recurrence over bf16 segments: tensor-core
+//                                                                        chunks where they take the sizes, or the
+//                                                                        token-by-token kernel
 //   fp8_gemm_path        0 auto | 1 stream | 2 umma | 3 generic | 4 rows   0   kernel of the E4M3 linear
 //   bf16_gemm            0 auto | 1 umma | 2 cublaslt | 3 rows  0         kernel of the BF16 linear
 //   decode_splits        0 auto | 1..8                         0         KV splits of the decode attention
@@ -47,6 +50,7 @@ enum Option : int {
     kOptHybridAttention,
     kOptStackAttention,
     kOptDeltaPrompt,
+    kOptStateSpacePrompt,
     kOptFp8GemmPath,
     kOptBf16Gemm,
     kOptDecodeSplits,

@@ -10,12 +10,18 @@
 //   warps 2-5   one thread per row: mask, online softmax with f32 weights, and the running output
 // The softmax weights enter the tensor core as a sum of two bf16 values, w = hi + lo, so that they keep 16 significant
 // bits; the denominator sums the unrounded weights.
+//
+// Latent attention takes the same kernel for its prompts (EXPANDED): keys and values of every head have been formed in
+// contiguous rows from the latents of the whole context, so a stage is one copy per 64 dimensions instead of one per page,
+// the leading key chunks hold a head's own part and the trailing ones the rotated part that all heads share, and the
+// output is gated on its way out.
 #include <cuda.h>
 
 #include "common.cuh"
 #include "launch.h"
 #include "stack_attention.h"
 #include "stack_common.cuh"
+#include "stack_latent.h"
 #include "tcgen05.cuh"
 #include "tensor_map.h"
 
@@ -56,6 +62,12 @@ struct Params {
     size_t out_pitch;
     unsigned int* status;
     uint32_t tile_tokens;
+    // EXPANDED: shape.kv_heads == shape.heads
+    uint32_t own_chunks;           // 64-dimension key chunks of a head's own part; the others are the shared part
+    uint32_t own_dim;              // first query dimension of the shared part
+    const uint32_t* bases;         // first row of each segment's context
+    const __nv_bfloat16* gate;     // token t, head h at gate + t * gate_pitch + h * vdim
+    size_t gate_pitch;
 };
 
 __device__ __forceinline__ void mma_smem(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc,
@@ -95,10 +107,11 @@ __device__ __forceinline__ void split_weights(float a, float b, uint32_t& high, 
     low = pack_bf16x2(a - rounded.x, b - rounded.y);
 }
 
-template <uint32_t KC, uint32_t VC>
+template <uint32_t KC, uint32_t VC, bool EXPANDED>
 __global__ void __launch_bounds__(kThreads, Layout<KC, VC>::kCtasPerSm)
 stack_attention_umma_kernel(const __grid_constant__ CUtensorMap query_map, const __grid_constant__ CUtensorMap key_map,
-                            const __grid_constant__ CUtensorMap value_map, const Params p) {
+                            const __grid_constant__ CUtensorMap value_map, const __grid_constant__ CUtensorMap shared_map,
+                            const Params p) {
     using L = Layout<KC, VC>;
     const uint32_t warp = threadIdx.x >> 5;
     const uint32_t lane = threadIdx.x & 31;
@@ -115,13 +128,22 @@ stack_attention_umma_kernel(const __grid_constant__ CUtensorMap query_map, const
     const uint32_t group = p.shape.heads / p.shape.kv_heads;
     const uint32_t first_position = p.positions[tile.first];
     const uint32_t last_position = first_position + tile.count - 1;
-    const size_t table_row = p.segments.slots[tile.segment];
-    if (table_row >= p.block_table_rows || last_position / kPageSize >= p.block_table_stride) {
-        return;
+    const uint32_t* __restrict__ table = nullptr;
+    uint32_t first_page = 0;
+    uint32_t context_row = 0;
+    uint32_t pages = last_position / kPageSize + 1;
+    if constexpr (EXPANDED) {
+        context_row = p.bases[tile.segment];
+        pages = (pages + kPagesPerStage - 1) / kPagesPerStage * kPagesPerStage;     // contexts end on whole stages
+    } else {
+        const size_t table_row = p.segments.slots[tile.segment];
+        if (table_row >= p.block_table_rows || last_position / kPageSize >= p.block_table_stride) {
+            return;
+        }
+        table = p.block_tables + table_row * p.block_table_stride;
+        first_page = first_visible(first_position, p.shape.chunk) / kPageSize;
+        pages -= first_page;
     }
-    const uint32_t* __restrict__ table = p.block_tables + table_row * p.block_table_stride;
-    const uint32_t first_page = first_visible(first_position, p.shape.chunk) / kPageSize;
-    const uint32_t pages = last_position / kPageSize - first_page + 1;
     const uint32_t stages_total = (pages + kPagesPerStage - 1) / kPagesPerStage;
 
     extern __shared__ uint8_t attention_smem[];
@@ -142,6 +164,7 @@ stack_attention_umma_kernel(const __grid_constant__ CUtensorMap query_map, const
         tma_prefetch_descriptor(&query_map);
         tma_prefetch_descriptor(&key_map);
         tma_prefetch_descriptor(&value_map);
+        if constexpr (EXPANDED) tma_prefetch_descriptor(&shared_map);
         for (uint32_t stage = 0; stage < L::kStages; ++stage) {
             mbar_init(bar_full + 8 * stage, 1);
             mbar_init(bar_empty + 8 * stage, 1);
@@ -170,7 +193,9 @@ stack_attention_umma_kernel(const __grid_constant__ CUtensorMap query_map, const
         if (lane == 0) {
             mbar_arrive_expect_tx(bar_q, KC * group * p.tile_tokens * 128);
             for (uint32_t chunk = 0; chunk < KC; ++chunk) {
-                tma_load_box_3d(q_base + chunk * kQueryChunkBytes, &query_map, bar_q, static_cast<int32_t>(chunk * 64),
+                // a query dimension beyond a part of the head meets a key dimension that the copy filled with zero
+                const uint32_t x = EXPANDED && chunk >= p.own_chunks ? p.own_dim + (chunk - p.own_chunks) * 64 : chunk * 64;
+                tma_load_box_3d(q_base + chunk * kQueryChunkBytes, &query_map, bar_q, static_cast<int32_t>(x),
                                 static_cast<int32_t>(kv_head * group), static_cast<int32_t>(tile.first));
             }
             for (uint32_t index = 0; index < stages_total; ++index) {
@@ -186,6 +211,28 @@ stack_attention_umma_kernel(const __grid_constant__ CUtensorMap query_map, const
                 }
                 const uint32_t bar = bar_full + 8 * stage;
                 const uint32_t count = min(kPagesPerStage, pages - index * kPagesPerStage);
+                if constexpr (EXPANDED) {
+                    const int32_t row = static_cast<int32_t>(context_row + index * kKeys);
+                    const int32_t head = static_cast<int32_t>(kv_head);
+                    const uint32_t target = ring + stage * L::kStageBytes;
+                    mbar_arrive_expect_tx(bar, L::kStageBytes);
+#pragma unroll
+                    for (uint32_t chunk = 0; chunk < KC; ++chunk) {
+                        if (chunk < p.own_chunks) {
+                            tma_load_box_3d(target + chunk * kChunkBytes, &key_map, bar, static_cast<int32_t>(chunk * 64),
+                                            head, row);
+                        } else {
+                            tma_load_2d(target + chunk * kChunkBytes, &shared_map, bar,
+                                        static_cast<int32_t>((chunk - p.own_chunks) * 64), row);
+                        }
+                    }
+#pragma unroll
+                    for (uint32_t chunk = 0; chunk < VC; ++chunk) {
+                        tma_load_box_3d(target + (KC + chunk) * kChunkBytes, &value_map, bar,
+                                        static_cast<int32_t>(chunk * 64), head, row);
+                    }
+                    continue;
+                }
                 // an unassigned page is flagged before anything of the stage is announced, and page 0 is read in its
                 // place so that the pipeline stays uniform
                 uint32_t entries[kPagesPerStage];
@@ -449,6 +496,14 @@ stack_attention_umma_kernel(const __grid_constant__ CUtensorMap query_map, const
 #pragma unroll
             for (uint32_t part = 0; part < 8 * VC; ++part) {
                 if (part * 8 < p.shape.vdim) {      // vdim is a multiple of 8
+                    if constexpr (EXPANDED) {
+                        float gate[8];
+                        load_values<8>(p.gate + static_cast<size_t>(tile.first + token) * p.gate_pitch +
+                                           kv_head * p.shape.vdim + part * 8,
+                                       gate);
+#pragma unroll
+                        for (uint32_t i = 0; i < 8; ++i) out[part * 8 + i] *= 1.0f / (1.0f + __expf(-gate[i]));
+                    }
                     uint4 value;
                     value.x = pack_bf16x2(out[part * 8] * inverse, out[part * 8 + 1] * inverse);
                     value.y = pack_bf16x2(out[part * 8 + 2] * inverse, out[part * 8 + 3] * inverse);
@@ -486,38 +541,55 @@ bool make_query_map(CUtensorMap* map, const StackAttentionLaunch& launch, uint32
                   CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <uint32_t KC, uint32_t VC>
-cudaError_t launch_sized(cudaStream_t stream, const StackAttentionLaunch& launch) {
+template <uint32_t KC, uint32_t VC, bool EXPANDED>
+cudaError_t launch_maps(cudaStream_t stream, const CUtensorMap& query_map, const CUtensorMap& key_map,
+                        const CUtensorMap& value_map, const CUtensorMap& shared_map, const Params& params) {
     using L = Layout<KC, VC>;
-    const StackAttentionShape& shape = launch.shape;
-    const uint32_t group = shape.heads / shape.kv_heads;
-    const uint32_t tile_tokens = kRows / group;
-    CUtensorMap query_map, key_map, value_map;
-    if (!make_query_map(&query_map, launch, group, tile_tokens) || !make_page_map(&key_map, launch, false) ||
-        !make_page_map(&value_map, launch, true)) {
-        return cudaErrorInvalidValue;
-    }
-    const auto kernel = stack_attention_umma_kernel<KC, VC>;
+    const auto kernel = stack_attention_umma_kernel<KC, VC, EXPANDED>;
     const cudaError_t status = cudaFuncSetAttribute(reinterpret_cast<const void*>(kernel),
                                                     cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                     static_cast<int>(L::kSharedBytes));
     if (status != cudaSuccess) return status;
-    Params params;
-    params.shape = shape;
-    params.block_tables = launch.block_tables;
-    params.block_table_stride = launch.block_table_stride;
-    params.block_table_rows = launch.block_table_rows;
-    params.num_pages = launch.num_pages;
-    params.positions = launch.positions;
-    params.segments = launch.segments;
-    params.out = static_cast<__nv_bfloat16*>(launch.out);
-    params.out_pitch = launch.out_pitch;
-    params.status = launch.status;
-    params.tile_tokens = tile_tokens;
-    const size_t tiles = tile_bound(launch.segments, tile_tokens);
-    return launch_kernel(kernel, static_cast<unsigned int>(tiles * shape.kv_heads), kThreads, L::kSharedBytes, stream, 1,
-                         query_map, key_map, value_map, params);
+    const size_t tiles = tile_bound(params.segments, params.tile_tokens);
+    return launch_kernel(kernel, static_cast<unsigned int>(tiles * params.shape.kv_heads), kThreads, L::kSharedBytes,
+                         stream, 1, query_map, key_map, value_map, shared_map, params);
 }
+
+// `key_chunks` and `value_chunks` of 64 dimensions
+template <bool EXPANDED>
+cudaError_t launch_chunks(cudaStream_t stream, uint32_t key_chunks, uint32_t value_chunks, const CUtensorMap& query_map,
+                          const CUtensorMap& key_map, const CUtensorMap& value_map, const CUtensorMap& shared_map,
+                          const Params& params) {
+    auto go = [&](auto narrow, auto wide) {
+        return (value_chunks > 1 ? wide : narrow)(stream, query_map, key_map, value_map, shared_map, params);
+    };
+    switch (key_chunks) {
+        case 1: return go(launch_maps<1, 1, EXPANDED>, launch_maps<1, 2, EXPANDED>);
+        case 2: return go(launch_maps<2, 1, EXPANDED>, launch_maps<2, 2, EXPANDED>);
+        case 3: return go(launch_maps<3, 1, EXPANDED>, launch_maps<3, 2, EXPANDED>);
+        case 4: return go(launch_maps<4, 1, EXPANDED>, launch_maps<4, 2, EXPANDED>);
+        default: return cudaErrorInvalidValue;
+    }
+}
+
+// [rows, heads, size] with the heads of a row side by side and rows `pitch` elements apart, in boxes of 64 dimensions of
+// one head x `box_rows`
+bool make_head_map(CUtensorMap* map, const void* base, size_t size, size_t heads, size_t rows, size_t pitch,
+                   uint32_t box_rows) {
+    EncodeTiledFn encode = encode_tiled_entry();
+    if (encode == nullptr) {
+        return false;
+    }
+    const cuuint64_t dims[3] = {size, heads, rows};
+    const cuuint64_t strides[2] = {size * 2, pitch * 2};
+    const cuuint32_t box[3] = {64, 1, box_rows};
+    const cuuint32_t element_strides[3] = {1, 1, 1};
+    return encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, element_strides,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+uint32_t chunks_of(uint32_t size) { return (size + 63) / 64; }
 
 }  // namespace
 
@@ -543,15 +615,69 @@ bool stack_attention_umma_supports(const StackAttentionLaunch& launch) {
 }
 
 cudaError_t launch_stack_attention_umma(cudaStream_t stream, const StackAttentionLaunch& launch) {
-    const uint32_t key_chunks = (launch.shape.dim + 63) / 64;
-    const bool wide = launch.shape.vdim > 64;
-    switch (key_chunks) {
-        case 1: return wide ? launch_sized<1, 2>(stream, launch) : launch_sized<1, 1>(stream, launch);
-        case 2: return wide ? launch_sized<2, 2>(stream, launch) : launch_sized<2, 1>(stream, launch);
-        case 3: return wide ? launch_sized<3, 2>(stream, launch) : launch_sized<3, 1>(stream, launch);
-        case 4: return wide ? launch_sized<4, 2>(stream, launch) : launch_sized<4, 1>(stream, launch);
-        default: return cudaErrorInvalidValue;
+    const StackAttentionShape& shape = launch.shape;
+    const uint32_t group = shape.heads / shape.kv_heads;
+    Params params = {};
+    params.shape = shape;
+    params.block_tables = launch.block_tables;
+    params.block_table_stride = launch.block_table_stride;
+    params.block_table_rows = launch.block_table_rows;
+    params.num_pages = launch.num_pages;
+    params.positions = launch.positions;
+    params.segments = launch.segments;
+    params.out = static_cast<__nv_bfloat16*>(launch.out);
+    params.out_pitch = launch.out_pitch;
+    params.status = launch.status;
+    params.tile_tokens = kRows / group;
+    CUtensorMap query_map, key_map, value_map;
+    if (!make_query_map(&query_map, launch, group, params.tile_tokens) || !make_page_map(&key_map, launch, false) ||
+        !make_page_map(&value_map, launch, true)) {
+        return cudaErrorInvalidValue;
     }
+    return launch_chunks<false>(stream, chunks_of(shape.dim), chunks_of(shape.vdim), query_map, key_map, value_map, key_map,
+                                params);
+}
+
+bool expanded_attention_supports(Activation type, const LatentAttentionShape& shape, size_t out_pitch, size_t gate_pitch,
+                                 size_t expanded_pitch) {
+    return type == Activation::kBf16 && shape.scale > 0.0f && shape.dim % 8 == 0 && shape.rot_dim % 8 == 0 &&
+           shape.vdim % 8 == 0 && shape.kv_rank % 8 == 0 && shape.vdim <= 128 &&
+           chunks_of(shape.dim) + chunks_of(shape.rot_dim) <= 4 && out_pitch % 8 == 0 && gate_pitch % 8 == 0 &&
+           expanded_pitch % 8 == 0;
+}
+
+cudaError_t launch_expanded_attention(cudaStream_t stream, const ExpandedAttentionLaunch& launch) {
+    const LatentAttentionShape& shape = launch.shape;
+    Params params = {};
+    params.shape = {shape.heads, shape.heads, shape.dim + shape.rot_dim, shape.vdim, 0, 0, shape.scale};
+    params.positions = launch.positions;
+    // segment offsets are absolute token indices, so leaving segments out is simply a later start
+    params.segments = launch.segments;
+    params.segments.offsets += launch.first_segment;
+    params.segments.slots += launch.first_segment;
+    params.segments.num_segments -= launch.first_segment;
+    params.out = static_cast<__nv_bfloat16*>(launch.out);
+    params.out_pitch = launch.out_pitch;
+    params.status = launch.status;
+    params.tile_tokens = kRows;
+    params.own_chunks = chunks_of(shape.dim);
+    params.own_dim = shape.dim;
+    params.bases = launch.bases + launch.first_segment;
+    params.gate = static_cast<const __nv_bfloat16*>(launch.gate);
+    params.gate_pitch = launch.gate_pitch;
+    const auto* expanded = static_cast<const __nv_bfloat16*>(launch.expanded);
+    CUtensorMap query_map, key_map, value_map, shared_map;
+    if (!make_head_map(&query_map, launch.query, shape.dim + shape.rot_dim, shape.heads, launch.segments.num_tokens,
+                       launch.query_pitch, kRows) ||
+        !make_head_map(&key_map, expanded, shape.dim, shape.heads, launch.rows, launch.expanded_pitch, kKeys) ||
+        !make_head_map(&value_map, expanded + static_cast<size_t>(shape.heads) * shape.dim, shape.vdim, shape.heads,
+                       launch.rows, launch.expanded_pitch, kKeys) ||
+        !make_swizzled_2d_map_width(&shared_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, launch.keys, launch.rows,
+                                    shape.rot_dim, shape.rot_dim * 2, kKeys)) {
+        return cudaErrorInvalidValue;
+    }
+    return launch_chunks<true>(stream, params.own_chunks + chunks_of(shape.rot_dim), chunks_of(shape.vdim), query_map,
+                               key_map, value_map, shared_map, params);
 }
 
 }  // namespace lfm25

@@ -55,17 +55,21 @@ def latent_entries(h, tensors, kv_rank, positions, base, rot_dims, eps):
     return latent, rotate(both[:, None, kv_rank:], positions, base, rot_dims)[:, 0]
 
 
-def latent_softmax(query, rotated_query, latents, rotated_keys, up_key, up_value, scale):
-    """One query position over every cached token: query [heads, dim], rotated_query [heads, rot_dim], latents [N, rank],
-    rotated_keys [N, rot_dim].  Returns [heads, vdim]."""
-    heads, dim = query.shape
+def expand(latents, up_key, up_value, heads):
+    """Unrotated keys [heads, N, dim] and values [heads, N, vdim] of latents [N, rank]."""
+    keys = [latents @ part.T for part in np.split(up_key, heads)]
+    values = [latents @ part.T for part in np.split(up_value, heads)]
+    return np.stack(keys), np.stack(values)
+
+
+def softmax_over(query, rotated_query, keys, values, rotated_keys, scale):
+    """One query position: query [heads, dim], rotated_query [heads, rot_dim], keys [heads, N, dim], values [heads, N, vdim],
+    rotated_keys [N, rot_dim] shared by the heads.  Returns [heads, vdim]."""
     out = []
-    for head in range(heads):
-        keys = latents @ up_key.reshape(heads, dim, -1)[head].T
-        values = latents @ up_value.reshape(heads, -1, latents.shape[1])[head].T
-        scores = (keys @ query[head] + rotated_keys @ rotated_query[head]) * scale
+    for head in range(len(query)):
+        scores = (keys[head] @ query[head] + rotated_keys @ rotated_query[head]) * scale
         weights = np.exp(scores - scores.max())
-        out.append((weights / weights.sum()) @ values)
+        out.append((weights / weights.sum()) @ values[head])
     return np.stack(out)
 
 
@@ -79,8 +83,9 @@ def latent_attention(h, tensors, sizes, eps, positions, cache):
     if sizes.get("kv_from") is None:
         latent, key = latent_entries(h, tensors, sizes["kv_rank"], positions, rot["base"], rot["dims"], eps)
         cache[0], cache[1] = np.concatenate([cache[0], latent]), np.concatenate([cache[1], key])
-    out = np.stack([latent_softmax(query[t, :, :dim], rotated_query[t], cache[0][:position + 1], cache[1][:position + 1],
-                                   tensors["uk"], tensors["uv"], sizes["scale"])
+    keys, values = expand(cache[0], tensors["uk"], tensors["uv"], heads)
+    out = np.stack([softmax_over(query[t, :, :dim], rotated_query[t], keys[:, :position + 1], values[:, :position + 1],
+                                 cache[1][:position + 1], sizes["scale"])
                     for t, position in enumerate(positions)])
     gated = out.reshape(len(h), -1) * sigmoid(linear(h, tensors["g"]))
     return linear(gated, tensors["o"])

@@ -5,6 +5,7 @@ import numpy as np
 import pytest
 
 import fegidra_cases as cases
+import stack_cases
 from oracle import fegidra as oracle_fegidra
 
 pytestmark = pytest.mark.gpu
@@ -14,31 +15,12 @@ TYPES = ("float32", "bfloat16")
 
 def run_layer(config, tensors, device, dtype, portions, seed=3):
     """Residual stream behind a one-layer model's layer, framework and restatement."""
-    import torch
-
-    from lfm25_inference_b200 import model as lfm_model
-    from lfm25_inference_b200 import ops, stack, workloads
     tokens = np.random.default_rng(seed).integers(0, config["vocab"], size=sum(portions)).astype(np.uint32)
     want = []
     cases.oracle_model(config, tensors).forward(tokens, cases.oracle_model(config, tensors).new_state(), want)
-    got, pages = [], (len(tokens) + 15) // 16
-    with torch.cuda.stream(torch.cuda.Stream(device)):
-        model = cases.product_model(config, tensors, device, dtype, num_pages=pages + 3, slots=2)
-        blaslt = ops.BlasLt()
-        executor = stack.StackExecutor(blaslt, model, len(tokens))
-        table = np.random.default_rng(7).permutation(pages + 3).astype(np.uint32)[:pages].reshape(1, -1)
-        table = np.concatenate([np.full_like(table, 0xFFFFFFFF), table])       # the sequence lives in slot 1
-        at = 0
-        for size in portions:
-            batch = workloads.MixedStepBatch(pages + 3, table, np.array([at]), np.array([size]),
-                                             np.array([1], np.uint32))
-            executor.forward_ragged(lfm_model.RaggedBatch(device, batch, tokens[at:at + size]))
-            got.append(executor.residual(size))
-            at += size
-        assert ops.device_status()[0] == 0
-        executor.close()
-        blaslt.close()
-    return np.concatenate(got), want[-1]
+    got = stack_cases.residual_in_portions(
+        lambda pages, slots: cases.product_model(config, tensors, device, dtype, pages, slots), device, tokens, portions)
+    return got, want[-1]
 
 
 def check_layer(config, seed, device, dtype, portions, rank=5, change=None):
