@@ -25,7 +25,7 @@ SOURCES = ["api.cu", "options.cu", "attention.cu", "kv_cache.cu", "fp8_elementwi
            "hybrid_attention_umma.cu", "model_ops.cu", "cublaslt_bf16.cu", "decode_executor.cu", "host_runtime.cu",
            "prefix_cache.cu", "scheduler.cu", "serving_engine.cu", "step_backends.cu", "stack_norm.cu", "stack_attention.cu",
            "stack_attention_umma.cu", "stack_attention_decode.cu", "delta_rule.cu", "head_linear.cu", "stack_latent.cu",
-           "stack_latent_decode.cu", "state_space.cu", "stack_executor.cu"]
+           "stack_latent_decode.cu", "state_space.cu", "state_space_chunk.cu", "stack_executor.cu"]
 COMPILE_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC"]
 LINK_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-shared", "-cudart", "static", "-ldl"]
 

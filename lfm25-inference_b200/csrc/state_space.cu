@@ -425,6 +425,9 @@ cudaError_t launch_state_space(cudaStream_t stream, const StateSpaceLaunch& laun
         rest.segments.slots += launch.decode_tokens;
         rest.segments.num_segments -= launch.decode_tokens;
     }
+    if (option(kOptStateSpacePrompt) == 0 && state_space_chunk_supports(rest)) {
+        return launch_state_space_chunk(stream, rest);
+    }
     return f32 ? launch_scan<float>(stream, rest) : launch_scan<__nv_bfloat16>(stream, rest);
 }
 

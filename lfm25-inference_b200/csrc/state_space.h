@@ -61,4 +61,7 @@ __device__ __forceinline__ float state_rate(const StateSpaceArgs<T>& args, uint3
     return expf(__bfloat162float(args.log_rate[head]));
 }
 
+bool state_space_chunk_supports(const StateSpaceLaunch& launch);
+cudaError_t launch_state_space_chunk(cudaStream_t stream, const StateSpaceLaunch& launch);
+
 }  // namespace lfm25
