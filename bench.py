@@ -23,8 +23,8 @@ copies of at least 512 MB, cuBLASLt on the same buffers beside every point, each
 max(bytes / HBM peak, flops / tensor peak).  A compact table of its E4M3 half is part of the default line
 (`gemm_roofline`).
 
-Workload `stack` times a layer-stack model (Fegidra) at LFM2.5-1.2B's sizes beside the LFM2 model, both in BF16:
-decode steps replayed from graphs at several batch sizes, mixed prefill steps, and every kernel's device time.
+Workload `stack` times a layer-stack model at LFM2.5-1.2B's sizes beside the closest other model in BF16 (--design
+fegidra: beside LFM2; --design ribivik: beside Fegidra): decode steps replayed from graphs at several batch sizes, mixed prefill steps, and every kernel's device time.
 
 `cpu_baseline` / `--impl reference`: the reference project is GPU-only, so the CPU arm is the multithreaded C
 restatement of its kernels (oracle/), timed on the same step (all 128 sequences, one step) on the host's cores.
@@ -77,6 +77,7 @@ def parse_arguments():
     parser.add_argument("--step-sequences", type=int, default=STEP_SEQUENCES,
                         help="step workload: sequences in the batch (the headline number needs the default)")
     parser.add_argument("--pool-pages", type=int, default=NUM_PAGES, help="pages in the K/V pool (same remark)")
+    parser.add_argument("--design", default="fegidra", choices=["fegidra", "ribivik"], help="stack workload: which model")
     parser.add_argument("--skip-cpu", action="store_true", help="omit the CPU baseline (profiling runs)")
     parser.add_argument("--skip-gemm", action="store_true", help="step workload: omit the gemm_roofline table")
     parser.add_argument("--gemm-dtype", default="all", choices=["all", "e4m3", "bf16"], help="gemm workload: which sites")
@@ -1456,7 +1457,7 @@ def run_serving_arm(arguments, rank, world):
 
 
 def run_stack_arm(arguments, rank, world):
-    """Layer-stack model beside the LFM2 model (stack_bench): one JSON line; every replica measures the same cases."""
+    """Layer-stack model beside the closest other one (stack_bench): one JSON line; every replica measures the same cases."""
     import torch
     import torch.distributed as dist
 
@@ -1470,16 +1471,16 @@ def run_stack_arm(arguments, rank, world):
     hbm, hbm_source = peaks()
     tensor, tensor_source = tensor_peaks()
     with ClockSampler(local_rank) as sampler:
-        result = stack_bench.run(device, arguments.steps, hbm, tensor)
+        result = stack_bench.run(device, arguments.steps, hbm, tensor, arguments.design)
     slowest = max_over_ranks([result["decode"][-1]["stack"]["ms_per_step"]], device, world)[0]
     if rank == 0:
         sequences = result["decode"][-1]["sequences"]
         print(json.dumps({
-            "metric": "decode tok/s (Fegidra at LFM2.5-1.2B sizes, random weights)",
+            "metric": f"decode tok/s ({arguments.design.capitalize()} at LFM2.5-1.2B sizes, random weights)",
             "value": aggregate_throughput(sequences, world, slowest), "unit": "tok/s", "n_gpus": world,
             "steps": arguments.steps, "warmup": arguments.warmup, "ms_per_step": slowest, "higher_is_better": True,
             "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-            "config": {"model": "Fegidra, width 2048, 16 layers", "sequences": sequences, "replicas": world,
+            "config": {"model": f"{arguments.design.capitalize()}, width 2048, 16 layers", "sequences": sequences, "replicas": world,
                        "l2": "more than 2 GB of weights streamed per step exceed L2"},
             "peaks": {"hbm_gbs": [hbm, hbm_source], "bf16_tflops": [tensor, tensor_source]},
             "cases": result, "device_status": list(ops.device_status()), "clocks": sampler.summary()}), flush=True)
