@@ -50,6 +50,7 @@ struct lfm25_stack_executor {
     void* context_keys;        // [C, widest rot_dim]
     void* expanded;            // [C, widest latent_up.n]: their keys and values
     uint32_t* context_bases;   // [T + 1]
+    uint32_t* token_order;     // [T]: the tokens that attend to latents, longest context first
     void* convolved;           // [T, widest channels] of a state-space mixer
     void* scanned;             // [T, widest heads * vdim]
     size_t context_capacity = 0;
@@ -227,6 +228,12 @@ struct Step {
     bool advance;
 };
 
+// What earlier layers of the step have left in scratch for later ones.
+struct Prepared {
+    const void* gathered = nullptr;    // the latent cache whose contexts lie in the context scratch
+    size_t ordered = 0;                // leading tokens that token_order sorts
+};
+
 int32_t run_attention(lfm25_stack_executor* self, const Step& step, const lfm25_stack_layer& layer) {
     const lfm25_stack_model& model = *self->model;
     cudaStream_t stream = self->blaslt->stream;
@@ -307,9 +314,8 @@ bool expands_contexts(const lfm25_stack_executor* self, const Step& step, const 
     return lfm25::expanded_attention_supports(self->type, shape, layer.output.k, layer.projection.n, layer.latent_up.n);
 }
 
-// `gathered`: the latent cache whose contexts lie in the context scratch already (layers that share a cache).
 int32_t run_latent_attention(lfm25_stack_executor* self, const Step& step, const lfm25_stack_layer& layer,
-                             const void** gathered) {
+                             Prepared* prepared) {
     const lfm25_stack_model& model = *self->model;
     cudaStream_t stream = self->blaslt->stream;
     const size_t tokens = step.segments.num_tokens;
@@ -379,6 +385,15 @@ int32_t run_latent_attention(lfm25_stack_executor* self, const Step& step, const
         attention.num_pages = model.num_pages;
         attention.request_slots = step.request_slots;
         attention.positions = step.positions;
+        attention.token_order = nullptr;
+        if (direct > 1 && direct <= lfm25::kMaxOrderTokens) {
+            if (prepared->ordered != direct) {
+                STACK_CUDA(lfm25::launch_context_order(stream, step.positions, direct, self->token_order),
+                           "context order launch failed");
+                prepared->ordered = direct;
+            }
+            attention.token_order = self->token_order;
+        }
         attention.tokens = direct;
         attention.context = std::max(step.decode_context, direct > step.decode_tokens ? step.prompt_context_rows : 0);
         attention.status = lfm25::device_status_words();
@@ -403,8 +418,8 @@ int32_t run_latent_attention(lfm25_stack_executor* self, const Step& step, const
     }
     if (!expand) return LFM25_OK;
     const size_t rows = step.prompt_context_rows;
-    if (*gathered != layer.value_cache) {
-        if (*gathered == nullptr) {
+    if (prepared->gathered != layer.value_cache) {
+        if (prepared->gathered == nullptr) {
             STACK_CUDA(lfm25::launch_context_bases(stream, step.segments, step.positions, step.decode_tokens,
                                                    self->context_bases),
                        "context layout launch failed");
@@ -427,7 +442,7 @@ int32_t run_latent_attention(lfm25_stack_executor* self, const Step& step, const
         gather.keys = self->context_keys;
         gather.rows = rows;
         STACK_CUDA(lfm25::launch_gather_context(stream, gather), "context gather launch failed");
-        *gathered = layer.value_cache;
+        prepared->gathered = layer.value_cache;
     }
     STACK_TRY(linear(self, layer.latent_up, self->context_latents, self->expanded, rows));
     lfm25::ExpandedAttentionLaunch attention;
@@ -504,12 +519,12 @@ int32_t run_state_space(lfm25_stack_executor* self, const Step& step, const lfm2
     return LFM25_OK;
 }
 
-int32_t run_mixer(lfm25_stack_executor* self, const Step& step, const lfm25_stack_layer& layer, const void** gathered) {
+int32_t run_mixer(lfm25_stack_executor* self, const Step& step, const lfm25_stack_layer& layer, Prepared* prepared) {
     STACK_TRY(linear(self, layer.projection, self->mixed, self->projected, step.segments.num_tokens));
     switch (layer.mixer) {
         case LFM25_MIXER_ATTENTION: return run_attention(self, step, layer);
         case LFM25_MIXER_GENERAL_DELTA: return run_general_delta(self, step, layer);
-        case LFM25_MIXER_LATENT_ATTENTION: return run_latent_attention(self, step, layer, gathered);
+        case LFM25_MIXER_LATENT_ATTENTION: return run_latent_attention(self, step, layer, prepared);
         default: return run_state_space(self, step, layer);
     }
 }
@@ -518,7 +533,7 @@ int32_t enqueue_parallel(lfm25_stack_executor* self, const Step& step) {
     const lfm25_stack_model& model = *self->model;
     cudaStream_t stream = self->blaslt->stream;
     const size_t tokens = step.segments.num_tokens;
-    const void* gathered = nullptr;
+    Prepared prepared;
     int current = 0;
     for (uint32_t index = 0; index < self->depth; ++index) {
         const lfm25_stack_layer& layer = model.layers[index];
@@ -542,7 +557,7 @@ int32_t enqueue_parallel(lfm25_stack_executor* self, const Step& step) {
         head.eps = model.norm_eps;
         STACK_CUDA(lfm25::launch_residual_norm_conv(stream, head), "residual norm convolution launch failed");
         current = 1 - current;
-        STACK_TRY(run_mixer(self, step, layer, &gathered));
+        STACK_TRY(run_mixer(self, step, layer, &prepared));
         if (layer.ff > 0) {
             STACK_TRY(linear(self, layer.up, self->normalized, self->up, tokens));
             const size_t column = mixer_columns(layer);
@@ -569,7 +584,7 @@ int32_t enqueue_sandwich(lfm25_stack_executor* self, const Step& step) {
     const lfm25_stack_model& model = *self->model;
     cudaStream_t stream = self->blaslt->stream;
     const size_t tokens = step.segments.num_tokens;
-    const void* gathered = nullptr;
+    Prepared prepared;
     lfm25::ResidualPostNormLaunch norm;
     norm.type = self->type;
     norm.residual = self->residual[0];
@@ -597,7 +612,7 @@ int32_t enqueue_sandwich(lfm25_stack_executor* self, const Step& step) {
     for (uint32_t index = 0; index < self->depth; ++index) {
         const lfm25_stack_layer& layer = model.layers[index];
         STACK_TRY(enter(layer.mixer_norm, self->mixed));
-        STACK_TRY(run_mixer(self, step, layer, &gathered));
+        STACK_TRY(run_mixer(self, step, layer, &prepared));
         STACK_TRY(linear(self, layer.output, self->joined, self->update, tokens));
         norm.post_norm = layer.mixer_post_norm;
         if (layer.ff > 0) {
@@ -804,13 +819,14 @@ int32_t lfm25_stack_executor_create(lfm25_blaslt* blaslt, const lfm25_stack_mode
                        &self->update, &self->head_input, &self->logits, reinterpret_cast<void**>(&self->raw),
                        reinterpret_cast<void**>(&self->sampled), &self->compressed, &self->absorbed, &self->weighted,
                        &self->context_latents, &self->context_keys, &self->expanded,
-                       reinterpret_cast<void**>(&self->context_bases), &self->convolved, &self->scanned};
+                       reinterpret_cast<void**>(&self->context_bases), reinterpret_cast<void**>(&self->token_order),
+                       &self->convolved, &self->scanned};
     const size_t sizes[] = {t * model->width * 4, t * model->width * 4, t * model->width * bytes,
                             t * model->width * bytes, t * projection * bytes, t * query * bytes, t * up * bytes,
                             t * joined * bytes, t * model->width * bytes, r * model->width * bytes,
                             r * model->head.n * bytes, t * raw * 4, r * 4, t * compressed * bytes, t * latents * bytes,
                             t * latents * bytes, c * context_rank * bytes, c * context_keys * bytes,
-                            c * context_columns * bytes, (t + 1) * 4, t * channels * bytes, t * scanned * bytes};
+                            c * context_columns * bytes, (t + 1) * 4, latents > 0 ? t * 4 : 0, t * channels * bytes, t * scanned * bytes};
     size_t total = 0;
     for (size_t size : sizes) total += (size + 255) & ~static_cast<size_t>(255);
     cudaError_t status = cudaMalloc(&self->allocation, total);

@@ -226,6 +226,7 @@ struct LatentAttentionLaunch {
     size_t num_pages;
     const uint32_t* request_slots; // [T]
     const uint32_t* positions;     // [T]
+    const uint32_t* token_order;   // a permutation of the tokens, in which they are started, or nullptr
     size_t tokens;
     size_t context;                // longest context among them when known, else 0
     unsigned int* status;

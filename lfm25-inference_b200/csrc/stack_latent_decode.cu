@@ -8,8 +8,8 @@
 //               arrive in one copy; behind them the rotated keys, chunk by chunk
 //   warp 1      tensor memory and the MMAs: S^T [64 keys, heads] = K Q^T over all chunks, then O^T [kv_rank, heads] +=
 //               latent^T P^T over the same shared memory, now read with the latent dimensions as rows
-//   warps 2-9   one key per thread (lanes 0 .. 15; two warps share a quadrant of tensor memory and take half of the heads
-//               each): mask and softmax weights in f32.  The weights are taken against a reference that follows the running
+//   others      one key per thread (lanes 0 .. 15; two or four warps share a quadrant of tensor memory and divide the heads
+//               among them): mask and softmax weights in f32.  The weights are taken against a reference that follows the running
 //               maximum only when it falls more than 2^8 behind; then the accumulators in tensor memory are rescaled
 // The weights enter the second product as a sum of two bf16 values (16 significant bits), the two parts as neighbouring
 // columns of one MMA; sums and accumulators are f32.  The splits of a token merge through the distributed shared memory of
@@ -33,8 +33,10 @@ namespace {
 
 namespace cg = cooperative_groups;
 
-constexpr uint32_t kSoftmaxWarps = 8;
-constexpr uint32_t kThreads = 64 + kSoftmaxWarps * 32;
+// Warps that share a quadrant of tensor memory, by the number of heads of a CTA
+constexpr __host__ __device__ uint32_t sharing_warps(uint32_t heads) { return heads <= 16 ? 2 : 4; }
+constexpr __host__ __device__ uint32_t softmax_threads(uint32_t heads) { return sharing_warps(heads) * 128; }
+constexpr __host__ __device__ uint32_t cta_threads(uint32_t heads) { return 64 + softmax_threads(heads); }
 constexpr uint32_t kPagesPerStage = 4;
 constexpr uint32_t kKeys = kPagesPerStage * kPageSize;       // 64
 constexpr uint32_t kGroupKeys = 8;
@@ -54,6 +56,7 @@ struct Params {
     size_t num_pages;
     const uint32_t* request_slots;
     const uint32_t* positions;
+    const uint32_t* token_order;
     __nv_bfloat16* out;
     unsigned int* status;
     uint32_t whole_chunks;               // chunks of 64 latent dimensions that are full
@@ -72,14 +75,16 @@ struct Control {
     float warp_max[4][N];
     float warp_sum[4][N];
     float total[N];
-    float share[kMaxSplits][N];     // of each split of the token, over the sum of all weights
+    // what every split of the token tells the others
+    float split_reference[kMaxSplits][N], split_total[kMaxSplits][N];
+    uint32_t split_unusable[kMaxSplits];
+    float share[kMaxSplits][N];     // what a split's result counts for
     uint64_t full[kMaxStages], empty[kMaxStages];
     uint64_t query, scores[2], weights[2], product[2];
     uint32_t tmem;
     volatile uint32_t abort;
     volatile uint32_t missing_page;
     volatile uint32_t failed[2];
-    uint32_t unusable, merged_unusable;      // of this split, of all splits of the token
 };
 
 // MMAs that add to the same accumulator wait for one another, which small ones feel: the steps of a score take turns among
@@ -163,10 +168,12 @@ __device__ __forceinline__ uint64_t descriptor(uint32_t address, uint32_t group_
 }
 
 // Barrier of the softmax warps
+template <uint32_t THREADS>
 __device__ __forceinline__ void softmax_barrier() {
     __syncwarp();
-    asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxWarps * 32) : "memory");
+    asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory");
 }
+template <uint32_t THREADS>
 __device__ __forceinline__ bool softmax_any(bool mine) {
     __syncwarp();
     uint32_t any;
@@ -178,17 +185,23 @@ __device__ __forceinline__ bool softmax_any(bool mine) {
         "selp.u32 %0, 1, 0, q;\n"
         "}\n"
         : "=r"(any)
-        : "r"(mine ? 1u : 0u), "n"(kSoftmaxWarps * 32)
+        : "r"(mine ? 1u : 0u), "n"(THREADS)
         : "memory");
     return any != 0;
 }
 
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.aligned;" ::: "memory"); }
+
 template <uint32_t N>
-__global__ void __launch_bounds__(kThreads, 1)
+__global__ void __launch_bounds__(cta_threads(N), 1)
 latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, const __grid_constant__ CUtensorMap rotated_map,
                              const __grid_constant__ CUtensorMap latent_map, const __grid_constant__ CUtensorMap tail_map,
                              const __grid_constant__ CUtensorMap key_map, const Params p) {
-    constexpr uint32_t kHalf = N / 2;       // heads per softmax thread
+    constexpr uint32_t kSharing = sharing_warps(N);
+    constexpr uint32_t kShare = N / kSharing;       // heads per softmax thread
+    constexpr uint32_t kSoftmax = softmax_threads(N);
+    constexpr uint32_t kThreads = cta_threads(N);
     constexpr uint32_t kSums = score_sums<N>();
     const uint32_t warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0);     // the same value to the compiler's eye as well
     const uint32_t lane = threadIdx.x & 31;
@@ -216,7 +229,7 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
         mbar_init(bar_query, 1);
         for (uint32_t buffer = 0; buffer < 2; ++buffer) {
             mbar_init(bar_scores + 8 * buffer, 1);
-            mbar_init(bar_weights + 8 * buffer, kSoftmaxWarps);
+            mbar_init(bar_weights + 8 * buffer, kSoftmax / 32);
             mbar_init(bar_product + 8 * buffer, 1);
             control.failed[buffer] = 0;
         }
@@ -239,13 +252,16 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
     tcgen05_fence_before();
     __syncthreads();
     tcgen05_fence_after();
+    // a CTA writes into the others' shared memory at its end, which may come before they have started
+    if (p.splits > 1) cluster_arrive();
     const uint32_t tmem_base = __shfl_sync(0xffffffffu, *reinterpret_cast<volatile uint32_t*>(&control.tmem), 0);
     const uint32_t tmem_out = tmem_base + 2 * kSums * N;         // [block][high heads | low heads]
     pdl_wait();
 
     const uint32_t split = blockIdx.x % p.splits;
     const uint32_t head0 = blockIdx.x / p.splits % p.head_blocks * N;
-    const uint32_t token = blockIdx.x / p.splits / p.head_blocks;
+    const uint32_t rank = blockIdx.x / p.splits / p.head_blocks;
+    const uint32_t token = p.token_order != nullptr ? p.token_order[rank] : rank;
     const size_t table_row = p.request_slots[token];
     const uint32_t position = p.positions[token];
     const bool valid = table_row < p.block_table_rows && position / kPageSize < p.block_table_stride;
@@ -416,13 +432,13 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
         const uint32_t quadrant = warp & 3;                 // the tensor-memory lanes this warp may touch
         const uint32_t lane_address = (quadrant * 32) << 16;
         const uint32_t thread = threadIdx.x - 64;
-        const uint32_t half = thread / 128;                 // which half of the heads
-        const uint32_t first_head = half * kHalf;
+        const uint32_t share = thread / 128;                // which part of the heads
+        const uint32_t first_head = share * kShare;
         const uint32_t key = quadrant * 16 + (lane & 15);   // of the stage; lanes 16 .. 31 hold nothing
         const float scale_log2 = p.scale * kLog2e;
-        float sum[kHalf];
+        float sum[kShare];
 #pragma unroll
-        for (uint32_t head = 0; head < kHalf; ++head) sum[head] = 0.0f;
+        for (uint32_t head = 0; head < kShare; ++head) sum[head] = 0.0f;
         bool ok = true;
         for (uint32_t index = 0; index < count; ++index) {
             const uint32_t stage = index % p.stages;
@@ -433,10 +449,10 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
             __syncwarp();
             const uint32_t stage_first = (split + index * p.splits) * kKeys;
             const bool visible = lane < 16 && stage_first + key <= position;
-            float score[kHalf];
+            float score[kShare];
             bool over = false;
 #pragma unroll
-            for (uint32_t part = 0; part < kHalf / 8; ++part) {
+            for (uint32_t part = 0; part < kShare / 8; ++part) {
                 uint32_t raw[kSums][8];
 #pragma unroll
                 for (uint32_t way = 0; way < kSums; ++way) {
@@ -455,14 +471,14 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
             }
             // whatever happened above, all warps meet here; the flag of this parity is written before the barrier only, so
             // that all of them leave the loop together
-            over = softmax_any(over);
+            over = softmax_any<kSoftmax>(over);
             if (control.failed[buffer]) {
                 ok = false;
                 break;
             }
             if (over) {
 #pragma unroll
-                for (uint32_t head = 0; head < kHalf; ++head) {
+                for (uint32_t head = 0; head < kShare; ++head) {
                     float best = score[head];
 #pragma unroll
                     for (uint32_t delta = 8; delta > 0; delta >>= 1) {
@@ -470,7 +486,7 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
                     }
                     if (lane == 0) control.warp_max[quadrant][first_head + head] = best;
                 }
-                softmax_barrier();
+                softmax_barrier<kSoftmax>();
                 if (thread < N) {
                     const float before = control.reference[thread];
                     float now = before;
@@ -479,24 +495,26 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
                     control.reference[thread] = now;
                     control.factor[thread] = now == before ? 1.0f : fast_exp2(before - now);
                 }
-                softmax_barrier();
+                softmax_barrier<kSoftmax>();
 #pragma unroll
-                for (uint32_t head = 0; head < kHalf; ++head) sum[head] *= control.factor[first_head + head];
+                for (uint32_t head = 0; head < kShare; ++head) sum[head] *= control.factor[first_head + head];
                 if (index > 0) {
                     ok = mbar_wait_bounded(bar_product + 8 * ((index - 1) & 1), ((index - 1) >> 1) & 1, p.wait_limit);
                     tcgen05_fence_after();
                     __syncwarp();
-                    // the first half of the warps rescales the high columns, the second the low ones
+                    // the high and the low columns of a block, divided among the warps of the quadrant
+                    constexpr uint32_t kColumns = 2 * N / kSharing;
                     for (uint32_t block = 0; block < p.blocks; ++block) {
 #pragma unroll 1
-                        for (uint32_t part = 0; part < N / 16; ++part) {
-                            const uint32_t address = tmem_out + lane_address + (block * 2 + half) * N + part * 16;
+                        for (uint32_t part = 0; part < kColumns / 16; ++part) {
+                            const uint32_t column = share * kColumns + part * 16;
+                            const uint32_t address = tmem_out + lane_address + block * 2 * N + column;
                             uint32_t raw[16];
                             tmem_load16_nowait(address, raw);
                             tmem_load_wait();
 #pragma unroll
                             for (uint32_t i = 0; i < 16; ++i) {
-                                raw[i] = __float_as_uint(__uint_as_float(raw[i]) * control.factor[part * 16 + i]);
+                                raw[i] = __float_as_uint(__uint_as_float(raw[i]) * control.factor[column % N + i]);
                             }
                             tmem_store16(address, raw);
                         }
@@ -510,7 +528,7 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
             }
             uint8_t* high_rows = smem + p.chunks * N * 128 + buffer * 2 * N * 128 + first_head * 128;
 #pragma unroll
-            for (uint32_t part = 0; part < kHalf / 8; ++part) {
+            for (uint32_t part = 0; part < kShare / 8; ++part) {
                 uint32_t high[4], low[4];
 #pragma unroll
                 for (uint32_t pair = 0; pair < 4; ++pair) {
@@ -539,7 +557,7 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
             if (stage_first + kKeys > position + 1) {
                 const uint32_t exists = position + 1 - stage_first;
                 const uint32_t rows = pages_of(index) * kPageSize - exists;
-                for (uint32_t item = thread; item < rows * p.latent_chunks * 8; item += kSoftmaxWarps * 32) {
+                for (uint32_t item = thread; item < rows * p.latent_chunks * 8; item += kSoftmax) {
                     const uint32_t chunk = item / (rows * 8);
                     const uint32_t row = exists + item / 8 % rows;
                     *reinterpret_cast<uint4*>(ring_bytes + stage * stage_bytes + row / kGroupKeys * group_bytes +
@@ -565,7 +583,7 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
             for (uint32_t block = 0; block < p.blocks; ++block) {
                 const uint32_t dim = block * 128 + quadrant * 32 + lane;
 #pragma unroll
-                for (uint32_t part = 0; part < kHalf / 8; ++part) {
+                for (uint32_t part = 0; part < kShare / 8; ++part) {
                     uint32_t high[8], low[8];
                     const uint32_t address = tmem_out + lane_address + block * 2 * N + first_head + part * 8;
                     tmem_load8_nowait(address, high);
@@ -580,11 +598,11 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
                 }
             }
 #pragma unroll
-            for (uint32_t head = 0; head < kHalf; ++head) {
+            for (uint32_t head = 0; head < kShare; ++head) {
                 const float total = warp_sum(sum[head]);
                 if (lane == 0) control.warp_sum[quadrant][first_head + head] = total;
             }
-            softmax_barrier();
+            softmax_barrier<kSoftmax>();
             if (thread < N) {
                 float total = 0.0f;
 #pragma unroll
@@ -618,27 +636,31 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
     // ---- splits of the token: every CTA of the cluster finishes a share of the outputs.  First what each split counts
     // for, per head, then the weighted sum of the splits' results, four columns at a time with all loads in flight.
     cg::cluster_group cluster = cg::this_cluster();
-    if (threadIdx.x == 0) control.unusable = control.abort | control.missing_page;
-    cluster.sync();
     const uint32_t heads = min(N, p.heads - head0);
+    cluster_wait();           // all have started
+    for (uint32_t item = threadIdx.x; item < heads * p.splits; item += kThreads) {
+        const uint32_t head = item % heads;
+        Control<N>* other = cluster.map_shared_rank(&control, item / heads);
+        other->split_reference[split][head] = control.reference[head];
+        other->split_total[split][head] = control.total[head];
+        if (head == 0) other->split_unusable[split] = control.abort | control.missing_page;
+    }
+    cluster.sync();
+    bool usable = true;
+    for (uint32_t rank = 0; rank < p.splits; ++rank) usable = usable && control.split_unusable[rank] == 0;
     if (threadIdx.x < heads) {
         float reference[kMaxSplits], total[kMaxSplits];
-        uint32_t flags = 0;
 #pragma unroll
         for (uint32_t rank = 0; rank < kMaxSplits; ++rank) {
-            const Control<N>* other = cluster.map_shared_rank(&control, min(rank, p.splits - 1));
-            reference[rank] = other->reference[threadIdx.x];
-            total[rank] = other->total[threadIdx.x];
-            flags |= other->unusable;
+            reference[rank] = rank < p.splits ? control.split_reference[rank][threadIdx.x] : -INFINITY;
+            total[rank] = rank < p.splits ? control.split_total[rank][threadIdx.x] : 0.0f;
         }
-        if (threadIdx.x == 0) control.merged_unusable = flags;
         float best = -INFINITY, sum = 0.0f;
 #pragma unroll
         for (uint32_t rank = 0; rank < kMaxSplits; ++rank) best = fmaxf(best, reference[rank]);
 #pragma unroll
         for (uint32_t rank = 0; rank < kMaxSplits; ++rank) {      // a split that saw no keys counts for nothing
-            reference[rank] =
-                rank >= p.splits || reference[rank] == -INFINITY ? 0.0f : fast_exp2(reference[rank] - best);
+            reference[rank] = reference[rank] == -INFINITY ? 0.0f : fast_exp2(reference[rank] - best);
             sum = fmaf(total[rank], reference[rank], sum);
         }
 #pragma unroll
@@ -649,7 +671,6 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
     __syncthreads();
     const uint32_t quads = p.kv_rank / 4;
     const uint32_t items = heads * quads;
-    const bool usable = control.merged_unusable == 0;
     const uint32_t mine = (items + p.splits - 1) / p.splits;
     const uint32_t last_item = min(items, (split + 1) * mine);
     __nv_bfloat16* target = p.out + (static_cast<size_t>(token) * p.heads + head0) * p.kv_rank;
@@ -774,6 +795,7 @@ cudaError_t launch_heads(cudaStream_t stream, const LatentAttentionLaunch& launc
     params.num_pages = launch.num_pages;
     params.request_slots = launch.request_slots;
     params.positions = launch.positions;
+    params.token_order = launch.token_order;
     params.out = static_cast<__nv_bfloat16*>(launch.out);
     params.status = launch.status;
     params.whole_chunks = whole;
@@ -781,7 +803,7 @@ cudaError_t launch_heads(cudaStream_t stream, const LatentAttentionLaunch& launc
     params.chunks = params.latent_chunks + chunks_of(shape.rot_dim);
     params.blocks = (shape.kv_rank + 127) / 128;
     params.head_blocks = (shape.heads + N - 1) / N;
-    params.splits = latent_attention_splits(launch.tokens * params.head_blocks, launch.context);
+    params.splits = latent_attention_splits(launch.tokens * params.head_blocks, launch.context, params.latent_chunks);
     params.stages = stages_for<N>(shape);
     params.tmem_columns = 32;
     while (params.tmem_columns < (2 * score_sums<N>() + 2 * params.blocks) * N) params.tmem_columns *= 2;
@@ -792,19 +814,29 @@ cudaError_t launch_heads(cudaStream_t stream, const LatentAttentionLaunch& launc
                                                     cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
     if (status != cudaSuccess) return status;
     const size_t blocks = launch.tokens * params.head_blocks * params.splits;
-    return launch_kernel(kernel, static_cast<unsigned int>(blocks), kThreads, shared, stream, params.splits, absorbed_map,
+    return launch_kernel(kernel, static_cast<unsigned int>(blocks), cta_threads(N), shared, stream, params.splits, absorbed_map,
                          rotated_map, latent_map, tail_map, key_map, params);
 }
 
 }  // namespace
 
-// CTAs per token and block of heads over the key axis: enough to even out unequal contexts over the machine while every
-// CTA keeps four stages of the longest one.
-uint32_t latent_attention_splits(size_t ctas, size_t context) {
-    const size_t stages = (context + kKeys - 1) / kKeys;
-    uint32_t splits = 1;
-    while (splits < kMaxSplits && ctas * splits * 2 <= 4 * 148 && stages >= 4 * splits * 2) splits *= 2;
-    return splits;
+// CTAs per token and block of heads over the key axis.  A CTA costs what several stages of keys cost before and behind its
+// own; the splits that minimise the longer of the whole work (contexts taken to be half of the longest on average, handed
+// out longest first) and the longest CTA.
+uint32_t latent_attention_splits(size_t ctas, size_t context, uint32_t latent_chunks) {
+    const double stages = static_cast<double>((context + kKeys - 1) / kKeys);
+    const double overhead = 40.0 / latent_chunks;
+    uint32_t best = 1;
+    double best_cost = 0.0;
+    for (uint32_t splits = 1; splits <= kMaxSplits && splits <= std::max(stages, 1.0); splits *= 2) {
+        const double all = ctas * (stages / 2 + splits * overhead) / 148.0;
+        const double cost = std::max(all, stages / splits + overhead);
+        if (splits == 1 || cost < best_cost) {
+            best = splits;
+            best_cost = cost;
+        }
+    }
+    return best;
 }
 
 bool latent_attention_umma_supports(const LatentAttentionLaunch& launch) {
