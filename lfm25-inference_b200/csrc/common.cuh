@@ -98,6 +98,21 @@ __device__ __forceinline__ bool mbar_try_wait(uint32_t bar, uint32_t parity) {
     return done != 0;
 }
 
+// Whether a phase of a barrier is over, without waiting (mbarrier.try_wait may suspend the thread)
+__device__ __forceinline__ bool mbar_test(uint32_t bar, uint32_t parity) {
+    uint32_t done;
+    asm volatile(
+        "{\n"
+        ".reg .pred p;\n"
+        "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n"
+        "selp.u32 %0, 1, 0, p;\n"
+        "}\n"
+        : "=r"(done)
+        : "r"(bar), "r"(parity)
+        : "memory");
+    return done != 0;
+}
+
 // Waits for a phase of an mbarrier for at most about `limit_ns` of wall time (one second unless the host set another
 // limit, see wait_limit_ns() in options.h).  Returns false when the limit is reached (the caller records the
 // failure and unwinds); it never spins without bound.  The bound is kept on the SM's cycle counter, which is cheap

@@ -28,17 +28,20 @@ constexpr uint32_t kRows = 64;        // tokens per CTA, 16 per warp
 constexpr uint32_t kDepth = 64;       // inputs per round
 constexpr uint32_t kPad = 8;          // elements behind each row of shared memory: conflict-free ldmatrix
 
+constexpr uint32_t kStages = 4;       // rounds in shared memory, one of them being multiplied
+
+template <uint32_t COLUMNS, bool OUTPUT_MAJOR>
+struct Tile {
+    __nv_bfloat16 x[kRows][kDepth + kPad];
+    __nv_bfloat16 w[OUTPUT_MAJOR ? COLUMNS : kDepth][(OUTPUT_MAJOR ? kDepth : COLUMNS) + kPad];
+};
+
 // COLUMNS outputs per CTA.  OUTPUT_MAJOR: the weight's inputs are contiguous (w_k == 1), else its outputs are (w_n == 1).
-// The next round's operands travel through registers while this one is multiplied.
 template <uint32_t COLUMNS, bool OUTPUT_MAJOR>
 __global__ void __launch_bounds__(kThreads)
 head_linear_mma_kernel(const HeadLinearArgs<__nv_bfloat16> args) {
-    constexpr uint32_t kWeightRows = OUTPUT_MAJOR ? COLUMNS : kDepth;
-    constexpr uint32_t kWeightRow = (OUTPUT_MAJOR ? kDepth : COLUMNS) + kPad;
-    constexpr uint32_t kInputVectors = kRows * kDepth / 8 / kThreads;
-    constexpr uint32_t kWeightVectors = COLUMNS * kDepth / 8 / kThreads;
-    __shared__ __align__(16) __nv_bfloat16 x_tile[kRows][kDepth + kPad];
-    __shared__ __align__(16) __nv_bfloat16 w_tile[kWeightRows][kWeightRow];
+    extern __shared__ __align__(16) unsigned char head_linear_smem[];
+    Tile<COLUMNS, OUTPUT_MAJOR>* tiles = reinterpret_cast<Tile<COLUMNS, OUTPUT_MAJOR>*>(head_linear_smem);
     pdl_launch_dependents();
     const uint32_t tile = blockIdx.x % args.column_tiles;
     const uint32_t head = blockIdx.x / args.column_tiles % args.heads;
@@ -48,51 +51,47 @@ head_linear_mma_kernel(const HeadLinearArgs<__nv_bfloat16> args) {
     const __nv_bfloat16* weight = args.weight + head * args.w_head;
     const uint32_t warp = threadIdx.x >> 5;
     const uint32_t lane = threadIdx.x & 31;
-    uint4 x_next[kInputVectors], w_next[kWeightVectors];
-    auto load_weight = [&](uint32_t depth) {
+    const uint32_t rounds = (args.k + kDepth - 1) / kDepth;
+    auto load_weight = [&](uint32_t round) {
+        auto& target = tiles[round % kStages].w;
 #pragma unroll
-        for (uint32_t part = 0; part < kWeightVectors; ++part) {
+        for (uint32_t part = 0; part < COLUMNS * kDepth / 8 / kThreads; ++part) {
             const uint32_t item = threadIdx.x + part * kThreads;
             constexpr uint32_t kPerRow = (OUTPUT_MAJOR ? kDepth : COLUMNS) / 8;
             const uint32_t outer = item / kPerRow, inner = item % kPerRow * 8;
             const uint32_t n = column0 + (OUTPUT_MAJOR ? outer : inner);
-            const uint32_t k = depth + (OUTPUT_MAJOR ? inner : outer);
-            w_next[part] = n < args.n && k < args.k
-                               ? *reinterpret_cast<const uint4*>(weight + n * args.w_n + k * args.w_k)
-                               : make_uint4(0, 0, 0, 0);
+            const uint32_t k = round * kDepth + (OUTPUT_MAJOR ? inner : outer);
+            const bool inside = n < args.n && k < args.k;
+            copy_async_16(&target[outer][inner], weight + (inside ? n * args.w_n + k * args.w_k : 0), inside);
         }
     };
-    auto load_input = [&](uint32_t depth) {
+    auto load_input = [&](uint32_t round) {
+        auto& target = tiles[round % kStages].x;
 #pragma unroll
-        for (uint32_t part = 0; part < kInputVectors; ++part) {
+        for (uint32_t part = 0; part < kRows * kDepth / 8 / kThreads; ++part) {
             const uint32_t item = threadIdx.x + part * kThreads;
-            const uint32_t row = row0 + item / (kDepth / 8), k = depth + item % (kDepth / 8) * 8;
-            x_next[part] = row < args.tokens && k < args.k
-                               ? *reinterpret_cast<const uint4*>(x + row * args.x_pitch + k)
-                               : make_uint4(0, 0, 0, 0);
+            const uint32_t row = item / (kDepth / 8), inner = item % (kDepth / 8) * 8;
+            const bool inside = row0 + row < args.tokens && round * kDepth + inner < args.k;
+            copy_async_16(&target[row][inner], x + (inside ? (row0 + row) * args.x_pitch + round * kDepth + inner : 0), inside);
         }
     };
-    load_weight(0);
+    for (uint32_t round = 0; round < kStages - 1 && round < rounds; ++round) load_weight(round);
     pdl_wait();
-    load_input(0);
+    for (uint32_t round = 0; round < kStages - 1; ++round) {
+        if (round < rounds) load_input(round);
+        copy_async_commit();
+    }
     float sum[COLUMNS / 8][4] = {};
-    for (uint32_t depth = 0; depth < args.k; depth += kDepth) {
-#pragma unroll
-        for (uint32_t part = 0; part < kInputVectors; ++part) {
-            const uint32_t item = threadIdx.x + part * kThreads;
-            *reinterpret_cast<uint4*>(&x_tile[item / (kDepth / 8)][item % (kDepth / 8) * 8]) = x_next[part];
-        }
-#pragma unroll
-        for (uint32_t part = 0; part < kWeightVectors; ++part) {
-            const uint32_t item = threadIdx.x + part * kThreads;
-            constexpr uint32_t kPerRow = (OUTPUT_MAJOR ? kDepth : COLUMNS) / 8;
-            *reinterpret_cast<uint4*>(&w_tile[item / kPerRow][item % kPerRow * 8]) = w_next[part];
-        }
+    for (uint32_t round = 0; round < rounds; ++round) {
+        copy_async_wait<kStages - 2>();
         __syncthreads();
-        if (depth + kDepth < args.k) {
-            load_weight(depth + kDepth);
-            load_input(depth + kDepth);
+        if (round + kStages - 1 < rounds) {
+            load_weight(round + kStages - 1);
+            load_input(round + kStages - 1);
         }
+        copy_async_commit();
+        const auto& x_tile = tiles[round % kStages].x;
+        const auto& w_tile = tiles[round % kStages].w;
 #pragma unroll
         for (uint32_t step = 0; step < kDepth / 16; ++step) {
             uint32_t a0, a1, a2, a3;
@@ -113,7 +112,6 @@ head_linear_mma_kernel(const HeadLinearArgs<__nv_bfloat16> args) {
                 mma_bf16_16816(sum[2 * pair + 1], a0, a1, a2, a3, b2, b3);
             }
         }
-        __syncthreads();
     }
 #pragma unroll
     for (uint32_t part = 0; part < 2; ++part) {
@@ -244,9 +242,13 @@ cudaError_t launch_mma(cudaStream_t stream, const HeadLinearLaunch& launch) {
     HeadLinearArgs<__nv_bfloat16> args = typed_args<__nv_bfloat16>(launch);
     args.column_tiles = (args.n + COLUMNS - 1) / COLUMNS;
     const size_t blocks = static_cast<size_t>(args.column_tiles) * args.heads * ((args.tokens + kRows - 1) / kRows);
-    const auto kernel =
-        launch.w_k == 1 ? head_linear_mma_kernel<COLUMNS, true> : head_linear_mma_kernel<COLUMNS, false>;
-    return launch_kernel(kernel, static_cast<unsigned int>(blocks), kThreads, 0, stream, 1, args);
+    const bool output_major = launch.w_k == 1;
+    const auto kernel = output_major ? head_linear_mma_kernel<COLUMNS, true> : head_linear_mma_kernel<COLUMNS, false>;
+    const size_t shared = kStages * (output_major ? sizeof(Tile<COLUMNS, true>) : sizeof(Tile<COLUMNS, false>));
+    const cudaError_t status = cudaFuncSetAttribute(reinterpret_cast<const void*>(kernel),
+                                                    cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
+    if (status != cudaSuccess) return status;
+    return launch_kernel(kernel, static_cast<unsigned int>(blocks), kThreads, shared, stream, 1, args);
 }
 
 }  // namespace

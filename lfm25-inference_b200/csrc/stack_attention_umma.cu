@@ -113,7 +113,7 @@ stack_attention_umma_kernel(const __grid_constant__ CUtensorMap query_map, const
                             const __grid_constant__ CUtensorMap value_map, const __grid_constant__ CUtensorMap shared_map,
                             const Params p) {
     using L = Layout<KC, VC>;
-    const uint32_t warp = threadIdx.x >> 5;
+    const uint32_t warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0);     // the same value to the compiler's eye as well
     const uint32_t lane = threadIdx.x & 31;
     pdl_launch_dependents();
     pdl_wait();
@@ -190,7 +190,7 @@ stack_attention_umma_kernel(const __grid_constant__ CUtensorMap query_map, const
 
     if (warp == 0) {
         // ------------------------------------------------------------------------------------ producer
-        if (lane == 0) {
+        if (elect_one()) {
             mbar_arrive_expect_tx(bar_q, KC * group * p.tile_tokens * 128);
             for (uint32_t chunk = 0; chunk < KC; ++chunk) {
                 // a query dimension beyond a part of the head meets a key dimension that the copy filled with zero
@@ -269,7 +269,7 @@ stack_attention_umma_kernel(const __grid_constant__ CUtensorMap query_map, const
         }
     } else if (warp == 1) {
         // ------------------------------------------------------------------------------------ MMA issuer
-        if (lane == 0) {
+        if (elect_one()) {
             // D = f32, A = B = bf16, M = 128; S: both K-major, N = keys of the stage; PV: B (the V rows) MN-major, N = 64
             const uint32_t idesc_common = (1u << 4) | (1u << 7) | (1u << 10) | ((kRows >> 4) << 24);
             const uint32_t idesc_pv = idesc_common | (1u << 16) | ((64u >> 3) << 17);

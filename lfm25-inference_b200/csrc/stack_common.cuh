@@ -79,6 +79,17 @@ __device__ __forceinline__ void store_values(float* target, const float (&values
     }
 }
 
+// 16 bytes global -> shared behind the thread's back; `inside` false: zeros (the source is not read)
+__device__ __forceinline__ void copy_async_16(void* target, const void* source, bool inside) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(target)), "l"(source), "r"(inside ? 16 : 0)
+                 : "memory");
+}
+__device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <uint32_t NEWER>
+__device__ __forceinline__ void copy_async_wait() {
+    asm volatile("cp.async.wait_group %0;" ::"n"(NEWER) : "memory");
+}
+
 __device__ __forceinline__ float warp_sum(float value) {
 #pragma unroll
     for (uint32_t delta = 16; delta > 0; delta >>= 1) {

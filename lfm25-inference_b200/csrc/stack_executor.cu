@@ -41,7 +41,7 @@ struct lfm25_stack_executor {
     void* joined;              // [T, widest output.k]: mixer output | activation
     void* update;              // [T, width]
     void* head_input;          // [R, width]
-    void* logits;              // [R, head.n]
+    void* logits;              // [R, head.n], before a cap
     float* raw;                // [T, widest heads * dim] when a delta rule needs it
     void* compressed;          // [T, widest q_rank]: latent attention's query latent
     void* absorbed;            // [T, widest heads * kv_rank]: queries against latents
@@ -56,6 +56,8 @@ struct lfm25_stack_executor {
     size_t context_capacity = 0;
     const void* last_post = nullptr;   // norm between `update` and the residual stream of the last step
     uint32_t* sampled;         // [R]
+    float* exported = nullptr; // [rows, vocab] logits on their way to the host, grown when asked for
+    size_t exported_bytes = 0;
     size_t last_tokens = 0;
     const float* last_residual = nullptr;
     std::vector<unsigned char> staging;
@@ -649,7 +651,7 @@ int32_t enqueue(lfm25_stack_executor* self, const Step& step) {
     }
     STACK_TRY(linear(self, model.head, self->head_input, self->logits, step.num_outputs));
     STACK_CUDA(lfm25::launch_argmax_rows(stream, self->type, self->logits, model.head.n, self->sampled, step.num_outputs,
-                                         model.vocab, model.logit_softcap),
+                                         model.vocab),
                "argmax launch failed");
     return LFM25_OK;
 }
@@ -848,6 +850,7 @@ int32_t lfm25_stack_executor_create(lfm25_blaslt* blaslt, const lfm25_stack_mode
 void lfm25_stack_executor_destroy(lfm25_stack_executor* self) {
     if (self == nullptr) return;
     cudaFree(self->allocation);
+    cudaFree(self->exported);
     delete self;
 }
 
@@ -923,26 +926,21 @@ int32_t lfm25_stack_executor_read_logits(lfm25_stack_executor* self, float* host
         return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "logits read exceeds the executor's capacity");
     }
     const lfm25_stack_model& model = *self->model;
-    const size_t bytes = lfm25::activation_bytes(self->type);
     cudaStream_t stream = self->blaslt->stream;
-    if (self->type == Activation::kF32) {
-        STACK_CUDA(cudaMemcpy2DAsync(host, model.vocab * 4, self->logits, model.head.n * 4, model.vocab * 4, rows,
-                                     cudaMemcpyDeviceToHost, stream),
-                   "logits download failed");
-        STACK_CUDA(cudaStreamSynchronize(stream), "logits download failed");
-        return LFM25_OK;
+    const size_t bytes = rows * model.vocab * sizeof(float);
+    if (bytes == 0) return LFM25_OK;
+    if (bytes > self->exported_bytes) {
+        cudaFree(self->exported);
+        self->exported = nullptr;
+        self->exported_bytes = 0;
+        STACK_CUDA(cudaMalloc(reinterpret_cast<void**>(&self->exported), bytes), "failed to allocate logits for export");
+        self->exported_bytes = bytes;
     }
-    self->staging.resize(rows * model.vocab * bytes);
-    STACK_CUDA(cudaMemcpy2DAsync(self->staging.data(), model.vocab * bytes, self->logits, model.head.n * bytes,
-                                 model.vocab * bytes, rows, cudaMemcpyDeviceToHost, stream),
-               "logits download failed");
+    STACK_CUDA(lfm25::launch_export_logits(stream, self->type, self->logits, model.head.n, self->exported, rows, model.vocab,
+                                           model.logit_softcap),
+               "logits export launch failed");
+    STACK_CUDA(cudaMemcpyAsync(host, self->exported, bytes, cudaMemcpyDeviceToHost, stream), "logits download failed");
     STACK_CUDA(cudaStreamSynchronize(stream), "logits download failed");
-    for (size_t index = 0; index < rows * model.vocab; ++index) {
-        uint16_t half;
-        memcpy(&half, self->staging.data() + index * 2, 2);
-        const uint32_t word = static_cast<uint32_t>(half) << 16;
-        memcpy(host + index, &word, 4);
-    }
     return LFM25_OK;
 }
 

@@ -94,10 +94,14 @@ cudaError_t launch_poly_norm(cudaStream_t stream, Activation type, const void* z
                              size_t out_pitch, size_t rows, size_t width, size_t pad, const float coefficients[4],
                              float eps);
 
-// Greedy choice: index of the row's largest logit, the lowest index among equals; NaN never wins.  softcap > 0: the
-// logits become softcap * tanh(logits / softcap) first, in place.
-cudaError_t launch_argmax_rows(cudaStream_t stream, Activation type, void* logits, size_t pitch, uint32_t* sampled,
-                               size_t rows, size_t vocab, float softcap);
+// Greedy choice: index of the row's largest logit, the lowest index among equals; NaN never wins.  A cap on the logits
+// keeps their order, so the choice is made before it.
+cudaError_t launch_argmax_rows(cudaStream_t stream, Activation type, const void* logits, size_t pitch,
+                               uint32_t* sampled, size_t rows, size_t vocab);
+
+// out[r, v] = the logit as f32; softcap > 0: softcap * tanh(logit / softcap)
+cudaError_t launch_export_logits(cudaStream_t stream, Activation type, const void* logits, size_t pitch, float* out,
+                                 size_t rows, size_t vocab, float softcap);
 
 // y[m, n] = sum_k x[m, k] w[n, k] with plain 32-bit multiply-adds: the matrix product of the f32 activation type and
 // of bf16 shapes that the tensor-core paths cannot take.

@@ -54,7 +54,7 @@ __device__ __forceinline__ int64_t latent_row(const LatentArgs<T>& args, size_t 
     return page < args.num_pages ? static_cast<int64_t>(page * kPageSize + position % kPageSize) : -1;
 }
 
-uint32_t latent_attention_splits(size_t ctas, size_t context, uint32_t latent_chunks);
+uint32_t latent_attention_splits(size_t clusters, size_t context, uint32_t latent_chunks);
 bool latent_attention_umma_supports(const LatentAttentionLaunch& launch);
 cudaError_t launch_latent_attention_umma(cudaStream_t stream, const LatentAttentionLaunch& launch);
 

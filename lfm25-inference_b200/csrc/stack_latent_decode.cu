@@ -112,35 +112,6 @@ __device__ __forceinline__ void mma_shared(uint32_t tmem_d, uint64_t desc_a, uin
         : "memory");
 }
 
-// One lane of a converged warp.  Chosen this way, unlike by its number, the compiler knows that a single lane runs the
-// branch and keeps the operands of tcgen05.mma in uniform registers: 28 cycles per MMA instead of 75.
-__device__ __forceinline__ bool elect_one() {
-    uint32_t chosen;
-    asm volatile(
-        "{\n"
-        ".reg .pred p;\n"
-        "elect.sync _|p, 0xffffffff;\n"
-        "selp.u32 %0, 1, 0, p;\n"
-        "}\n"
-        : "=r"(chosen));
-    return chosen != 0;
-}
-
-// Whether a phase of a barrier is over, without waiting (mbarrier.try_wait may suspend the thread)
-__device__ __forceinline__ bool mbar_test(uint32_t bar, uint32_t parity) {
-    uint32_t done;
-    asm volatile(
-        "{\n"
-        ".reg .pred p;\n"
-        "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n"
-        "selp.u32 %0, 1, 0, p;\n"
-        "}\n"
-        : "=r"(done)
-        : "r"(bar), "r"(parity)
-        : "memory");
-    return done != 0;
-}
-
 __device__ __forceinline__ void load_3d(uint32_t dst, const void* tensor_map, uint32_t bar, int32_t x, int32_t y, int32_t z) {
     asm volatile(
         "cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
@@ -821,16 +792,21 @@ cudaError_t launch_heads(cudaStream_t stream, const LatentAttentionLaunch& launc
 }  // namespace
 
 // CTAs per token and block of heads over the key axis.  A CTA costs what several stages of keys cost before and behind its
-// own; the splits that minimise the longer of the whole work (contexts taken to be half of the longest on average, handed
-// out longest first) and the longest CTA.
-uint32_t latent_attention_splits(size_t ctas, size_t context, uint32_t latent_chunks) {
+// own, and the larger a cluster is, the fewer SMs its shape lets the machine use (one CTA per SM; cluster counts as the
+// occupancy calculator reports them).  The cheapest split when contexts are half of the longest on average and handed out
+// longest first.
+uint32_t latent_attention_splits(size_t clusters, size_t context, uint32_t latent_chunks) {
+    constexpr size_t kResident[] = {148, 74, 33, 15};            // clusters of 1, 2, 4, 8 CTAs
     const double stages = static_cast<double>((context + kKeys - 1) / kKeys);
     const double overhead = 40.0 / latent_chunks;
     uint32_t best = 1;
     double best_cost = 0.0;
-    for (uint32_t splits = 1; splits <= kMaxSplits && splits <= std::max(stages, 1.0); splits *= 2) {
-        const double all = ctas * (stages / 2 + splits * overhead) / 148.0;
-        const double cost = std::max(all, stages / splits + overhead);
+    for (uint32_t step = 0; step < 4; ++step) {
+        const uint32_t splits = 1u << step;
+        if (splits > 1 && splits > stages) break;
+        const size_t waves = (clusters + kResident[step] - 1) / kResident[step];
+        const double longest = stages / splits + overhead;
+        const double cost = std::max(longest, waves * (stages / (2 * splits) + overhead));
         if (splits == 1 || cost < best_cost) {
             best = splits;
             best_cost = cost;

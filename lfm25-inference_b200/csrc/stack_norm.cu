@@ -509,22 +509,15 @@ __device__ __forceinline__ Candidate warp_best(Candidate best) {
 constexpr uint32_t kArgmaxThreads = 512;
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kArgmaxThreads)
-argmax_kernel(T* __restrict__ logits, size_t pitch, uint32_t* __restrict__ sampled, uint32_t vocab, float softcap) {
+argmax_kernel(const T* __restrict__ logits, size_t pitch, uint32_t* __restrict__ sampled, uint32_t vocab) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ Candidate held[kArgmaxThreads / 32];
-    T* row = logits + blockIdx.x * pitch;
+    const T* row = logits + blockIdx.x * pitch;
     Candidate best = {-INFINITY, 0xffffffffu};
     for (uint32_t column = threadIdx.x * VEC; column < vocab; column += kArgmaxThreads * VEC) {
         float value[VEC];
         load_values<VEC>(row + column, value);
-        if (softcap > 0.0f) {
-            // the choice is made among the uncapped logits: tanh keeps the order but not small differences
-            float capped[VEC];
-#pragma unroll
-            for (int i = 0; i < VEC; ++i) capped[i] = softcap * tanhf(value[i] / softcap);
-            store_values<VEC>(row + column, capped);
-        }
 #pragma unroll
         for (int i = 0; i < VEC; ++i) {
             if (value[i] > best.value || (value[i] == best.value && column + i < best.index)) {
@@ -544,6 +537,20 @@ argmax_kernel(T* __restrict__ logits, size_t pitch, uint32_t* __restrict__ sampl
         if (lane == 0) {
             sampled[blockIdx.x] = best.index < vocab ? best.index : 0u;
         }
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+export_logits_kernel(const T* __restrict__ logits, size_t pitch, float* __restrict__ out, size_t vocab, float softcap) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t blocks = (vocab + kThreads - 1) / kThreads;
+    const size_t row = blockIdx.x / blocks;
+    const size_t column = blockIdx.x % blocks * kThreads + threadIdx.x;
+    if (column < vocab) {
+        const float value = to_float<T>(logits[row * pitch + column]);
+        out[row * vocab + column] = softcap > 0.0f ? softcap * tanhf(value / softcap) : value;
     }
 }
 
@@ -766,13 +773,13 @@ cudaError_t launch_squared_relu(cudaStream_t stream, Activation type, void* z, s
     return vector ? go(tag, squared_relu_kernel<__nv_bfloat16, 8>) : go(tag, squared_relu_kernel<__nv_bfloat16, 1>);
 }
 
-cudaError_t launch_argmax_rows(cudaStream_t stream, Activation type, void* logits, size_t pitch, uint32_t* sampled,
-                               size_t rows, size_t vocab, float softcap) {
+cudaError_t launch_argmax_rows(cudaStream_t stream, Activation type, const void* logits, size_t pitch,
+                               uint32_t* sampled, size_t rows, size_t vocab) {
     const bool vector = vocab % 8 == 0 && pitch % 8 == 0 && aligned_to(logits, 16);
     auto go = [&](auto* typed, auto kernel) {
         using T = std::remove_pointer_t<decltype(typed)>;
         return launch_kernel(kernel, static_cast<unsigned int>(rows), kArgmaxThreads, 0, stream, 1,
-                             static_cast<T*>(logits), pitch, sampled, static_cast<uint32_t>(vocab), softcap);
+                             static_cast<const T*>(logits), pitch, sampled, static_cast<uint32_t>(vocab));
     };
     if (type == Activation::kF32) {
         float* tag = nullptr;
@@ -780,6 +787,17 @@ cudaError_t launch_argmax_rows(cudaStream_t stream, Activation type, void* logit
     }
     __nv_bfloat16* tag = nullptr;
     return vector ? go(tag, argmax_kernel<__nv_bfloat16, 8>) : go(tag, argmax_kernel<__nv_bfloat16, 1>);
+}
+
+cudaError_t launch_export_logits(cudaStream_t stream, Activation type, const void* logits, size_t pitch, float* out,
+                                 size_t rows, size_t vocab, float softcap) {
+    const unsigned int blocks = static_cast<unsigned int>((vocab + kThreads - 1) / kThreads * rows);
+    if (type == Activation::kF32) {
+        return launch_kernel(export_logits_kernel<float>, blocks, kThreads, 0, stream, 1, static_cast<const float*>(logits),
+                             pitch, out, vocab, softcap);
+    }
+    return launch_kernel(export_logits_kernel<__nv_bfloat16>, blocks, kThreads, 0, stream, 1,
+                         static_cast<const __nv_bfloat16*>(logits), pitch, out, vocab, softcap);
 }
 
 cudaError_t launch_linear_simt(cudaStream_t stream, Activation type, const void* x, const void* weight, void* y,

@@ -14,6 +14,35 @@ namespace {
 
 // ------------------------------------------------------------------------------------------------ channel convolution
 
+// The logistic function, to the accuracy that a result in T can show
+template <typename T>
+__device__ __forceinline__ float sigmoid_of(float z) {
+    return sizeof(T) == 4 ? sigmoidf(z) : __fdividef(1.0f, 1.0f + __expf(-z));
+}
+
+// VEC consecutive values as they lie in memory
+template <typename T, int VEC>
+struct Vector {
+    static constexpr int kWords = VEC * sizeof(T) >= 16 ? VEC * sizeof(T) / 16 : 1;
+    uint4 words[kWords];
+    T single;
+    __device__ __forceinline__ void load(const T* source) {
+        if constexpr (VEC == 1) {
+            single = *source;
+        } else {
+#pragma unroll
+            for (int i = 0; i < kWords; ++i) words[i] = reinterpret_cast<const uint4*>(source)[i];
+        }
+    }
+    __device__ __forceinline__ void values(float (&out)[VEC]) const {
+        if constexpr (VEC == 1) {
+            out[0] = to_float<T>(single);
+        } else {
+            load_values<VEC>(reinterpret_cast<const T*>(words), out);
+        }
+    }
+};
+
 constexpr uint32_t kConvThreads = 128;
 constexpr uint32_t kConvRows = 16;
 
@@ -77,22 +106,32 @@ channel_conv_kernel(const ConvArgs<T> args) {
         float window[TAPS][VEC];
 #pragma unroll
         for (int j = 1; j < TAPS; ++j) load_input(first - (TAPS - j), window[j]);
-        for (uint32_t row = 0; row < tile.count; ++row) {
+        constexpr uint32_t kBatch = 8;               // rows whose loads are in flight together
+        for (uint32_t base = 0; base < tile.count; base += kBatch) {
+            Vector<T, VEC> next[kBatch];
 #pragma unroll
-            for (int j = 0; j + 1 < TAPS; ++j) {
-#pragma unroll
-                for (int i = 0; i < VEC; ++i) window[j][i] = window[j + 1][i];
+            for (uint32_t i = 0; i < kBatch; ++i) {
+                if (base + i < tile.count) next[i].load(inputs + (first + base + i) * args.pitch);
             }
-            load_values<VEC>(inputs + (first + row) * args.pitch, window[TAPS - 1]);
-            float sum[VEC];
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) {
-                sum[i] = bias[i];
+            for (uint32_t step = 0; step < kBatch; ++step) {
+                if (base + step >= tile.count) break;
 #pragma unroll
-                for (int j = 0; j < TAPS; ++j) sum[i] = fmaf(tap[j][i], window[j][i], sum[i]);
-                sum[i] *= sigmoidf(sum[i]);
+                for (int j = 0; j + 1 < TAPS; ++j) {
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) window[j][i] = window[j + 1][i];
+                }
+                next[step].values(window[TAPS - 1]);
+                float sum[VEC];
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) {
+                    sum[i] = bias[i];
+#pragma unroll
+                    for (int j = 0; j < TAPS; ++j) sum[i] = fmaf(tap[j][i], window[j][i], sum[i]);
+                    sum[i] *= sigmoid_of<T>(sum[i]);
+                }
+                store_values<VEC>(out + (base + step) * args.channels, sum);
             }
-            store_values<VEC>(out + row * args.channels, sum);
         }
     } else {
         for (uint32_t row = 0; row < tile.count; ++row) {
@@ -106,7 +145,7 @@ channel_conv_kernel(const ConvArgs<T> args) {
                 for (int i = 0; i < VEC; ++i) sum[i] = fmaf(weight[i], value[i], sum[i]);
             }
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) sum[i] *= sigmoidf(sum[i]);
+            for (int i = 0; i < VEC; ++i) sum[i] *= sigmoid_of<T>(sum[i]);
             store_values<VEC>(out + row * args.channels, sum);
         }
     }
@@ -360,47 +399,77 @@ cudaError_t launch_scan(cudaStream_t stream, const StateSpaceLaunch& launch) {
 
 // ------------------------------------------------------------------------------------------------ gated norm
 
-template <typename T, int VEC>
+// One warp per row and part where a part fits the registers of a warp (HELD vectors per lane), else one CTA.
+template <typename T, int VEC, int HELD>
 __global__ void __launch_bounds__(512)
 gated_group_norm_kernel(const T* __restrict__ y, const T* __restrict__ z, size_t z_pitch,
-                        const __nv_bfloat16* __restrict__ norm, T* __restrict__ out, size_t out_pitch, size_t width,
-                        uint32_t groups, float eps) {
+                        const __nv_bfloat16* __restrict__ norm, T* __restrict__ out, size_t out_pitch, size_t tokens,
+                        size_t width, uint32_t groups, float eps) {
     pdl_launch_dependents();
     __shared__ float scratch[16];
     pdl_wait();
-    const size_t token = blockIdx.x / groups;
     const size_t part = width / groups;
-    const size_t first = blockIdx.x % groups * part;
-    auto gated = [&](size_t column, float (&value)[VEC]) {
+    auto gated = [&](size_t token, size_t column, float (&value)[VEC]) {
         float gate[VEC];
-        load_values<VEC>(y + token * width + first + column, value);
-        load_values<VEC>(z + token * z_pitch + first + column, gate);
+        load_values<VEC>(y + token * width + column, value);
+        load_values<VEC>(z + token * z_pitch + column, gate);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) value[i] *= gate[i] * sigmoidf(gate[i]);
+        for (int i = 0; i < VEC; ++i) value[i] *= gate[i] * sigmoid_of<T>(gate[i]);
     };
-    auto emit = [&](size_t column, float (&value)[VEC], float scale) {
+    auto emit = [&](size_t token, size_t column, float (&value)[VEC], float scale) {
         float weight[VEC];
-        load_values<VEC>(norm + first + column, weight);
+        load_values<VEC>(norm + column, weight);
 #pragma unroll
         for (int i = 0; i < VEC; ++i) value[i] *= scale * weight[i];
-        store_values<VEC>(out + token * out_pitch + first + column, value);
+        store_values<VEC>(out + token * out_pitch + column, value);
     };
-    // the first vector of every thread stays in registers
-    float held[VEC], sum = 0.0f;
-    const size_t mine = threadIdx.x * VEC;
-    for (size_t column = mine; column < part; column += blockDim.x * VEC) {
-        float value[VEC];
-        gated(column, value);
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) {
-            sum = fmaf(value[i], value[i], sum);
-            if (column == mine) held[i] = value[i];
+    float sum = 0.0f;
+    if constexpr (HELD > 0) {
+        const size_t item = static_cast<size_t>(blockIdx.x) * (blockDim.x / 32) + threadIdx.x / 32;
+        if (item >= tokens * groups) {
+            return;
         }
-    }
-    const float scale = inverse_rms(block_sum(sum, scratch), part, eps);
-    for (size_t column = mine; column < part; column += blockDim.x * VEC) {
-        if (column != mine) gated(column, held);
-        emit(column, held, scale);
+        const size_t token = item / groups;
+        const size_t first = item % groups * part;
+        const size_t mine = (threadIdx.x & 31) * VEC;
+        float held[HELD][VEC];
+#pragma unroll
+        for (int step = 0; step < HELD; ++step) {
+            const size_t column = mine + step * 32 * VEC;
+            if (column < part) gated(token, first + column, held[step]);
+        }
+#pragma unroll
+        for (int step = 0; step < HELD; ++step) {
+            if (mine + step * 32 * VEC < part) {
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) sum = fmaf(held[step][i], held[step][i], sum);
+            }
+        }
+        const float scale = inverse_rms(warp_sum(sum), part, eps);
+#pragma unroll
+        for (int step = 0; step < HELD; ++step) {
+            const size_t column = mine + step * 32 * VEC;
+            if (column < part) emit(token, first + column, held[step], scale);
+        }
+    } else {
+        const size_t token = blockIdx.x / groups;
+        const size_t first = blockIdx.x % groups * part;
+        const size_t mine = threadIdx.x * VEC;
+        float held[VEC];                       // the thread's first vector stays in registers
+        for (size_t column = mine; column < part; column += blockDim.x * VEC) {
+            float value[VEC];
+            gated(token, first + column, value);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) {
+                sum = fmaf(value[i], value[i], sum);
+                if (column == mine) held[i] = value[i];
+            }
+        }
+        const float scale = inverse_rms(block_sum(sum, scratch), part, eps);
+        for (size_t column = mine; column < part; column += blockDim.x * VEC) {
+            if (column != mine) gated(token, first + column, held);
+            emit(token, first + column, held, scale);
+        }
     }
 }
 
@@ -436,20 +505,25 @@ cudaError_t launch_gated_group_norm(cudaStream_t stream, const GatedGroupNormLau
     const bool vector = part % 8 == 0 && launch.z_pitch % 8 == 0 && launch.out_pitch % 8 == 0 && aligned_to(launch.y, 16) &&
                         aligned_to(launch.z, 16) && aligned_to(launch.norm, 16) && aligned_to(launch.out, 16);
     const size_t vectors = vector ? part / 8 : part;
-    const unsigned int threads = static_cast<unsigned int>(std::min<size_t>((vectors + 31) / 32 * 32, 512));
+    const size_t items = launch.tokens * launch.groups;
+    const bool warps = vector && vectors <= 64;
+    const unsigned int threads = warps ? 128 : static_cast<unsigned int>(std::min<size_t>((vectors + 31) / 32 * 32, 512));
+    const unsigned int blocks = static_cast<unsigned int>(warps ? (items + 3) / 4 : items);
     auto go = [&](auto* typed, auto kernel) {
         using T = std::remove_pointer_t<decltype(typed)>;
-        return launch_kernel(kernel, static_cast<unsigned int>(launch.tokens * launch.groups), threads, 0, stream, 1,
-                             static_cast<const T*>(launch.y), static_cast<const T*>(launch.z), launch.z_pitch,
-                             static_cast<const __nv_bfloat16*>(launch.norm), static_cast<T*>(launch.out), launch.out_pitch,
-                             launch.width, launch.groups, launch.eps);
+        return launch_kernel(kernel, blocks, threads, 0, stream, 1, static_cast<const T*>(launch.y),
+                             static_cast<const T*>(launch.z), launch.z_pitch, static_cast<const __nv_bfloat16*>(launch.norm),
+                             static_cast<T*>(launch.out), launch.out_pitch, launch.tokens, launch.width, launch.groups,
+                             launch.eps);
     };
-    if (launch.type == Activation::kF32) {
-        float* tag = nullptr;
-        return vector ? go(tag, gated_group_norm_kernel<float, 8>) : go(tag, gated_group_norm_kernel<float, 1>);
-    }
-    __nv_bfloat16* tag = nullptr;
-    return vector ? go(tag, gated_group_norm_kernel<__nv_bfloat16, 8>) : go(tag, gated_group_norm_kernel<__nv_bfloat16, 1>);
+    auto sized = [&](auto* typed) {
+        using T = std::remove_pointer_t<decltype(typed)>;
+        if (!vector) return go(typed, gated_group_norm_kernel<T, 1, 0>);
+        if (!warps) return go(typed, gated_group_norm_kernel<T, 8, 0>);
+        return vectors <= 32 ? go(typed, gated_group_norm_kernel<T, 8, 1>) : go(typed, gated_group_norm_kernel<T, 8, 2>);
+    };
+    return launch.type == Activation::kF32 ? sized(static_cast<float*>(nullptr))
+                                           : sized(static_cast<__nv_bfloat16*>(nullptr));
 }
 
 }  // namespace lfm25

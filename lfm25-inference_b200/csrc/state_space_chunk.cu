@@ -37,13 +37,6 @@ constexpr size_t shared_bytes(uint32_t padded, uint32_t buffers) {
     return buffers * chunk_bytes(padded) + 2 * (padded + kTokens) * kColumnPitch * 2 + sizeof(Tables);
 }
 
-__device__ __forceinline__ void copy_async(void* target, const void* source, bool inside) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(target)), "l"(source), "r"(inside ? 16 : 0)
-                 : "memory");
-}
-__device__ __forceinline__ void copies_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-__device__ __forceinline__ void copies_wait() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
-
 __device__ __forceinline__ void split_pair(float a, float b, uint32_t& high, uint32_t& low) {
     high = pack_bf16x2(a, b);
     const float2 rounded = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&high));
@@ -97,19 +90,19 @@ state_space_chunk_kernel(const StateSpaceArgs<__nv_bfloat16> args, uint32_t colu
             const bool inside = first + row < end && n < args.size;
             const __nv_bfloat16* source =
                 args.mixed + (inside ? static_cast<size_t>(first + row) * args.mixed_pitch + inner + group * args.size + n : 0);
-            copy_async(b + row * pitch + n, source, inside);
-            copy_async(c + row * pitch + n, source + (inside ? args.groups * args.size : 0), inside);
+            copy_async_16(b + row * pitch + n, source, inside);
+            copy_async_16(c + row * pitch + n, source + (inside ? args.groups * args.size : 0), inside);
         }
         for (uint32_t item = threadIdx.x; item < kTokens * kColumns / 8; item += kThreads) {
             const uint32_t row = item / (kColumns / 8), v = item % (kColumns / 8) * 8;
             const bool inside = first + row < end && column0 + v < args.vdim;
-            copy_async(x + row * kColumnPitch + v,
+            copy_async_16(x + row * kColumnPitch + v,
                        args.mixed + (inside ? static_cast<size_t>(first + row) * args.mixed_pitch + head * args.vdim +
                                                   column0 + v
                                             : 0),
                        inside);
         }
-        copies_commit();
+        copy_async_commit();
     };
     // warp 0: step sizes of a chunk, two tokens per lane
     auto load_steps = [&](uint32_t first, float (&steps)[2]) {
@@ -168,7 +161,7 @@ state_space_chunk_kernel(const StateSpaceArgs<__nv_bfloat16> args, uint32_t colu
             }
             if (first + kTokens < end) load_steps(first + kTokens, steps);
         }
-        copies_wait();
+        copy_async_wait<0>();
         __syncthreads();
         if (buffers == 2 && first + kTokens < end) load_chunk(first + kTokens, buffer ^ 1);
         const __nv_bfloat16* b = tiles + buffer * tile_elements;
