@@ -457,3 +457,65 @@ def test_captured_steps_match_eager_ones(device, mixed_case):
             executor.close()
             blaslt.close()
     assert np.array_equal(produced[0], produced[1])
+
+
+def test_command_line_and_trace_replay(device, mixed_case, tmp_path):
+    """A model folder through the two programs, each in a process of its own."""
+    import json
+    import os
+    import subprocess
+    import sys
+
+    import torch
+
+    from lfm25_inference_b200 import checkpoint
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    config, tensors, tokens, want = mixed_case
+    (tmp_path / "config.json").write_text(json.dumps(config))
+    checkpoint.write(str(tmp_path / "model.safetensors"),
+                     {name: torch.from_numpy(values).to(torch.bfloat16) for name, values in tensors.items()})
+
+    def run(program, *arguments, **options):
+        done = subprocess.run([sys.executable, os.path.join(root, "bin", program), *arguments], capture_output=True,
+                              text=True, timeout=300, **options)
+        assert done.returncode == 0, done.stderr[-2000:]
+        return done.stdout
+
+    prompts = [tokens[:9], tokens[20:61]]
+    produced = run("lfm25", "generate", "--model", str(tmp_path), "--dtype", "float32", "--max-new-tokens", "8",
+                   *[word for prompt in prompts for word in ("--tokens", ",".join(map(str, prompt)))]).split()
+    for prompt, line in zip(prompts, produced):
+        expected, margins = greedy_with_margin(config, tensors, prompt, 8)
+        sure = next((i for i, margin in enumerate(margins) if margin < 1e-3), len(expected))
+        assert [int(word) for word in line.split(",")][:sure] == expected[:sure] and sure > 2
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": tokens[:70].tolist(), "want": [3, 69]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": tokens[70:71].tolist(), "want": [0]}], "end": ["a"]},
+             {"step": 2, "entries": [{"id": "a", "tokens": tokens[:2].tolist(), "want": [1]}], "end": ["a"]}]
+    for dtype in TYPES:
+        out = run("trace_run", "--model", str(tmp_path), "--dtype", dtype, "--out", str(tmp_path), "--max-tokens", "80",
+                  input="".join(json.dumps(step) + "\n" for step in steps))
+        assert [line for line in out.splitlines() if line.startswith("done")] == ["done 0", "done 1", "done 2"]
+        for step, places in ((0, [3, 69]), (1, [70]), (2, [1])):
+            got = np.fromfile(tmp_path / f"{step}.f32", dtype="<f4").reshape(len(places), config["vocab"])
+            assert cases.relative_error(got, want[places]).max() <= cases.SHARP[dtype]
+
+
+@pytest.mark.parametrize("portions", [[180], [90, 2, 1, 1, 60, 26], [179, 1]], ids=["whole", "mixed", "decoded"])
+def test_pages_that_hold_not_a_number(device, portions):
+    """What a page held before it was handed out reaches no result: caches full of NaN patterns around the sequence."""
+    import torch
+    config = cases.config_of([cases.latent_layer(6, 64, 32, 32, 48, 96, ff=0), cases.latent_layer(2, kv_rank=40, ff=0)])
+    tensors = cases.random_tensors(config, 89)
+    tokens = np.random.default_rng(91).integers(0, config["vocab"], size=180).astype(np.uint32)
+    want, model = [], cases.oracle_model(config, tensors)
+    model.forward(tokens, model.new_state(), want)
+    for dtype in TYPES:
+        def poisoned(pages, slots):
+            made = cases.product_model(config, tensors, device, dtype, pages, slots)
+            for pair in made.caches:
+                for cache in pair:
+                    cache.fill_(float("nan"))
+            torch.cuda.current_stream().synchronize()
+            return made
+        got = stack_cases.residual_in_portions(poisoned, device, tokens, portions)
+        assert cases.relative_error(got, want[-1]).max() <= {"float32": 1e-5, "bfloat16": 6e-2}[dtype]
