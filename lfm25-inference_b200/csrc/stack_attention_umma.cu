@@ -45,7 +45,7 @@ struct Layout {
     static constexpr uint32_t kSharedBytes = KC * kQueryChunkBytes + kStages * kStageBytes + kControlBytes + 1024;
     static constexpr uint32_t kColumnPv = 2 * kKeys;         // two S buffers in front, two PV buffers behind
     static constexpr uint32_t kTmemColumns = 2 * kKeys + 2 * 64 * VC <= 256 ? 256 : 512;
-    static constexpr uint32_t kCtasPerSm = KC + VC <= 2 ? 2 : 1;
+    static constexpr uint32_t kCtasPerSm = VC == 1 && kTmemColumns <= 256 && kSharedBytes <= 112 * 1024 ? 2 : 1;
     static_assert(2 * kKeys + 2 * 64 * VC <= 512, "tensor memory");
     static_assert(kSharedBytes <= 227 * 1024, "shared memory");
 };
