@@ -765,7 +765,7 @@ int32_t lfm25_stack_executor_step_graph(lfm25_stack_executor* executor, const lf
 int32_t lfm25_stack_executor_forward_ragged(lfm25_stack_executor* executor, const lfm25_ragged_batch* batch,
                                             size_t num_output_rows);
 int32_t lfm25_stack_executor_download_sampled(lfm25_stack_executor* executor, uint32_t* host, size_t count);
-/* Logits of the last step as f32 [rows, vocab] on the host; synchronises the stream. */
+/* Logits of the last step as f32 [rows, vocab] on the host, capped where the model caps them; synchronises the stream. */
 int32_t lfm25_stack_executor_read_logits(lfm25_stack_executor* executor, float* host, size_t rows);
 /* The f32 residual stream entering the final norm, [tokens, width]: what `layers` layers of the last step's tokens left
  * (layers counts from 1).  A debugging and test aid: runs the next steps' layers only up to `layers` when set with

@@ -194,7 +194,8 @@ stack_attention_umma_kernel(const __grid_constant__ CUtensorMap query_map, const
             mbar_arrive_expect_tx(bar_q, KC * group * p.tile_tokens * 128);
             for (uint32_t chunk = 0; chunk < KC; ++chunk) {
                 // a query dimension beyond a part of the head meets a key dimension that the copy filled with zero
-                const uint32_t x = EXPANDED && chunk >= p.own_chunks ? p.own_dim + (chunk - p.own_chunks) * 64 : chunk * 64;
+                const bool shared_part = EXPANDED && chunk >= p.own_chunks;
+                const uint32_t x = shared_part ? p.own_dim + (chunk - p.own_chunks) * 64 : chunk * 64;
                 tma_load_box_3d(q_base + chunk * kQueryChunkBytes, &query_map, bar_q, static_cast<int32_t>(x),
                                 static_cast<int32_t>(kv_head * group), static_cast<int32_t>(tile.first));
             }

@@ -347,8 +347,9 @@ int32_t run_latent_attention(lfm25_stack_executor* self, const Step& step, const
     post.eps = model.norm_eps;
     STACK_CUDA(lfm25::launch_latent_projection(stream, post), "latent projection launch failed");
     STACK_TRY(linear(self, layer.query_up, self->compressed, self->query, tokens));
-    STACK_CUDA(lfm25::launch_rotate_queries(stream, self->type, self->query, layer.query_up.n, layer.inv_freq, step.positions, tokens,
-                                            layer.heads, layer.dim, layer.rot_dim, layer.rot_dims),
+    STACK_CUDA(lfm25::launch_rotate_queries(stream, self->type, self->query, layer.query_up.n, layer.inv_freq,
+                                            step.positions, tokens, layer.heads, layer.dim, layer.rot_dim,
+                                            layer.rot_dims),
                "query rotation launch failed");
     const unsigned char* gate = static_cast<const unsigned char*>(self->projected) + gate_column(layer) * bytes;
     const bool expand = expands_contexts(self, step, layer);
@@ -759,8 +760,8 @@ int32_t lfm25_stack_executor_create(lfm25_blaslt* blaslt, const lfm25_stack_mode
         model->final_norm == nullptr || model->head.weight == nullptr || model->records == nullptr) {
         return lfm25::report_error(LFM25_ERR_NULL_POINTER, "stack model is incomplete");
     }
-    if (model->activation > LFM25_ACTIVATION_F32 || model->block > LFM25_BLOCK_SANDWICH || model->width == 0 || model->vocab == 0 ||
-        model->head.n < model->vocab || model->head.k != model->width || model->record_bytes % 256 != 0 ||
+    if (model->activation > LFM25_ACTIVATION_F32 || model->block > LFM25_BLOCK_SANDWICH || model->width == 0 ||
+        model->vocab == 0 || model->head.n < model->vocab || model->head.k != model->width || model->record_bytes % 256 != 0 ||
         model->num_request_slots == 0 || model->num_pages == 0) {
         return lfm25::report_error(LFM25_ERR_INVALID_ARGUMENT, "stack model sizes are inconsistent");
     }
@@ -828,7 +829,8 @@ int32_t lfm25_stack_executor_create(lfm25_blaslt* blaslt, const lfm25_stack_mode
                             t * joined * bytes, t * model->width * bytes, r * model->width * bytes,
                             r * model->head.n * bytes, t * raw * 4, r * 4, t * compressed * bytes, t * latents * bytes,
                             t * latents * bytes, c * context_rank * bytes, c * context_keys * bytes,
-                            c * context_columns * bytes, (t + 1) * 4, latents > 0 ? t * 4 : 0, t * channels * bytes, t * scanned * bytes};
+                            c * context_columns * bytes, (t + 1) * 4, latents > 0 ? t * 4 : 0, t * channels * bytes,
+                            t * scanned * bytes};
     size_t total = 0;
     for (size_t size : sizes) total += (size + 255) & ~static_cast<size_t>(255);
     cudaError_t status = cudaMalloc(&self->allocation, total);

@@ -132,7 +132,8 @@ cudaError_t launch_projection(cudaStream_t stream, const LatentProjectionLaunch&
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
 rotate_queries_kernel(T* __restrict__ query, size_t token_pitch, const float* __restrict__ inv_freq,
-                      const uint32_t* __restrict__ positions, uint32_t heads, uint32_t dim, uint32_t rot_dim, uint32_t half) {
+                      const uint32_t* __restrict__ positions, uint32_t heads, uint32_t dim, uint32_t rot_dim,
+                      uint32_t half) {
     pdl_launch_dependents();
     extern __shared__ float2 angles[];                // [half] (cos, sin)
     pdl_wait();
@@ -187,7 +188,8 @@ latent_attention_plain_kernel(const LatentArgs<T> args, uint32_t head_blocks) {
     for (uint32_t i = threadIdx.x; i < kPlainHeads * shape.kv_rank; i += kPlainThreads) {
         const uint32_t head = i / shape.kv_rank;
         latent_query[i] =
-            head < count ? to_float<T>(args.absorbed[(token * shape.heads + head0) * shape.kv_rank + i]) * shape.scale : 0.0f;
+            head < count ? to_float<T>(args.absorbed[(token * shape.heads + head0) * shape.kv_rank + i]) * shape.scale
+                         : 0.0f;
         sum[i] = 0.0f;
     }
     for (uint32_t i = threadIdx.x; i < kPlainHeads * shape.rot_dim; i += kPlainThreads) {

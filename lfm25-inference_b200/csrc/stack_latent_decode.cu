@@ -9,8 +9,8 @@
 //   warp 1      tensor memory and the MMAs: S^T [64 keys, heads] = K Q^T over all chunks, then O^T [kv_rank, heads] +=
 //               latent^T P^T over the same shared memory, now read with the latent dimensions as rows
 //   others      one key per thread (lanes 0 .. 15; two or four warps share a quadrant of tensor memory and divide the heads
-//               among them): mask and softmax weights in f32.  The weights are taken against a reference that follows the running
-//               maximum only when it falls more than 2^8 behind; then the accumulators in tensor memory are rescaled
+//               among them): mask and softmax weights in f32.  The weights are taken against a reference that follows the
+//               running maximum only when it falls more than 2^8 behind; then the accumulators in tensor memory are rescaled
 // The weights enter the second product as a sum of two bf16 values (16 significant bits), the two parts as neighbouring
 // columns of one MMA; sums and accumulators are f32.  The splits of a token merge through the distributed shared memory of
 // their cluster.
@@ -87,13 +87,6 @@ struct Control {
     volatile uint32_t failed[2];
 };
 
-// MMAs that add to the same accumulator wait for one another, which small ones feel: the steps of a score take turns among
-// this many accumulators, which the softmax adds up.
-template <uint32_t N>
-constexpr __host__ __device__ uint32_t score_sums() {
-    return N <= 32 ? 4 : 2;
-}
-
 template <uint32_t N>
 constexpr size_t shared_bytes(uint32_t chunks, uint32_t stages) {
     return 1024 + static_cast<size_t>(chunks) * N * 128 + 4 * N * 128 +
@@ -112,7 +105,8 @@ __device__ __forceinline__ void mma_shared(uint32_t tmem_d, uint64_t desc_a, uin
         : "memory");
 }
 
-__device__ __forceinline__ void load_3d(uint32_t dst, const void* tensor_map, uint32_t bar, int32_t x, int32_t y, int32_t z) {
+__device__ __forceinline__ void load_3d(uint32_t dst, const void* tensor_map, uint32_t bar, int32_t x, int32_t y,
+                                        int32_t z) {
     asm volatile(
         "cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
         ::"r"(dst), "l"(reinterpret_cast<uint64_t>(tensor_map)), "r"(bar), "r"(x), "r"(y), "r"(z)
@@ -122,7 +116,8 @@ __device__ __forceinline__ void load_3d(uint32_t dst, const void* tensor_map, ui
 __device__ __forceinline__ void load_4d(uint32_t dst, const void* tensor_map, uint32_t bar, int32_t x, int32_t y, int32_t z,
                                         int32_t w) {
     asm volatile(
-        "cp.async.bulk.tensor.4d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6}], [%2];"
+        "cp.async.bulk.tensor.4d.shared::cluster.global.tile.mbarrier::complete_tx::bytes "
+        "[%0], [%1, {%3, %4, %5, %6}], [%2];"
         ::"r"(dst), "l"(reinterpret_cast<uint64_t>(tensor_map)), "r"(bar), "r"(x), "r"(y), "r"(z), "r"(w)
         : "memory");
 }
@@ -166,14 +161,15 @@ __device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.w
 
 template <uint32_t N>
 __global__ void __launch_bounds__(cta_threads(N), 1)
-latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, const __grid_constant__ CUtensorMap rotated_map,
-                             const __grid_constant__ CUtensorMap latent_map, const __grid_constant__ CUtensorMap tail_map,
+latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map,
+                             const __grid_constant__ CUtensorMap rotated_map,
+                             const __grid_constant__ CUtensorMap latent_map,
+                             const __grid_constant__ CUtensorMap tail_map,
                              const __grid_constant__ CUtensorMap key_map, const Params p) {
     constexpr uint32_t kSharing = sharing_warps(N);
     constexpr uint32_t kShare = N / kSharing;       // heads per softmax thread
     constexpr uint32_t kSoftmax = softmax_threads(N);
     constexpr uint32_t kThreads = cta_threads(N);
-    constexpr uint32_t kSums = score_sums<N>();
     const uint32_t warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0);     // the same value to the compiler's eye as well
     const uint32_t lane = threadIdx.x & 31;
     extern __shared__ uint8_t latent_smem[];
@@ -226,7 +222,7 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
     // a CTA writes into the others' shared memory at its end, which may come before they have started
     if (p.splits > 1) cluster_arrive();
     const uint32_t tmem_base = __shfl_sync(0xffffffffu, *reinterpret_cast<volatile uint32_t*>(&control.tmem), 0);
-    const uint32_t tmem_out = tmem_base + 2 * kSums * N;         // [block][high heads | low heads]
+    const uint32_t tmem_out = tmem_base + 2 * N;                 // [block][high heads | low heads]
     pdl_wait();
 
     const uint32_t split = blockIdx.x % p.splits;
@@ -296,7 +292,8 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
                     const int32_t row = static_cast<int32_t>(source * kPageSize);
                     const uint32_t target = ring + stage * stage_bytes + offset;
                     if (part < 2) {
-                        load_4d(target, &latent_map, bar, 0, 0, 0, row / static_cast<int32_t>(kGroupKeys) + static_cast<int32_t>(part));
+                        load_4d(target, &latent_map, bar, 0, 0, 0,
+                                row / static_cast<int32_t>(kGroupKeys) + static_cast<int32_t>(part));
                     } else if (part < 4) {
                         tma_load_2d(target, &tail_map, bar, 0, row + static_cast<int32_t>((part - 2) * kGroupKeys));
                     } else {
@@ -334,7 +331,7 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
             bool ok = mbar_wait_bounded(bar_query, 0, p.wait_limit);
             auto issue_scores = [&](uint32_t index) {       // the stage has arrived
                 tcgen05_fence_after();
-                const uint32_t target = tmem_base + (index & 1) * kSums * N;
+                const uint32_t target = tmem_base + (index & 1) * N;
                 const uint32_t stage = ring + index % p.stages * stage_bytes;
                 if (issuer) {
                     uint64_t k_desc = descriptor(stage, group_bytes, 16);
@@ -343,8 +340,7 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
                         if (chunk == p.latent_chunks) k_desc = descriptor(stage + kGroups * group_bytes, kChunkBytes, 16);
 #pragma unroll
                         for (uint32_t ks = 0; ks < 4; ++ks) {   // 16 dimensions = 32 bytes inside the swizzled row per step
-                            mma_shared(target + ks % kSums * N, k_desc + ks * 2, q_desc + ks * 2, idesc_scores,
-                                       chunk + ks / kSums);
+                            mma_shared(target, k_desc + ks * 2, q_desc + ks * 2, idesc_scores, chunk + ks);
                         }
                         k_desc += (chunk < p.latent_chunks ? kChunkBytes : kGroups * kChunkBytes) >> 4;
                         q_desc += N * 128 >> 4;
@@ -363,7 +359,7 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
                 const uint32_t stage = index % p.stages;
                 const uint32_t buffer = index & 1;
                 const uint32_t present = pages_of(index);
-                // the next stage's scores first if it is there: the tensor core computes them while this stage's softmax runs
+                // the next stage's scores first if it is there: the tensor core computes them during this stage's softmax
                 bool ahead = false;
                 if (index + 1 < count) {
                     ahead = __all_sync(0xffffffffu, mbar_test(bar_full + 8 * ((index + 1) % p.stages),
@@ -424,18 +420,12 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
             bool over = false;
 #pragma unroll
             for (uint32_t part = 0; part < kShare / 8; ++part) {
-                uint32_t raw[kSums][8];
-#pragma unroll
-                for (uint32_t way = 0; way < kSums; ++way) {
-                    tmem_load8_nowait(tmem_base + lane_address + (buffer * kSums + way) * N + first_head + part * 8, raw[way]);
-                }
+                uint32_t raw[8];
+                tmem_load8_nowait(tmem_base + lane_address + buffer * N + first_head + part * 8, raw);
                 tmem_load_wait();
 #pragma unroll
                 for (uint32_t i = 0; i < 8; ++i) {
-                    float value = __uint_as_float(raw[0][i]);
-#pragma unroll
-                    for (uint32_t way = 1; way < kSums; ++way) value += __uint_as_float(raw[way][i]);
-                    value = visible ? value * scale_log2 : -INFINITY;
+                    const float value = visible ? __uint_as_float(raw[i]) * scale_log2 : -INFINITY;
                     score[part * 8 + i] = value;
                     over |= value > control.reference[first_head + part * 8 + i] + kSlack;
                 }
@@ -600,7 +590,8 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
             uint2 packed;
             packed.x = pack_bf16x2(value.x * share, value.y * share);
             packed.y = pack_bf16x2(value.z * share, value.w * share);
-            *reinterpret_cast<uint2*>(p.out + (static_cast<size_t>(token) * p.heads + head0) * p.kv_rank + item * 4) = packed;
+            *reinterpret_cast<uint2*>(p.out + (static_cast<size_t>(token) * p.heads + head0) * p.kv_rank + item * 4) =
+                packed;
         }
         return;
     }
@@ -650,7 +641,8 @@ latent_attention_umma_kernel(const __grid_constant__ CUtensorMap absorbed_map, c
         const float4* parts[kSplits];
 #pragma unroll
         for (uint32_t rank = 0; rank < kSplits; ++rank) {
-            parts[rank] = reinterpret_cast<const float4*>(cluster.map_shared_rank(reinterpret_cast<float*>(ring_bytes), rank));
+            parts[rank] =
+                reinterpret_cast<const float4*>(cluster.map_shared_rank(reinterpret_cast<float*>(ring_bytes), rank));
         }
         for (uint32_t item = split * mine + threadIdx.x; item < last_item; item += kThreads) {
             const uint32_t head = item / quads;
@@ -777,7 +769,7 @@ cudaError_t launch_heads(cudaStream_t stream, const LatentAttentionLaunch& launc
     params.splits = latent_attention_splits(launch.tokens * params.head_blocks, launch.context, params.latent_chunks);
     params.stages = stages_for<N>(shape);
     params.tmem_columns = 32;
-    while (params.tmem_columns < (2 * score_sums<N>() + 2 * params.blocks) * N) params.tmem_columns *= 2;
+    while (params.tmem_columns < (2 + 2 * params.blocks) * N) params.tmem_columns *= 2;
     params.wait_limit = wait_limit_ns();
     const size_t shared = shared_bytes<N>(params.chunks, params.stages);
     const auto kernel = latent_attention_umma_kernel<N>;
@@ -785,8 +777,8 @@ cudaError_t launch_heads(cudaStream_t stream, const LatentAttentionLaunch& launc
                                                     cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shared));
     if (status != cudaSuccess) return status;
     const size_t blocks = launch.tokens * params.head_blocks * params.splits;
-    return launch_kernel(kernel, static_cast<unsigned int>(blocks), cta_threads(N), shared, stream, params.splits, absorbed_map,
-                         rotated_map, latent_map, tail_map, key_map, params);
+    return launch_kernel(kernel, static_cast<unsigned int>(blocks), cta_threads(N), shared, stream, params.splits,
+                         absorbed_map, rotated_map, latent_map, tail_map, key_map, params);
 }
 
 }  // namespace
@@ -827,7 +819,7 @@ bool latent_attention_umma_supports(const LatentAttentionLaunch& launch) {
 cudaError_t launch_latent_attention_umma(cudaStream_t stream, const LatentAttentionLaunch& launch) {
     // as many heads per CTA as there are and as fit: the cache is read once per block of heads
     if (launch.shape.heads > 32 && stages_for<64>(launch.shape) > 0 &&
-        (2 * score_sums<64>() + 2 * ((launch.shape.kv_rank + 127) / 128)) * 64 <= 512) {
+        (2 + 2 * ((launch.shape.kv_rank + 127) / 128)) * 64 <= 512) {
         return launch_heads<64>(stream, launch);
     }
     if (launch.shape.heads > 16 && stages_for<32>(launch.shape) > 0) {

@@ -178,8 +178,8 @@ cudaError_t launch_conv(cudaStream_t stream, const ChannelConvLaunch& launch) {
                         launch.record.offset % 16 == 0;
     const size_t per_cta = static_cast<size_t>(kConvThreads) * (vector ? 8 : 1);
     args.channel_blocks = static_cast<uint32_t>((launch.channels + per_cta - 1) / per_cta);
-    void (*kernel)(const ConvArgs<T>) = vector ? (launch.taps == 4 ? channel_conv_kernel<T, 8, 4> : channel_conv_kernel<T, 8, 0>)
-                                               : channel_conv_kernel<T, 1, 0>;
+    void (*kernel)(const ConvArgs<T>) = channel_conv_kernel<T, 1, 0>;
+    if (vector) kernel = launch.taps == 4 ? channel_conv_kernel<T, 8, 4> : channel_conv_kernel<T, 8, 0>;
     return launch_kernel(kernel,
                          static_cast<unsigned int>(tile_bound(launch.segments, args.tile_rows) * args.channel_blocks),
                          kConvThreads, 0, stream, 1, args);

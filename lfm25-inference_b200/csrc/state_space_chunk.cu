@@ -31,7 +31,9 @@ struct Tables {
 };
 
 // Bytes of one buffer of a chunk's B, C and x
-__host__ __device__ constexpr size_t chunk_bytes(uint32_t padded) { return (2 * kTokens * (padded + kPad) + kTokens * kColumnPitch) * 2; }
+__host__ __device__ constexpr size_t chunk_bytes(uint32_t padded) {
+    return (2 * kTokens * (padded + kPad) + kTokens * kColumnPitch) * 2;
+}
 constexpr size_t shared_bytes(uint32_t padded, uint32_t buffers) {
     // state and weighted x, both as two bf16 parts
     return buffers * chunk_bytes(padded) + 2 * (padded + kTokens) * kColumnPitch * 2 + sizeof(Tables);
@@ -88,8 +90,8 @@ state_space_chunk_kernel(const StateSpaceArgs<__nv_bfloat16> args, uint32_t colu
         for (uint32_t item = threadIdx.x; item < kTokens * vectors; item += kThreads) {
             const uint32_t row = item / vectors, n = item % vectors * 8;
             const bool inside = first + row < end && n < args.size;
-            const __nv_bfloat16* source =
-                args.mixed + (inside ? static_cast<size_t>(first + row) * args.mixed_pitch + inner + group * args.size + n : 0);
+            const __nv_bfloat16* source = args.mixed;
+            if (inside) source += static_cast<size_t>(first + row) * args.mixed_pitch + inner + group * args.size + n;
             copy_async_16(b + row * pitch + n, source, inside);
             copy_async_16(c + row * pitch + n, source + (inside ? args.groups * args.size : 0), inside);
         }
@@ -178,7 +180,8 @@ state_space_chunk_kernel(const StateSpaceArgs<__nv_bfloat16> args, uint32_t colu
                     for (uint32_t half = 0; half < 2; ++half) {
                         uint32_t high, low;
                         split_pair(held[unit][tile][2 * half], held[unit][tile][2 * half + 1], high, low);
-                        const uint32_t at = (piece / 2 * 16 + row0 + half * 8) * kColumnPitch + piece % 2 * 32 + tile * 8 + pair;
+                        const uint32_t row = piece / 2 * 16 + row0 + half * 8;
+                        const uint32_t at = row * kColumnPitch + piece % 2 * 32 + tile * 8 + pair;
                         *reinterpret_cast<uint32_t*>(state_high + at) = high;
                         *reinterpret_cast<uint32_t*>(state_low + at) = low;
                     }
@@ -361,8 +364,8 @@ cudaError_t launch_state_space_chunk(cudaStream_t stream, const StateSpaceLaunch
     const uint32_t column_blocks = (launch.vdim + kColumns - 1) / kColumns;
     const size_t blocks = launch.segments.num_segments * launch.heads * column_blocks;
     // two CTAs per SM hide each other's loads; where there are not enough of them, a second buffer does
-    const uint32_t buffers =
-        blocks <= 148 || shared_bytes(padded, 1) > kSharedLimit / 2 - 1024 ? (shared_bytes(padded, 2) <= kSharedLimit ? 2 : 1) : 1;
+    const bool alone = blocks <= 148 || shared_bytes(padded, 1) > kSharedLimit / 2 - 1024;
+    const uint32_t buffers = alone && shared_bytes(padded, 2) <= kSharedLimit ? 2 : 1;
     const size_t shared = shared_bytes(padded, buffers);
     const auto kernel = padded <= 64    ? state_space_chunk_kernel<1>
                         : padded <= 128 ? state_space_chunk_kernel<2>
