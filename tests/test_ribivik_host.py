@@ -48,7 +48,7 @@ def test_recurrence_step_by_hand():
     assert np.allclose(new, want) and np.allclose(y, want[0] - want[1] + 0.5 * want[2] + 7.0 * x)
 
 
-def test_gate_comes_before_the_norm_of_each_part():
+def test_gated_output_is_normed_part_by_part():
     y, z = np.array([[1.0, 2.0, 3.0, 4.0]]), np.array([[0.5, -1.0, 2.0, 0.0]])
     gated = y * z / (1.0 + np.exp(-z))
     want = np.concatenate([part / np.sqrt((part ** 2).mean() + 0.1) for part in (gated[0, :2], gated[0, 2:])])
